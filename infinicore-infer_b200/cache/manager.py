@@ -45,6 +45,10 @@ class StateViews:
     def __len__(self) -> int:
         return len(self.views)
 
+    def rest(self, first: int) -> "StateViews":
+        """The tensors from ``first`` on: what a part hands to another whose states follow its own."""
+        return StateViews(self.views[first:])
+
 
 class CacheManager:
     def __init__(self, needs: Sequence[object], num_pages: int, page_size: int, max_requests: int,

@@ -1,5 +1,6 @@
 """Configuration: typed specifications, the MiniCPM/FM9G config, the architecture registry."""
-from .specs import (AttentionSpec, BlockSpec, ConfigError, ConvAttentionSpec, FrequencyRampSpec, GLUSpec, LatentAttentionSpec,
+from .specs import (AttentionSpec, BlockSpec, ConfigError, ConvAttentionSpec, FrequencyBandSpec, FrequencyRampSpec, GLUSpec,
+                    LatentAttentionSpec, ParallelBlockSpec,
                     DeltaRuleSpec, StepVectorSpec, LayerNormSpec, LinearAttentionSpec, MLPSpec, ModelSpec, PairRotarySpec, ParallelMixerSpec, PostNormBlockSpec, ReinjectSpec, RMSNormSpec,
                     RopeSpec, RoutedExpertsSpec, RunEntry, SandwichBlockSpec, SelectiveScanSpec, SwiGLUSpec, default_order)
 from .minicpm import MiniCPMConfig
@@ -7,6 +8,7 @@ from .sitelorn import SitelornConfig
 from .vunelix import VunelixConfig
 from .vipovik import VipovikConfig
 from .fapenex import FapenexConfig
+from .fupapel import FupapelConfig
 from .presets import PRESETS, Preset
 from .registry import (architecture_names, config_class_for, read_config,
                        register_architecture)
@@ -19,9 +21,11 @@ register_architecture("sitelorn", SitelornConfig)
 register_architecture("vunelix", VunelixConfig)
 register_architecture("vipovik", VipovikConfig)
 register_architecture("fapenex", FapenexConfig)
+register_architecture("fupapel", FupapelConfig)
 
 __all__ = [
     "DeltaRuleSpec", "StepVectorSpec", "FapenexConfig",
+    "FrequencyBandSpec", "FupapelConfig", "ParallelBlockSpec",
     "MLPSpec", "ParallelMixerSpec", "VipovikConfig",
     "FrequencyRampSpec", "LatentAttentionSpec", "ReinjectSpec", "RoutedExpertsSpec", "SandwichBlockSpec", "SelectiveScanSpec", "VunelixConfig",
     "ConvAttentionSpec", "GLUSpec", "LayerNormSpec", "LinearAttentionSpec", "PairRotarySpec", "PostNormBlockSpec", "SitelornConfig",

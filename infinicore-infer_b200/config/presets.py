@@ -97,4 +97,21 @@ PRESETS: Dict[str, Preset] = {
             {"type": "latent_attention", "mixer": {"heads": 3, "dim": 16, "vdim": 24, "kv_rank": 32, "q_rank": 40, "scale": 0.25,
                                                    "mask": {"size": 17}}, "mlp": None},
         ]), 0.1, 0.05, 16),
+    # a small Fupapel: mixers and feed-forwards side by side behind a token shift, one layer of each mixer and one that borrows
+    # its keys, routed experts with identities in groups and a layer without feed-forward
+    "fupapel-tiny": Preset(dict(
+        architecture="Fupapel", vocab=320, width=96, norm={"eps": 1e-5}, residual_mult=0.8, layers=[
+            {"type": "attention_2", "mixer": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 24, "scale": 0.25, "conv": 3, "mask": {"size": 24},
+                                              "rot": {"base": 1e4, "dims": 16, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 64}}},
+             "mlp": {"kind": "moe", "router": {"experts": 6, "identity": 2, "top": 2, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": 48}}},
+            {"type": "attention", "mixer": {"heads": 4, "kv_heads": 1, "dim": 32, "vdim": 16, "scale": 0.2, "mask": {"size": 40},
+                                            "rot": {"base": 5e4, "dims": 8}},
+             "mlp": {"kind": "moe", "router": {"experts": 4, "identity": 1, "top": 2, "groups": {"count": 1, "keep": 1}}, "expert": {"ff": 64}}},
+            {"type": "latent_attention", "mixer": {"heads": 3, "dim": 16, "rot_dim": 8, "vdim": 24, "kv_rank": 32, "q_rank": 40, "scale": 0.25,
+                                                   "rot": {"base": 1e5, "dims": 8}}, "mlp": None},
+            {"type": "attention_2", "mixer": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 24, "scale": 0.25, "conv": 2, "mask": {"size": 32},
+                                              "rot": {"base": 1e4, "dims": 16, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 64}},
+                                              "kv_from": 0},
+             "mlp": {"kind": "moe", "router": {"experts": 3, "identity": 3, "top": 2, "groups": {"count": 3, "keep": 2}}, "expert": {"ff": 32}}},
+        ]), 0.1, 0.05, 16),
 }

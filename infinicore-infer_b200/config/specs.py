@@ -97,30 +97,57 @@ class FrequencyRampSpec:
     slow: float
     magnitude_slope: float = 0.1
 
+    def stretch(self, f, dims: int, base: float):
+        """(stretched frequencies, the factor of cos and sin) from the plain frequencies."""
+        import math
+        where = lambda turns: dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+        lo, hi = max(math.floor(where(self.fast)), 0), min(math.ceil(where(self.slow)), dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dims // 2)]
+        return [fi / self.factor * r + fi * (1.0 - r) for fi, r in zip(f, ramp)], self.magnitude_slope * math.log(self.factor) + 1.0
+
+
+@dataclass(frozen=True)
+class FrequencyBandSpec:
+    """Another stretching of a rotation (Llama 3.1's): a pair of frequency f keeps it where its wavelength 2 pi / f is below
+    ``original`` / ``high``, gets f / ``factor`` where it is above ``original`` / ``low``, and between the two the mixture
+    (1 - s) f / factor + s f with s = (original / wavelength - low) / (high - low).  Cos and sin keep their magnitude."""
+    factor: float
+    original: float
+    low: float
+    high: float
+
+    def stretch(self, f, dims: int, base: float):
+        """(stretched frequencies, the factor of cos and sin) from the plain frequencies."""
+        import math
+        out = []
+        for fi in f:
+            turns = self.original * fi / (2.0 * math.pi)         # wavelengths that fit into `original`
+            if turns < self.low:
+                out.append(fi / self.factor)
+            elif turns > self.high:
+                out.append(fi)
+            else:
+                s = (turns - self.low) / (self.high - self.low) if self.high > self.low else 1.0
+                out.append((1.0 - s) * fi / self.factor + s * fi)
+        return out, 1.0
+
 
 @dataclass(frozen=True)
 class PairRotarySpec:
     """Rotation of the first ``dims`` elements of a head in pairs by the angle ``p * base ** (-2i / dims)``, formed in
     float32 from the position; the other elements pass unchanged.  ``layout`` "pairs": pair i is elements (2i, 2i+1);
     "halves": elements (i, i + dims / 2).  Needs no table and no longest position.  ``scaling`` stretches the frequencies
-    (``FrequencyRampSpec``)."""
+    (``FrequencyRampSpec``, ``FrequencyBandSpec``)."""
     dims: int
     base: float
-    scaling: Optional[FrequencyRampSpec] = None
+    scaling: Optional[object] = None
     layout: str = "pairs"
     kind: str = "pair_rotary"
 
     def frequencies(self):
         """(f_i for i < dims / 2 in float64, the factor of cos and sin)."""
-        import math
         f = [float(self.base) ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
-        s = self.scaling
-        if s is None:
-            return f, 1.0
-        where = lambda turns: self.dims * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
-        lo, hi = max(math.floor(where(s.fast)), 0), min(math.ceil(where(s.slow)), self.dims - 1)
-        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(self.dims // 2)]
-        return [fi / s.factor * r + fi * (1.0 - r) for fi, r in zip(f, ramp)], s.magnitude_slope * math.log(s.factor) + 1.0
+        return (f, 1.0) if self.scaling is None else self.scaling.stretch(f, self.dims, float(self.base))
 
 
 @dataclass(frozen=True)
@@ -138,7 +165,11 @@ class ConvAttentionSpec:
     Further options: ``bias``: q, k and v have biases (``q`` + ``bias_suffix``), added in the projection; ``head_norm``
     "before_rotation": every head of q and k passes an RMS norm BEFORE the rotation, with one weight of ``head_dim`` per
     projection shared by its heads (``q`` + ``norm_suffix``), eps ``qk_norm_eps``; ``chunk`` C (instead of a window): a query
-    at position i sees the keys j <= i with floor(j / C) = floor(i / C), chunks counted from position 0 of the sequence."""
+    at position i sees the keys j <= i with floor(j / C) = floor(i / C), chunks counted from position 0 of the sequence;
+    ``element_gate``: every element of the heads' outputs side by side is multiplied by the sigmoid of its own row of
+    ``gate_name`` [heads * v_head_dim, hidden] (instead of one gate per head); ``temp_name``: a tensor [heads] that
+    multiplies the heads' scores; ``sink_name``: with ``sink`` a tensor [heads], the scores of the heads' sinks (neither
+    scaled nor multiplied by ``temp_name``), instead of 0."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -166,6 +197,9 @@ class ConvAttentionSpec:
     bias: bool = False
     bias_suffix: str = ".b"
     chunk: Optional[int] = None
+    element_gate: bool = False
+    temp_name: Optional[str] = None
+    sink_name: Optional[str] = None
     kind: str = "conv_attention"
 
 
@@ -232,7 +266,8 @@ class LatentAttentionSpec:
 
     ``q_rank`` > 0: the queries go through a latent of their own, c_q = RMSnorm(``q_down_name`` h) with the weight
     ``q_down_name`` + ``norm_suffix``, q = ``q_up_name`` c_q.  ``window`` W: a query at position i sees the keys j with
-    0 <= i - j < W.  ``rot_dim`` may be 0 (no rotated part)."""
+    0 <= i - j < W.  ``rot_dim`` may be 0 (no rotated part).  ``output_gate`` "head": one gate per head (``gate_name`` [heads,
+    hidden]).  ``sink_name``: a tensor [heads] with the score of one more key per head that has no value (not scaled)."""
     hidden_size: int
     num_heads: int
     head_dim: int
@@ -242,8 +277,9 @@ class LatentAttentionSpec:
     softmax_scale: float
     norm_eps: float
     position: Optional[PairRotarySpec] = None
-    output_gate: bool = True
+    output_gate: object = True         # False, True (a gate per element) or "head"
     window: Optional[int] = None
+    sink_name: Optional[str] = None
     q_rank: int = 0
     q_down_name: str = "dq"
     q_up_name: str = "uq"
@@ -290,6 +326,11 @@ class RoutedExpertsSpec:
     their sum (+ 1e-20) and multiply the units' OUTPUTS (``scale_input`` False); that is the softmax over the chosen
     logits alone.  ``act`` "swish_clamp": a unit's inner value is g' sigmoid(1.702 g') (u' + 1) with g' = min(gate h, limit),
     u' = clamp(up h, -limit, limit).  ``router_bias``: the logits are router h + ``router_name`` + ``bias_suffix``.
+    ``score_form`` "softmax": scores are softmax(router h) over all outputs, and the chosen ones' scores multiply the units'
+    outputs as they are.  With it: ``correction_name``, a tensor that is added to the scores for the choice only;
+    ``num_identity`` router outputs behind the experts' stand for units that return their input and have no matrices;
+    ``groups`` (count, keep): the outputs form ``count`` groups of neighbours, and only those of the ``keep`` groups whose best
+    choice score is largest can be chosen.
     ``shared_gate_name``: the shared unit's output is multiplied by sigmoid(w . h), one number per row, w that tensor
     ([1, hidden], below ``shared_prefix``)."""
     hidden_size: int
@@ -305,6 +346,9 @@ class RoutedExpertsSpec:
     router_bias: bool = False
     bias_suffix: str = ".b"
     shared_gate_name: Optional[str] = None
+    num_identity: int = 0
+    correction_name: Optional[str] = None
+    groups: Optional[Tuple[int, int]] = None
     expert_prefix: str = "e{}."
     shared_prefix: str = "shared."
     gate_name: str = "gate"
@@ -446,6 +490,25 @@ class PostNormBlockSpec:
     mixer_norm_prefix: str = "norm1"
     ffn_norm_prefix: str = "norm2"
     kind: str = "postnorm"
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """One layer whose two sublayers stand side by side, each behind a norm of its own of the same stream:
+    x += s * (mixer(shift(norm_a(x))) + feed_forward(norm_b(x))).  ``feed_forward`` None: the layer has a mixer only.
+    ``shift_name``: a tensor [hidden] below the layer's prefix; what the mixer reads is h_t + (h_(t-1) - h_t) * that tensor,
+    h the norm's output (h_(-1) = 0); None: h itself."""
+    mixer: object
+    feed_forward: Optional[object]
+    mixer_norm: object
+    ffn_norm: Optional[object]
+    residual_scale: float = 1.0
+    shift_name: Optional[str] = None
+    mixer_prefix: str = "mix."
+    ffn_prefix: str = "mlp."
+    mixer_norm_prefix: str = "norm1"
+    ffn_norm_prefix: str = "norm2"
+    kind: str = "parallel_block"
 
 
 @dataclass(frozen=True)

@@ -30,8 +30,9 @@ struct AttnArgs {
     int T, nh, nkvh, dh, page_size, max_blocks, window;
     float scale;
     // what only the row kernel takes: values of another size than the keys (v_pages [pages, nkvh, page_size, dv], out
-    // [T, nh, dv]), a sink (a key of score 0 without a value: one more term, exp(0), in the normaliser), and a float32
-    // gate per row and head whose sigmoid multiplies the head's output (gate[t * gate_ld + h]; null: none)
+    // [T, nh, dv]); and a sink (a key without a value whose score is sink_w[h], 0 where sink_w is null: one more term in
+    // the normaliser), and a float32 gate whose sigmoid multiplies the output: gate[t * gate_ld + h] a head's (null: none),
+    // or with gate_elem gate[t * gate_ld + h * dv + e] each element's
     int dv, sink;
     const float *gate;
     int gate_ld;
@@ -39,6 +40,8 @@ struct AttnArgs {
     // when the window has passed them
     float cap;
     int keep_first;
+    const float *sink_w;
+    int gate_elem;
 };
 
 // ---------------------------------------------------------------------------------------
@@ -119,20 +122,22 @@ attention_row_kernel(AttnArgs a) {
         }
     }
     }
-    if (a.sink) {       // one more key of score 0 that brings no value
-        const float m_new = fmaxf(m, 0.f);
+    if (a.sink) {       // one more key that brings no value
+        const float sink = a.sink_w != nullptr ? a.sink_w[h] : 0.f;
+        const float m_new = fmaxf(m, sink);
         const float corr = expf(m - m_new);
-        l = l * corr + expf(-m_new);
+        l = l * corr + expf(sink - m_new);
 #pragma unroll
         for (int i = 0; i < NS; ++i) acc[i] *= corr;
     }
     T *orow = (T *)a.out + ((size_t)t * a.nh + h) * dv;
     float inv = 1.f / l;
-    if (a.gate != nullptr) inv *= 1.f / (1.f + expf(-a.gate[(size_t)t * a.gate_ld + h]));
+    const float *gate = a.gate != nullptr ? a.gate + (size_t)t * a.gate_ld + (size_t)h * (a.gate_elem ? dv : 1) : nullptr;
+    if (gate != nullptr && !a.gate_elem) inv *= jk_sigmoid(gate[0]);
 #pragma unroll
     for (int i = 0; i < NS; ++i) {
         const int e = lane + 32 * i;
-        if (e < dv) orow[e] = from_f32<T>(acc[i] * inv);
+        if (e < dv) orow[e] = from_f32<T>(acc[i] * inv * (a.gate_elem && gate != nullptr ? jk_sigmoid(gate[e]) : 1.f));
     }
 }
 
@@ -148,14 +153,14 @@ JK_EXPORT int jk_attention_rows(const void *q, const void *k_pages, const void *
                                 int dtype, const int *positions, const int *row_req,
                                 const int *block_table, int max_blocks, int page_size, int T, int nh,
                                 int nkvh, int dh, float scale, int window, int dv, int sink, const float *gate, int gate_ld,
-                                float cap, int keep_first, cudaStream_t stream) {
+                                float cap, int keep_first, const float *sink_w, int gate_elem, cudaStream_t stream) {
     if (T == 0) return JK_OK;
     if (dv <= 0) dv = dh;
     AttnArgs a{q, k_pages, v_pages, out, positions, row_req, block_table,
-               T, nh, nkvh, dh, page_size, max_blocks, window, scale, dv, sink, gate, gate_ld, cap, window > 0 ? keep_first : 0};
+               T, nh, nkvh, dh, page_size, max_blocks, window, scale, dv, sink, gate, gate_ld, cap, window > 0 ? keep_first : 0, sink_w, gate_elem};
     if (int rc = check_args(a)) return rc;
     JK_REQUIRE(dh <= ROW_MAX_DH && dv <= ROW_MAX_DH, "attention: head size %d / %d exceeds %d", dh, dv, ROW_MAX_DH);
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh, "attention: a gate row of %d holds no %d heads", gate_ld, nh);
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dv : 1), "attention: a gate row of %d holds no %d heads", gate_ld, nh);
     JK_REQUIRE(T <= 65535, "attention: %d rows exceed one launch (65535)", T);
     dim3 grid((nh + ROW_WARPS - 1) / ROW_WARPS, T);
     const size_t smem = (size_t)ROW_WARPS * dh * sizeof(float);
@@ -219,11 +224,13 @@ struct DecodeArgs {
     int nrows, nh, nkvh, dh, page_size, max_blocks, window, splits, page_shift;
     float scale_log2;              // softmax scale * log2(e)
     int cluster;                   // 1: the splits of a row are one thread-block cluster and merge among themselves
-    int sink;                      // 1: every softmax has one more key of score 0 that brings no value
+    int sink;                      // 1: every softmax has one more key that brings no value, of score sink_w[h] (null: 0)
     const float *gate;             // float32 [T, gate_ld]: head h's output is multiplied by sigmoid(gate[t, h]); null: none
     int gate_ld;
     float cap_log2;                // a cap on the scores times log2(e): s <- cap tanh(s / cap) (0: none)
     int keep_first;                // with a window: keys at positions below this stay visible when the window has passed them
+    const float *sink_w;
+    int gate_elem;                 // 1: the gate has one column per output element, gate[t, h dh + e]
 };
 
 // cap tanh(s / cap) through one exponential and one quotient (both to about 1e-7 of their result: the sum of a capped
@@ -244,12 +251,12 @@ struct KeyRange {
     __device__ __forceinline__ int position(int v) const { return v >= lo ? v : v - first; }
 };
 
-// The factor that turns a row's merged accumulator into its output: 1 / L, where L (relative to the maximum M, in units
-// of log2) takes the sink's term 2^(0 - M) if there is a sink, times the head's gate.
-__device__ __forceinline__ float decode_finish(const DecodeArgs &a, float M, float L, int t, int h) {
-    if (a.sink) L += exp2f(-M);
+// The factor that turns element e of a row's merged accumulator into its output: 1 / L, where L (relative to the maximum
+// M, in units of log2) takes the sink's term 2^(sink - M) if there is a sink, times the head's or the element's gate.
+__device__ __forceinline__ float decode_finish(const DecodeArgs &a, float M, float L, int t, int h, int e) {
+    if (a.sink) L += exp2f(jk_sink_log2(a.sink_w, h) - M);
     float f = 1.f / L;
-    if (a.gate != nullptr) f *= 1.f / (1.f + expf(-a.gate[(size_t)t * a.gate_ld + h]));
+    if (a.gate != nullptr) f *= jk_sigmoid(a.gate[(size_t)t * a.gate_ld + (a.gate_elem ? (size_t)h * a.dh + e : (size_t)h)]);
     return f;
 }
 
@@ -448,7 +455,7 @@ attention_decode_kernel(DecodeArgs a) {
         }
         const size_t slot = ((size_t)ri * a.nh + h0 + hh) * a.splits + split;
         if (a.splits == 1) {
-            a.out[((size_t)t * a.nh + h0 + hh) * dh + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + hh));
+            a.out[((size_t)t * a.nh + h0 + hh) * dh + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + hh, e));
         } else {
             a.part_acc[slot * dh + e] = A;
             if (e == 0) { a.part_ml[slot * 2] = M; a.part_ml[slot * 2 + 1] = L; }
@@ -476,7 +483,7 @@ __global__ void attention_combine_kernel(DecodeArgs a) {
             const float ms = a.part_ml[(base + s) * 2];
             if (ms > -INFINITY) A += exp2f(ms - M) * a.part_acc[(base + s) * a.dh + e];
         }
-        a.out[((size_t)t * a.nh + h) * a.dh + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h));
+        a.out[((size_t)t * a.nh + h) * a.dh + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h, e));
     }
 }
 
@@ -516,9 +523,9 @@ JK_EXPORT int jk_attention_decode(const void *q, const void *k_pages, const void
                                   const int *row_req, const int *block_table, int max_blocks,
                                   int page_size, int nh, int nkvh, int dh, float scale, int window,
                                   int splits, int sink, const float *gate, int gate_ld, float cap, int keep_first,
-                                  cudaStream_t stream) {
+                                  const float *sink_w, int gate_elem, cudaStream_t stream) {
     if (nrows == 0) return JK_OK;
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh, "attention_decode: a gate row of %d holds no %d heads", gate_ld, nh);
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dh : 1), "attention_decode: a gate row of %d holds no %d heads", gate_ld, nh);
     JK_REQUIRE(cap >= 0.f && keep_first >= 0, "attention_decode: cap %g, %d kept keys", cap, keep_first);
     JK_REQUIRE(nrows > 0 && nh > 0 && nkvh > 0 && nh % nkvh == 0, "attention_decode: rows %d heads %d/%d", nrows, nh, nkvh);
     JK_REQUIRE(dh % 8 == 0 && dh >= 8 && dh <= 256, "attention_decode: head size %d (takes multiples of 8 up to 256)", dh);
@@ -532,7 +539,8 @@ JK_EXPORT int jk_attention_decode(const void *q, const void *k_pages, const void
                  scratch ? scratch + (size_t)nrows * nh * splits * dh : nullptr,
                  rows, positions, row_req, block_table,
                  nrows, nh, nkvh, dh, page_size, max_blocks, window, splits, 0,
-                 scale * 1.4426950408889634f, 0, sink, gate, gate_ld, cap * 1.4426950408889634f, window > 0 ? keep_first : 0};
+                 scale * 1.4426950408889634f, 0, sink, gate, gate_ld, cap * 1.4426950408889634f, window > 0 ? keep_first : 0,
+                 sink_w, gate_elem};
     const bool pow2 = (page_size & (page_size - 1)) == 0;
     while ((1 << a.page_shift) < page_size) ++a.page_shift;
     const int g = nh / nkvh;
@@ -579,11 +587,13 @@ struct PrefillArgs {
     const int *block_table;  // [nreq, max_blocks]
     int ntiles, nh, nkvh, page_size, max_blocks, window, tile_rows;
     float scale_log2;
-    int sink;                // 1: every softmax has one more key of score 0 that brings no value
+    int sink;                // 1: every softmax has one more key that brings no value, of score sink_w[h] (null: 0)
     const float *gate;       // float32 [T, gate_ld]: head h's output is multiplied by sigmoid(gate[t, h]); null: none
     int gate_ld;
     float cap_raw;           // a cap on the scores divided by the softmax scale: raw s <- cap tanh(s / cap) (0: none)
     int keep_first;          // with a window: keys at positions below this stay visible when the window has passed them
+    const float *sink_w;
+    int gate_elem;           // 1: the gate has one column per output element, gate[t, h DH + e]
 };
 
 constexpr int PF_BM = 64;
@@ -773,17 +783,27 @@ attention_prefill_kernel(PrefillArgs a) {
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
     if (a.sink) {       // the sink's term relative to each row's maximum (raw scores; the exponent is scaled)
-        l_a += exp2f(-m_a * a.scale_log2);
-        l_b += exp2f(-m_b * a.scale_log2);
+        const float sink = jk_sink_log2(a.sink_w, h);
+        l_a += exp2f(sink - m_a * a.scale_log2);
+        l_b += exp2f(sink - m_b * a.scale_log2);
     }
     float inv_a = 1.f / l_a, inv_b = 1.f / l_b;
+    const float *gate_a = nullptr, *gate_b = nullptr;       // with a gate per element: where the two rows' gates of this head start
     if (a.gate != nullptr) {
-        if (row_a < nrows) inv_a *= 1.f / (1.f + expf(-a.gate[(size_t)(row0 + row_a) * a.gate_ld + h]));
-        if (row_b < nrows) inv_b *= 1.f / (1.f + expf(-a.gate[(size_t)(row0 + row_b) * a.gate_ld + h]));
+        const size_t at = (size_t)h * (a.gate_elem ? DH : 1);
+        if (row_a < nrows) gate_a = a.gate + (size_t)(row0 + row_a) * a.gate_ld + at;
+        if (row_b < nrows) gate_b = a.gate + (size_t)(row0 + row_b) * a.gate_ld + at;
+        if (!a.gate_elem) {
+            if (gate_a) inv_a *= jk_sigmoid(*gate_a);
+            if (gate_b) inv_b *= jk_sigmoid(*gate_b);
+            gate_a = gate_b = nullptr;
+        }
     }
 #pragma unroll
     for (int i = 0; i < DH / 8; ++i) {
         const int col = i * 8 + 2 * (lane & 3);
+        if (gate_a) { o[i][0] *= jk_sigmoid(gate_a[col]); o[i][1] *= jk_sigmoid(gate_a[col + 1]); }
+        if (gate_b) { o[i][2] *= jk_sigmoid(gate_b[col]); o[i][3] *= jk_sigmoid(gate_b[col + 1]); }
         if (row_a < nrows)
             *reinterpret_cast<__nv_bfloat162 *>(a.out + ((size_t)(row0 + row_a) * a.nh + h) * DH + col) =
                 __floats2bfloat162_rn(o[i][0] * inv_a, o[i][1] * inv_a);
@@ -1081,7 +1101,7 @@ attention_decode_gqa_kernel(DecodeArgs a) {
             fin[r * DH + e] = A;
             if (e == 0) { fin_ml[2 * r] = M; fin_ml[2 * r + 1] = L; }
         } else if (a.splits == 1) {
-            a.out[((size_t)t * a.nh + h0 + r) * DH + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r));
+            a.out[((size_t)t * a.nh + h0 + r) * DH + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, e));
         } else {
             const size_t slot = pbase + (size_t)r * a.splits;
             a.part_acc[slot * DH + e] = A;
@@ -1106,7 +1126,7 @@ attention_decode_gqa_kernel(DecodeArgs a) {
                         A += f * ld_cluster_f32(fin + idx, p);
                     }
                 }
-                a.out[((size_t)t * a.nh + h0 + r) * DH + (idx % DH)] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r));
+                a.out[((size_t)t * a.nh + h0 + r) * DH + (idx % DH)] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, idx % DH));
             }
         }
         cluster_sync_all();                        // nobody leaves while its shared memory may still be read
@@ -1189,17 +1209,17 @@ JK_EXPORT int jk_attention_prefill(const void *q, const void *k_pages, const voi
                                    const int *tiles, int ntiles, int tile_rows, const int *req_start, const int *req_pos,
                                    const int *block_table, int max_blocks, int page_size, int nh, int nkvh,
                                    int dh, float scale, int window, int sink, const float *gate, int gate_ld, float cap, int keep_first,
-                                   cudaStream_t stream) {
+                                   const float *sink_w, int gate_elem, cudaStream_t stream) {
     if (ntiles == 0) return JK_OK;
     JK_REQUIRE(ntiles > 0 && nh > 0 && nkvh > 0 && nh % nkvh == 0, "attention_prefill: tiles %d heads %d/%d", ntiles, nh, nkvh);
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh, "attention_prefill: a gate row of %d holds no %d heads", gate_ld, nh);
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dh : 1), "attention_prefill: a gate row of %d holds no %d heads", gate_ld, nh);
     JK_REQUIRE(ntiles * (tile_rows / PF_BM) <= 65535, "attention_prefill: %d tiles exceed one launch", ntiles);
     JK_REQUIRE(page_size > 0 && max_blocks > 0, "attention_prefill: page size %d, blocks %d, window %d",
                page_size, max_blocks, window);
     PrefillArgs a{(const __nv_bfloat16 *)q, (const __nv_bfloat16 *)k_pages, (const __nv_bfloat16 *)v_pages,
                   (__nv_bfloat16 *)out, tiles, req_start, req_pos, block_table,
                   ntiles, nh, nkvh, page_size, max_blocks, window, tile_rows, scale * 1.4426950408889634f, sink, gate, gate_ld,
-                  cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0};
+                  cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w, gate_elem};
     JK_REQUIRE(cap >= 0.f && keep_first >= 0 && scale > 0.f, "attention_prefill: cap %g, %d kept keys, scale %g", cap, keep_first, scale);
     JK_REQUIRE(tile_rows >= PF_BM && tile_rows % PF_BM == 0, "attention_prefill: tiles of %d rows (a multiple of %d is needed)", tile_rows, PF_BM);
     switch (dh) {
@@ -1267,5 +1287,5 @@ JK_EXPORT int jk_attention_decode_static(const void *q, const void *k_pages, con
     // every partial slot that the merge kernel reads is written by the split kernel of this same call,
     // so what an earlier call left in the array needs no clearing
     return jk_attention_decode(q, k_pages, v_pages, out, need ? scratch : nullptr, rows, nrows, positions, row_req,
-                               block_table, max_blocks, page_size, nh, nkvh, dh, scale, window, splits, 0, nullptr, 0, 0.f, 0, stream);
+                               block_table, max_blocks, page_size, nh, nkvh, dh, scale, window, splits, 0, nullptr, 0, 0.f, 0, nullptr, 0, stream);
 }

@@ -59,11 +59,13 @@ struct AtArgs {
     int *status;
     int ntiles, nh, nkvh, page_size, max_blocks, window;
     float scale_log2;
-    int sink;                 // 1: every softmax has one more key of score 0 that brings no value
+    int sink;                 // 1: every softmax has one more key that brings no value, of score sink_w[h] (null: 0)
     const float *gate;        // float32 [T, gate_ld]: head h's output is multiplied by sigmoid(gate[t, h]); null: none
     int gate_ld;
     float cap_raw;            // a cap on the scores divided by the softmax scale: raw s <- cap tanh(s / cap) (0: none)
     int keep_first;           // with a window: keys at positions below this stay visible when the window has passed them
+    const float *sink_w;
+    int gate_elem;            // 1: the gate has one column per output element, gate[t, h dh + e]
 };
 
 // ---- PTX wrappers (see gemm_tcgen05.cu for the same set) -----------------------------------------
@@ -505,9 +507,11 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             // a half that saw no key has reference -inf, sum 0 and an accumulator of zeros
             const float m_all = fmaxf(m_ref, other.x);
             const float w_mine = ex2(m_ref - m_all), w_other = ex2(other.x - m_all);
-            // a sink adds its term 2^(0 - m_all); a gate multiplies the row's output
-            float inv = 1.f / (l * w_mine + other.y * w_other + (a.sink ? exp2f(-m_all) : 0.f));
-            if (a.gate != nullptr && row < nrows) inv *= 1.f / (1.f + expf(-a.gate[(size_t)(row0 + row) * a.gate_ld + h]));
+            // a sink adds its term 2^(sink - m_all); a gate multiplies the row's output
+            float inv = 1.f / (l * w_mine + other.y * w_other + (a.sink ? exp2f(jk_sink_log2(a.sink_w, h) - m_all) : 0.f));
+            const float *gate = a.gate != nullptr && row < nrows ? a.gate + (size_t)(row0 + row) * a.gate_ld : nullptr;
+            if (gate != nullptr && !a.gate_elem) { inv *= jk_sigmoid(gate[h]); gate = nullptr; }
+            if (gate != nullptr) gate += (size_t)h * DH + half * (DH / 2);         // the gates of this thread's columns
             const float w0 = (half ? w_other : w_mine) * inv, w1 = (half ? w_mine : w_other) * inv;
             // this thread writes columns [half * DH / 2, + DH / 2) of its row
             __nv_bfloat16 *dst = a.out + ((size_t)(row0 + row) * a.nh + h) * DH + half * (DH / 2);
@@ -521,10 +525,22 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
                         unsigned w[4];
+                        float z[8];
+                        if (gate != nullptr) {
+                            const float *g = gate + c * 32 + j;
+                            if ((uintptr_t)g % 16 == 0) {
+                                *reinterpret_cast<float4 *>(z) = *reinterpret_cast<const float4 *>(g);
+                                *reinterpret_cast<float4 *>(z + 4) = *reinterpret_cast<const float4 *>(g + 4);
+                            } else {
+#pragma unroll
+                                for (int q = 0; q < 8; ++q) z[q] = g[q];
+                            }
+                        }
 #pragma unroll
                         for (int q = 0; q < 4; ++q) {
-                            const float lo = __uint_as_float(o0[j + 2 * q]) * w0 + __uint_as_float(o1[j + 2 * q]) * w1;
-                            const float hi = __uint_as_float(o0[j + 2 * q + 1]) * w0 + __uint_as_float(o1[j + 2 * q + 1]) * w1;
+                            float lo = __uint_as_float(o0[j + 2 * q]) * w0 + __uint_as_float(o1[j + 2 * q]) * w1;
+                            float hi = __uint_as_float(o0[j + 2 * q + 1]) * w0 + __uint_as_float(o1[j + 2 * q + 1]) * w1;
+                            if (gate != nullptr) { lo *= jk_sigmoid(z[2 * q]); hi *= jk_sigmoid(z[2 * q + 1]); }
                             const __nv_bfloat162 b = __floats2bfloat162_rn(lo, hi);
                             w[q] = *reinterpret_cast<const unsigned *>(&b);
                         }
@@ -607,9 +623,9 @@ JK_EXPORT int jk_attention_tcgen05(const void *q, const void *k_pages, const voi
                                    int ntiles, int ntok, const int *req_start, const int *req_pos, const int *block_table,
                                    int max_blocks, int num_pages, int page_size, int nh, int nkvh, int dh, float scale,
                                    int window, int *status, int sink, const float *gate, int gate_ld, float cap, int keep_first,
-                                   cudaStream_t stream) {
+                                   const float *sink_w, int gate_elem, cudaStream_t stream) {
     if (ntiles == 0) return JK_OK;
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh, "attention_tcgen05: a gate row of %d holds no %d heads", gate_ld, nh);
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dh : 1), "attention_tcgen05: a gate row of %d holds no %d heads", gate_ld, nh);
     JK_REQUIRE(jk_attention_tcgen05_supports(dh, page_size), "attention_tcgen05: head size %d with pages of %d is not built", dh, page_size);
     JK_REQUIRE(ntiles > 0 && nh > 0 && nkvh > 0 && nh % nkvh == 0 && ntiles <= 65535, "attention_tcgen05: tiles %d heads %d/%d", ntiles, nh, nkvh);
     JK_REQUIRE(max_blocks > 0 && status != nullptr && num_pages > 0, "attention_tcgen05: bad arguments");
@@ -619,7 +635,7 @@ JK_EXPORT int jk_attention_tcgen05(const void *q, const void *k_pages, const voi
     if (int rc = tensor_map(v_pages, (long long)num_pages * nkvh * page_size, dh, page_size, &mv)) return rc;
     AtArgs a{(__nv_bfloat16 *)out, tiles, req_start, req_pos, block_table, status,
              ntiles, nh, nkvh, page_size, max_blocks, window, scale * 1.4426950408889634f, sink, gate, gate_ld,
-             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0};
+             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w, gate_elem};
     JK_REQUIRE(cap >= 0.f && keep_first >= 0 && scale > 0.f, "attention_tcgen05: cap %g, %d kept keys, scale %g", cap, keep_first, scale);
     if (dh == 64) return launch_at<64>(mq, mk, mv, a, stream);
     return launch_at<128>(mq, mk, mv, a, stream);

@@ -3,6 +3,7 @@
 //
 //   norm_add            stream += rmsnorm(sublayer output) * w, and in the same pass the next sublayer's input
 //                       rmsnorm(stream) * w'
+//   norm_pair           two norms of one stream for two sublayers side by side, the first mixed with the row before it
 //   concat_cast         [a | b] side by side as a product's operand; add_bias_rows
 //   latent_qkv          queries split into their plain and rotated parts, the latent vector normed, the shared rotated
 //                       key part turned, both written into the row's place of the paged cache
@@ -150,6 +151,178 @@ JK_EXPORT int jk_norm_add(const float *delta, float *x, const float *w, float ep
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Two norms of one stream, the first with a token shift: with n_t = x[t] / sqrt(mean(x[t]^2) + eps) * w,
+//     h[t]  = T(n_t + (n_(t-1) - n_t) * mu)        (mu null: T(n_t))
+//     h2[t] = T(x[t] / sqrt(mean(x[t]^2) + eps2) * w2)        (h2 null: not made)
+// n_(t-1) of a portion's first row is last[slot] (float32; zeros when a request takes the slot).  A block takes RB rows in a
+// row: a thread keeps its elements of the row before, so a row is read once and the row ahead of the block's first once
+// more.  The kept row of a request with one row in the step moves on here (its elements are one thread's); of the others it
+// does in norm_pair_last, which makes the norm of their last row once more, after this kernel has read the slots.
+// ---------------------------------------------------------------------------------------------------------------
+struct NormPairArgs {
+    const float *x, *w, *mu, *w2;
+    float eps, eps2;
+    float *last;
+    const int *row_req, *req_start, *slot_ids;
+    void *h, *h2;
+    int T, d, RB;
+};
+
+constexpr int NP_THREADS = 512;
+
+__device__ __forceinline__ float sumsq4(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
+__device__ __forceinline__ float4 scale4(float4 v, float s, float4 w) { return make_float4(v.x * s * w.x, v.y * s * w.y, v.z * s * w.z, v.w * s * w.w); }
+__device__ __forceinline__ float4 mix4(float4 n, float4 before, float4 mu) {
+    return make_float4(fmaf(before.x - n.x, mu.x, n.x), fmaf(before.y - n.y, mu.y, n.y), fmaf(before.z - n.z, mu.z, n.z), fmaf(before.w - n.w, mu.w, n.w));
+}
+
+template <typename T, int NV>       // NV vectors of four elements a thread
+__global__ void __launch_bounds__(NP_THREADS) norm_pair_kernel(NormPairArgs a) {
+    pdl_trigger();
+    __shared__ float scratch[33];
+    const int n4 = a.d / 4, t0 = blockIdx.x * a.RB, t1 = min(a.T, t0 + a.RB), step = blockDim.x;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 w[NV], w2[NV], mu[NV], before[NV], next[NV];
+    auto load = [&](float4 (&v)[NV], const float *row) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = threadIdx.x + i * step;
+            v[i] = c < n4 ? reinterpret_cast<const float4 *>(row)[c] : zero;
+        }
+    };
+    load(w, a.w);               // weights are there before any kernel of the step
+    if (a.h2 != nullptr) load(w2, a.w2);
+    if (a.mu != nullptr) load(mu, a.mu);
+    pdl_wait();
+    load(next, a.x + (size_t)t0 * a.d);
+    if (a.mu != nullptr && a.req_start[a.row_req[t0]] != t0) {
+        load(before, a.x + (size_t)(t0 - 1) * a.d);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss += sumsq4(before[i]);
+        const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) before[i] = scale4(before[i], inv, w[i]);
+    }
+    for (int t = t0; t < t1; ++t) {
+        float4 v[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) v[i] = next[i];
+        if (t + 1 < t1) load(next, a.x + (size_t)(t + 1) * a.d);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss += sumsq4(v[i]);
+        const float mean = block_sum(ss, scratch) / (float)a.d;
+        const float inv = 1.f / sqrtf(mean + a.eps), inv2 = 1.f / sqrtf(mean + a.eps2);
+        float *kept = nullptr;
+        bool only_row = false;
+        if (a.mu != nullptr) {
+            const int req = a.row_req[t];
+            if (a.req_start[req] == t) {
+                kept = a.last + (size_t)a.slot_ids[req] * a.d;
+                only_row = a.req_start[req + 1] == t + 1;
+                load(before, kept);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = threadIdx.x + i * step;
+            if (c >= n4) continue;
+            const float4 n = scale4(v[i], inv, w[i]);
+            store4((T *)a.h + (size_t)t * a.d + 4 * c, a.mu != nullptr ? mix4(n, before[i], mu[i]) : n);
+            if (a.h2 != nullptr) store4((T *)a.h2 + (size_t)t * a.d + 4 * c, scale4(v[i], inv2, w2[i]));
+            if (only_row) reinterpret_cast<float4 *>(kept)[c] = n;
+            before[i] = n;
+        }
+    }
+}
+
+// any width and alignment: a block a row, the row before normed once more
+template <typename T>
+__global__ void __launch_bounds__(NP_THREADS) norm_pair_plain_kernel(NormPairArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    const float *x = a.x + (size_t)t * a.d, *xb = nullptr;
+    float *kept = nullptr;
+    bool only_row = false;
+    if (a.mu != nullptr) {
+        const int req = a.row_req[t];
+        if (a.req_start[req] == t) {
+            kept = a.last + (size_t)a.slot_ids[req] * a.d;
+            only_row = a.req_start[req + 1] == t + 1;
+        } else {
+            xb = x - a.d;
+        }
+    }
+    float ss = 0.f, sb = 0.f;
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
+        ss += x[c] * x[c];
+        if (xb != nullptr) sb += xb[c] * xb[c];
+    }
+    const float mean = block_sum(ss, scratch) / (float)a.d;
+    const float inv = 1.f / sqrtf(mean + a.eps), inv2 = 1.f / sqrtf(mean + a.eps2);
+    const float inv_b = xb != nullptr ? 1.f / sqrtf(block_sum(sb, scratch) / (float)a.d + a.eps) : 0.f;
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
+        const float n = x[c] * inv * a.w[c];
+        float out = n;
+        if (a.mu != nullptr) {
+            const float before = xb != nullptr ? xb[c] * inv_b * a.w[c] : kept[c];
+            out = fmaf(before - n, a.mu[c], n);
+            if (only_row) kept[c] = n;
+        }
+        ((T *)a.h)[(size_t)t * a.d + c] = from_f32<T>(out);
+        if (a.h2 != nullptr) ((T *)a.h2)[(size_t)t * a.d + c] = from_f32<T>(x[c] * inv2 * a.w2[c]);
+    }
+}
+
+// the kept rows of requests with several rows in the step
+__global__ void __launch_bounds__(NP_THREADS) norm_pair_last_kernel(NormPairArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int req = blockIdx.x, end = a.req_start[req + 1];
+    if (end - a.req_start[req] <= 1) return;
+    const float *x = a.x + (size_t)(end - 1) * a.d;
+    float *kept = a.last + (size_t)a.slot_ids[req] * a.d;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) ss += x[c] * x[c];
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) kept[c] = x[c] * inv * a.w[c];
+}
+
+JK_EXPORT int jk_norm_pair(const float *x, const float *w, const float *mu, float eps, const float *w2, float eps2, float *last,
+                           const int *row_req, const int *req_start, const int *slot_ids, void *h, void *h2, int dtype, int T, int nreq,
+                           int d, cudaStream_t stream) {
+    if (T == 0) return JK_OK;
+    JK_REQUIRE(x && w && h && T > 0 && d > 0, "norm_pair: rows %d, width %d", T, d);
+    JK_REQUIRE(h2 == nullptr || w2 != nullptr, "norm_pair: a second norm without its weight");
+    JK_REQUIRE(mu == nullptr || (last && row_req && req_start && slot_ids && nreq > 0), "norm_pair: a token shift without its kept rows");
+    const bool vec = d % 4 == 0 && d <= 4 * 4 * NP_THREADS && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)mu % 16 == 0 &&
+                     (uintptr_t)w2 % 16 == 0 && (uintptr_t)last % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)h2 % 16 == 0;
+    // rows a block: one where the rows do not fill the SMs four times over
+    const int RB = std::max(1, std::min(8, T / (4 * 148)));
+    NormPairArgs a{x, w, mu, w2, eps, eps2, last, row_req, req_start, slot_ids, h, h2, T, d, RB};
+    const int n4 = (d + 3) / 4;
+    const int threads = std::max(64, std::min(NP_THREADS, (n4 + 31) / 32 * 32));
+    const dim3 grid((T + RB - 1) / RB);
+#define LAUNCH(TT)                                                                                                   \
+    if (!vec) jk_launch(norm_pair_plain_kernel<TT>, dim3(T), dim3(threads), 0, stream, a);                           \
+    else if (n4 <= threads) jk_launch(norm_pair_kernel<TT, 1>, grid, dim3(threads), 0, stream, a);                   \
+    else if (n4 <= 2 * threads) jk_launch(norm_pair_kernel<TT, 2>, grid, dim3(threads), 0, stream, a);               \
+    else jk_launch(norm_pair_kernel<TT, 4>, grid, dim3(threads), 0, stream, a)
+    BLOCKS_BY_DTYPE(dtype, "norm_pair", LAUNCH);
+#undef LAUNCH
+    JK_CHECK_LAUNCH("norm_pair");
+    if (mu != nullptr && T > nreq) {
+        jk_launch(norm_pair_last_kernel, dim3(nreq), dim3(threads), 0, stream, a);
+        JK_CHECK_LAUNCH("norm_pair_last");
+    }
+    return JK_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // out[t] = T([a[t] | b[t]]): two float32 streams side by side as the operand of one product.
 // ---------------------------------------------------------------------------------------------------------------
 template <typename T>
@@ -195,8 +368,9 @@ JK_EXPORT int jk_add_bias_rows(float *x, const float *bias, int rows, int d, cud
 // Queries and cache rows of the latent attention, from the float32 rows u [T, ld] of one fused product:
 //   u[t, q_off + h (dn + dr) + e]      head h of the query: dn plain elements, then dr that are rotated
 //   u[t, kv_off + e]                   e < R: the latent vector before its norm; then dr elements of the shared key part
-// Rotation of the first `rot_dims` of the dr elements in pairs (2i, 2i+1) by p * freq[i], formed in float32, with cos and
-// sin times `mag`.  Out: q_plain [T, H dn] (the operand of the per-head product that moves the key map to the query),
+// Rotation of the first `rot_dims` of the dr elements in pairs (2i, 2i+1) (rot_half: (i, i + rot_dims / 2)) by p * freq[i],
+// formed in float32, with cos and sin times `mag`.  kv_off < 0: the queries only; a query latent (q_norm_w): the cache row and
+// the query latent only.  Out: q_plain [T, H dn] (the operand of the per-head product that moves the key map to the query),
 // the rotated parts into q_full [T, H, R + dr] behind the R elements which that product fills, and the cache row of the
 // position, [latent * norm weight / rms | rotated key part], into pages [pages, page_size, R + dr].  One block per row.
 // ---------------------------------------------------------------------------------------------------------------
@@ -211,7 +385,22 @@ struct LatentQkvArgs {
     void *q_plain, *q_full, *pages;
     const float *q_norm_w;      // with it: q_plain [T, q_rank] = rmsnorm(u[q_off .. q_off + q_rank)) * q_norm_w, the queries' own latent
     int q_rank;                 // vector (the heads' queries are then a product of it, made by the records that follow)
+    int rot_half;
 };
+
+// element e of a part whose first rot_dims elements are rotated (src: the part's elements)
+__device__ __forceinline__ float latent_rotated(const LatentQkvArgs &a, const float *src, int e, float fpos) {
+    const float val = src[e];
+    if (e >= a.rot_dims) return val;
+    const int half = a.rot_dims >> 1;
+    const bool first = a.rot_half ? e < half : !(e & 1);
+    const int pair = a.rot_half ? (first ? e : e - half) : e >> 1;
+    const float other = src[a.rot_half ? (first ? e + half : e - half) : e ^ 1];
+    float sn, cs;
+    sincosf(fpos * a.freq[pair], &sn, &cs);
+    sn *= a.mag; cs *= a.mag;
+    return first ? fmaf(val, cs, -other * sn) : fmaf(val, cs, other * sn);
+}
 
 template <typename T>
 __global__ void latent_qkv_kernel(LatentQkvArgs a) {
@@ -224,15 +413,18 @@ __global__ void latent_qkv_kernel(LatentQkvArgs a) {
     const float fpos = (float)pos;
     const int dq = a.dn + a.dr, D = a.R + a.dr;
     // the latent vector's norm
-    float ss = 0.f;
-    for (int e = threadIdx.x; e < a.R; e += blockDim.x) {
-        const float v = u[a.kv_off + e];
-        ss += v * v;
+    T *crow = nullptr;
+    if (a.kv_off >= 0) {
+        float ss = 0.f;
+        for (int e = threadIdx.x; e < a.R; e += blockDim.x) {
+            const float v = u[a.kv_off + e];
+            ss += v * v;
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.R + a.eps);
+        const int page = a.block_table[(size_t)a.row_req[t] * a.max_blocks + pos / a.page_size];
+        crow = (T *)a.pages + ((size_t)page * a.page_size + (size_t)(pos % a.page_size)) * D;
+        for (int e = threadIdx.x; e < a.R; e += blockDim.x) crow[e] = from_f32<T>(u[a.kv_off + e] * inv * a.norm_w[e]);
     }
-    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.R + a.eps);
-    const int page = a.block_table[(size_t)a.row_req[t] * a.max_blocks + pos / a.page_size];
-    T *crow = (T *)a.pages + ((size_t)page * a.page_size + (size_t)(pos % a.page_size)) * D;
-    for (int e = threadIdx.x; e < a.R; e += blockDim.x) crow[e] = from_f32<T>(u[a.kv_off + e] * inv * a.norm_w[e]);
     if (a.q_norm_w != nullptr) {
         float sq = 0.f;
         for (int e = threadIdx.x; e < a.q_rank; e += blockDim.x) {
@@ -242,20 +434,13 @@ __global__ void latent_qkv_kernel(LatentQkvArgs a) {
         const float inv_q = 1.f / sqrtf(block_sum(sq, scratch) / (float)a.q_rank + a.eps);
         for (int e = threadIdx.x; e < a.q_rank; e += blockDim.x)
             ((T *)a.q_plain)[(size_t)t * a.q_rank + e] = from_f32<T>(u[a.q_off + e] * inv_q * a.q_norm_w[e]);
+        for (int e = threadIdx.x; e < a.dr; e += blockDim.x) crow[a.R + e] = from_f32<T>(latent_rotated(a, u + a.kv_off + a.R, e, fpos));
         return;
     }
-    // rotated parts: the shared key part (head index H) and every head's query part
-    for (int idx = threadIdx.x; idx < (a.H + 1) * a.dr; idx += blockDim.x) {
+    // rotated parts: every head's query part and (head index H) the shared key part
+    for (int idx = threadIdx.x; idx < (a.kv_off >= 0 ? a.H + 1 : a.H) * a.dr; idx += blockDim.x) {
         const int h = idx / a.dr, e = idx % a.dr;
-        const float *src = h == a.H ? u + a.kv_off + a.R : u + a.q_off + (size_t)h * dq + a.dn;
-        float val = src[e];
-        if (e < a.rot_dims) {
-            float sn, cs;
-            sincosf(fpos * a.freq[e >> 1], &sn, &cs);
-            sn *= a.mag; cs *= a.mag;
-            const float other = src[e ^ 1];
-            val = (e & 1) ? fmaf(val, cs, other * sn) : fmaf(val, cs, -other * sn);
-        }
+        const float val = latent_rotated(a, h == a.H ? u + a.kv_off + a.R : u + a.q_off + (size_t)h * dq + a.dn, e, fpos);
         if (h == a.H) crow[a.R + e] = from_f32<T>(val);
         else ((T *)a.q_full)[((size_t)t * a.H + h) * D + a.R + e] = from_f32<T>(val);
     }
@@ -268,14 +453,15 @@ __global__ void latent_qkv_kernel(LatentQkvArgs a) {
 JK_EXPORT int jk_latent_qkv(const float *u, int ld, int q_off, int kv_off, int H, int dn, int dr, int R, int rot_dims, const float *freq,
                             float mag, const float *norm_w, float eps, const int *positions, const int *row_req, const int *block_table,
                             int max_blocks, int page_size, void *q_plain, void *q_full, void *pages, int dtype, int T,
-                            const float *q_norm_w, int q_rank, cudaStream_t stream) {
+                            const float *q_norm_w, int q_rank, int rot_half, cudaStream_t stream) {
     if (T == 0) return JK_OK;
-    JK_REQUIRE(u && norm_w && positions && row_req && block_table && q_plain && (q_full || q_norm_w) && pages, "latent_qkv: an argument is missing");
-    JK_REQUIRE(q_norm_w == nullptr || (q_rank > 0 && dr == 0), "latent_qkv: queries through a latent of %d elements beside a rotated part of %d", q_rank, dr);
+    JK_REQUIRE(u && positions && row_req && q_plain && (q_full || q_norm_w), "latent_qkv: an argument is missing");
+    JK_REQUIRE(kv_off < 0 || (norm_w && block_table && pages), "latent_qkv: a cache row without its pages");
+    JK_REQUIRE(q_norm_w == nullptr || (q_rank > 0 && kv_off >= 0), "latent_qkv: a query latent of %d elements without the keys' latent", q_rank);
     JK_REQUIRE(H > 0 && dn >= 0 && dr >= 0 && R > 0 && page_size > 0, "latent_qkv: heads %d, sizes %d + %d, latent %d", H, dn, dr, R);
     JK_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0 && (rot_dims == 0 || freq), "latent_qkv: rotation of %d of %d elements", rot_dims, dr);
     LatentQkvArgs a{u, ld, q_off, kv_off, H, dn, dr, R, rot_dims, freq, mag, eps, norm_w, positions, row_req, block_table,
-                    max_blocks, page_size, q_plain, q_full, pages, q_norm_w, q_rank};
+                    max_blocks, page_size, q_plain, q_full, pages, q_norm_w, q_rank, rot_half};
     const int work = q_norm_w ? std::max(q_rank, R) : H * (dn + dr);
     const int threads = work >= 2048 ? 512 : (work >= 512 ? 256 : 128);
 #define LAUNCH(TT) jk_launch(latent_qkv_kernel<TT>, dim3(T), dim3(threads), 0, stream, a)
@@ -503,10 +689,11 @@ __device__ __forceinline__ void tile_product_split(const float *__restrict__ A, 
     }
 }
 
-// out[t, h * out_hs + n] = T(sum_k in[t, h * K + k] * w[h, n, k]) (* sigmoid(gate[t * gate_ld + h * N + n]))
+// out[t, h * out_hs + n] = T(sum_k in[t, h * K + k] * w[h, n, k]) (* sigmoid(gate[t * gate_ld + h * N + n]), or with gate_head
+// sigmoid(gate[t * gate_ld + h]))
 template <typename T>
 __global__ void __launch_bounds__(256) head_linear_kernel(const T *__restrict__ in, const T *__restrict__ w, T *__restrict__ out, int rows, int H,
-                                                          int N, int K, int out_hs, const float *__restrict__ gate, int gate_ld) {
+                                                          int N, int K, int out_hs, const float *__restrict__ gate, int gate_ld, int gate_head) {
     pdl_trigger();
     pdl_wait();
     const int h = blockIdx.z, m0 = blockIdx.x * GT_M, n0 = blockIdx.y * GT_N;
@@ -519,18 +706,18 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const T *__restrict__ 
         const int t = m0 + r, n = n0 + c;
         if (t >= rows || n >= N) continue;
         float v = acc[e];
-        if (gate != nullptr) v *= sigmoid_f(gate[(size_t)t * gate_ld + (size_t)h * N + n]);
+        if (gate != nullptr) v *= sigmoid_f(gate[(size_t)t * gate_ld + (gate_head ? (size_t)h : (size_t)h * N + n)]);
         out[((size_t)t * H + h) * out_hs + n] = from_f32<T>(v);
     }
 }
 
 JK_EXPORT int jk_head_linear(const void *in, const void *w, void *out, int dtype, int rows, int H, int N, int K, int out_hs,
-                             const float *gate, int gate_ld, cudaStream_t stream) {
+                             const float *gate, int gate_ld, int gate_head, cudaStream_t stream) {
     if (rows == 0) return JK_OK;
     JK_REQUIRE(in && w && out && rows > 0 && H > 0 && N > 0 && K > 0 && out_hs >= N, "head_linear: rows %d, heads %d, %d x %d into %d", rows, H, N, K, out_hs);
     JK_REQUIRE(H <= 65535, "head_linear: %d heads exceed one launch", H);
     dim3 grid((rows + GT_M - 1) / GT_M, (N + GT_N - 1) / GT_N, H);
-#define LAUNCH(T) jk_launch(head_linear_kernel<T>, grid, dim3(256), 0, stream, (const T *)in, (const T *)w, (T *)out, rows, H, N, K, out_hs, gate, gate_ld)
+#define LAUNCH(T) jk_launch(head_linear_kernel<T>, grid, dim3(256), 0, stream, (const T *)in, (const T *)w, (T *)out, rows, H, N, K, out_hs, gate, gate_ld, gate_head)
     BLOCKS_BY_DTYPE(dtype, "head_linear", LAUNCH);
 #undef LAUNCH
     JK_CHECK_LAUNCH("head_linear");
@@ -555,7 +742,11 @@ struct LatentAttnArgs {
     int T, H, R, dr, page_size, max_blocks, splits;
     float scale;
     int window;             // the mask as one number (jk_mask_lo): 0 every earlier key, W > 0 the last W keys
+    const float *sink_w;    // [H] or null: one more key per softmax, of this score and without a value
 };
+
+// what a sink adds to the normaliser that belongs to the maximum m
+__device__ __forceinline__ float latent_sink(const float *sink_w, int h, float m) { return sink_w != nullptr ? expf(sink_w[h] - m) : 0.f; }
 
 template <typename T, int NS>
 __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(LatentAttnArgs a) {
@@ -637,7 +828,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(LatentA
         return;
     }
     T *orow = (T *)a.out + ((size_t)t * a.H + h) * a.R;
-    const float inv = 1.f / l;
+    const float inv = 1.f / (l + latent_sink(a.sink_w, h, m));
 #pragma unroll
     for (int i = 0; i < NS; ++i) {
         const int e = lane + 32 * i;
@@ -651,7 +842,8 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(LatentA
 constexpr int LM_THREADS = 128, LM_MAX_SPLITS = 64;
 
 template <typename T>
-__global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const float *__restrict__ part, T *__restrict__ out, int rows_heads, int R, int splits) {
+__global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const float *__restrict__ part, T *__restrict__ out, int H, int R, int splits,
+                                                                  const float *__restrict__ sink_w) {
     pdl_trigger();
     pdl_wait();
     __shared__ float factor[LM_MAX_SPLITS];
@@ -674,7 +866,7 @@ __global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const float *_
             ms[i] = ms[i] > -INFINITY ? expf(ms[i] - M) : 0.f;
             l += ls[i] * ms[i];
         }
-        l = warp_sum(l);
+        l = warp_sum(l) + latent_sink(sink_w, idx % H, M);
         const float inv = 1.f / l;
 #pragma unroll
         for (int i = 0; i < LM_MAX_SPLITS / 32; ++i) {
@@ -717,6 +909,7 @@ struct LatentTcArgs {
     float scale;
     int buffers;        // 2: the tile after the one at work is on its way; 1: where two would leave an SM room for one block only
     int window;         // the mask as one number (jk_mask_lo)
+    const float *sink_w;    // as above
 };
 
 __device__ __forceinline__ void ldmatrix_x2(unsigned &r0, unsigned &r1, const void *smem_row) {
@@ -942,7 +1135,7 @@ __global__ void __launch_bounds__(256) latent_attention_tc_kernel(LatentTcArgs a
             if (nw == 0 && (lane & 3) == 0) { p[a.R] = m; p[a.R + 1] = l; }
         } else {
             __nv_bfloat16 *orow = a.out + ((size_t)t * a.H + h) * a.R;
-            const float inv = 1.f / l;
+            const float inv = 1.f / (l + latent_sink(a.sink_w, h, m));
 #pragma unroll
             for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -967,7 +1160,8 @@ JK_EXPORT long long jk_latent_attention_scratch(int T, int H, int R, int splits)
 // `req_start` [nreq + 1] (may be null): with it, bfloat16 rows go to the tensor-core kernel (latent sizes up to 512).
 JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, float *part, int dtype, const int *positions,
                                   const int *row_req, const int *block_table, int max_blocks, int page_size, int T, int H, int R,
-                                  int dr, float scale, int splits, const int *req_start, int nreq, int window, cudaStream_t stream) {
+                                  int dr, float scale, int splits, const int *req_start, int nreq, int window, const float *sink_w,
+                                  cudaStream_t stream) {
     if (T == 0) return JK_OK;
     JK_REQUIRE(window >= 0, "latent_attention: window %d", window);
     JK_REQUIRE(q && pages && out && positions && row_req && block_table, "latent_attention: an argument is missing");
@@ -992,7 +1186,7 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
         const bool second_block_fits = fixed + 2 * tile > 112 * 1024 && fixed + tile <= 112 * 1024;
         const int buffers = (second_block_fits && (long long)((T + RT - 1) / RT) * grid.y * grid.z > sms) ? 1 : 2;
         LatentTcArgs ta{(const __nv_bfloat16 *)q, (const __nv_bfloat16 *)pages, (__nv_bfloat16 *)out, part, positions, req_start, block_table,
-                        nreq, H, R, dr, page_size, max_blocks, splits, HT, RT, ldk, scale, buffers, window};
+                        nreq, H, R, dr, page_size, max_blocks, splits, HT, RT, ldk, scale, buffers, window, sink_w};
         const size_t smem_tc = fixed + buffers * tile;
         JK_REQUIRE(grid.y <= 65535, "latent_attention: %d heads", H);
 #define LAUNCH_TC(NT_)                                                                                                                       \
@@ -1005,12 +1199,12 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
         JK_CHECK_LAUNCH("latent_attention_tc");
         if (splits > 1) {
             const int n = T * H;
-            jk_launch(latent_merge_kernel<__nv_bfloat16>, dim3(n), dim3(LM_THREADS), 0, stream, (const float *)part, (__nv_bfloat16 *)out, n, R, splits);
+            jk_launch(latent_merge_kernel<__nv_bfloat16>, dim3(n), dim3(LM_THREADS), 0, stream, (const float *)part, (__nv_bfloat16 *)out, H, R, splits, sink_w);
             JK_CHECK_LAUNCH("latent_merge");
         }
         return JK_OK;
     }
-    LatentAttnArgs a{q, pages, out, part, positions, row_req, block_table, T, H, R, dr, page_size, max_blocks, splits, scale, window};
+    LatentAttnArgs a{q, pages, out, part, positions, row_req, block_table, T, H, R, dr, page_size, max_blocks, splits, scale, window, sink_w};
     const size_t smem = ((size_t)LA_WARPS * D + 32 * (size_t)(D + 1)) * sizeof(float);
     JK_REQUIRE(smem <= 220 * 1024, "latent_attention: rows of %d elements do not fit shared memory", D);
     dim3 grid((H + LA_WARPS - 1) / LA_WARPS, T, splits);
@@ -1031,7 +1225,7 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
     JK_CHECK_LAUNCH("latent_attention");
     if (splits > 1) {
         const int n = T * H;
-#define LAUNCH(TT) jk_launch(latent_merge_kernel<TT>, dim3(n), dim3(LM_THREADS), 0, stream, (const float *)part, (TT *)out, n, R, splits)
+#define LAUNCH(TT) jk_launch(latent_merge_kernel<TT>, dim3(n), dim3(LM_THREADS), 0, stream, (const float *)part, (TT *)out, H, R, splits, sink_w)
         BLOCKS_BY_DTYPE(dtype, "latent_merge", LAUNCH);
 #undef LAUNCH
         JK_CHECK_LAUNCH("latent_merge");
@@ -1329,17 +1523,41 @@ JK_EXPORT int jk_selective_scan(const float *x, const float *low, int ld_low, in
 // Options: a bias on the logits (`bias` [E]); a gate per row, sigmoid(gate_w . h), on what the sum is added to (a shared
 // unit's output that waits in delta).
 // ---------------------------------------------------------------------------------------------------------------
+// The largest of n values (the lower index wins a tie) over a warp; every lane gets (value, index).  An index within the
+// list whatever the values are.
+__device__ __forceinline__ int warp_argmax(const float *v, int n, float *value) {
+    const int lane = threadIdx.x & 31;
+    float best = -INFINITY;
+    int at = n;
+    for (int e = lane; e < n; e += 32)
+        if (v[e] > best) { best = v[e]; at = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+    }
+    *value = best;
+    return at < n ? at : n - 1;
+}
+
+// N router outputs, of which the first E stand for experts with matrices and the rest for units that return their input.
+// score_form 0: sigmoid; 1: softmax over all, the chosen ones' scores divided by their sum; 2: softmax over all, as they are.
+// Forms 0 and 1 choose by the logits, form 2 by score + correction; with groups only outputs of the `group_keep` groups
+// (of N / group_count neighbours) whose best choice score is largest can be chosen.
 template <typename T>
-__global__ void route_topk_kernel(const T *__restrict__ h, const float *__restrict__ router, int D, int E, int top, int *__restrict__ ids,
+__global__ void route_topk_kernel(const T *__restrict__ h, const float *__restrict__ router, int D, int N, int E, int top, int *__restrict__ ids,
                                   float *__restrict__ scores, int *__restrict__ counts, int score_form, const float *__restrict__ bias,
-                                  const float *__restrict__ gate_w, float *__restrict__ row_gate) {
+                                  const float *__restrict__ gate_w, float *__restrict__ row_gate, const float *__restrict__ correction,
+                                  int group_count, int group_keep) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float z[];        // [E]
+    extern __shared__ float z[];        // [N] logits, then scores; [N] choice scores; [group_count] best of a group; [group_count] kept
+    float *choice = z + N, *group_best = choice + N, *group_kept = group_best + group_count;
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     const T *row = h + (size_t)t * D;
     const bool vec = D % 8 == 0 && (uintptr_t)row % 16 == 0 && (uintptr_t)router % 16 == 0;
-    for (int e = warp; e < E; e += nwarp) {
+    for (int e = warp; e < N; e += nwarp) {
         const float *w = router + (size_t)e * D;
         float dot = 0.f;
         if (vec) {          // eight elements a lane a pass, the passes' loads independent of one another
@@ -1365,29 +1583,55 @@ __global__ void route_topk_kernel(const T *__restrict__ h, const float *__restri
         if (lane == 0) row_gate[t] = sigmoid_f(dot);
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        // score_form 1: softmax over all experts; the chosen ones' scores divided by their sum
-        float zmax = -INFINITY, total = 1.f, chosen = 0.f;
-        if (score_form == 1) {
-            for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, z[e]);
-            total = 0.f;
-            for (int e = 0; e < E; ++e) total += expf(z[e] - zmax);
-        }
-        for (int k = 0; k < top; ++k) {
-            int best = -1;
-            float bz = -INFINITY;
-            for (int e = 0; e < E; ++e)
-                if (best < 0 || z[e] > bz) { bz = z[e]; best = e; }
-            ids[(size_t)t * top + k] = best;
-            const float sc = score_form == 1 ? expf(bz - zmax) / total : sigmoid_f(bz);
-            scores[(size_t)t * top + k] = sc;
-            chosen += sc;
-            atomicAdd(&counts[best], 1);
-            z[best] = -INFINITY;
-        }
-        if (score_form == 1)
-            for (int k = 0; k < top; ++k) scores[(size_t)t * top + k] /= chosen + 1e-20f;
+    if (warp != 0) return;
+    float zmax = -INFINITY, total = 0.f, unused;
+    if (score_form != 0) {
+        for (int e = lane; e < N; e += 32) zmax = fmaxf(zmax, z[e]);
+        zmax = warp_max(zmax);
+        for (int e = lane; e < N; e += 32) total += expf(z[e] - zmax);
+        total = warp_sum(total);
     }
+    for (int e = lane; e < N; e += 32) {        // a lane's own outputs: no other lane touches them before the barrier
+        const float logit = z[e], s = score_form != 0 ? expf(logit - zmax) / total : sigmoid_f(logit);
+        choice[e] = score_form == 2 ? s + (correction ? correction[e] : 0.f) : logit;
+        z[e] = s;
+    }
+    __syncwarp();
+    if (group_count > 0) {
+        const int size = N / group_count;
+        for (int g = lane; g < group_count; g += 32) {
+            float b = -INFINITY;
+            for (int i = 0; i < size; ++i) b = fmaxf(b, choice[g * size + i]);
+            group_best[g] = b;
+            group_kept[g] = 0.f;
+        }
+        __syncwarp();
+        for (int k = 0; k < group_keep; ++k) {
+            const int g = warp_argmax(group_best, group_count, &unused);
+            __syncwarp();
+            if (lane == 0) { group_best[g] = -INFINITY; group_kept[g] = 1.f; }
+            __syncwarp();
+        }
+        for (int e = lane; e < N; e += 32)
+            if (group_kept[e / size] == 0.f) choice[e] = -INFINITY;
+        __syncwarp();
+    }
+    float chosen = 0.f;
+    for (int k = 0; k < top; ++k) {
+        const int best = warp_argmax(choice, N, &unused);
+        const float sc = z[best];
+        chosen += sc;
+        __syncwarp();
+        if (lane == 0) {
+            ids[(size_t)t * top + k] = best;
+            scores[(size_t)t * top + k] = sc;
+            if (best < E) atomicAdd(&counts[best], 1);
+            choice[best] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    if (score_form == 1)
+        for (int k = lane; k < top; k += 32) scores[(size_t)t * top + k] /= chosen + 1e-20f;
 }
 
 // entry_row[pos], entry_score[pos] for pos in [starts[e], starts[e + 1]); pair_entry[pair] = pos
@@ -1591,43 +1835,103 @@ __global__ void __launch_bounds__(256) expert_rows_kernel(const T *__restrict__ 
     }
 }
 
-// delta[t] (+)= sum over the row's choices, in their order, of y[pair_entry[t * top + k]] (times the choice's score where
-// `entry_score` is given: the form in which the score multiplies a unit's output)
-__global__ void expert_combine_kernel(const float *__restrict__ y, const int *__restrict__ pair_entry, float *__restrict__ delta, int D, int top,
-                                      int add, size_t total, const float *__restrict__ entry_score, const float *__restrict__ row_gate) {
+// v[t] = (what waits in delta, times the row's gate, if `add`) + sum over the row's choices, in their order, of y[pair_entry[t *
+// top + k]], times the choice's score where scores multiply a unit's output (`out_scores`); a choice beyond the E experts is
+// the row's own input h[t].  delta[t] = v, or with a stream x: x[t] += x_scale * v + pend_scale * pend[t] (a product that waits
+// for the stream).  V elements a thread.
+struct CombineArgs {
+    const float *y;
+    const int *pair_entry, *ids;
+    const float *out_scores;        // [T, top] or null
+    int E, D, top, add;
+    float *delta;
+    const float *row_gate;
+    const void *h;
+    float *x;
+    float x_scale;
+    const float *pend;
+    float pend_scale;
+};
+
+template <typename T, int V>
+__global__ void expert_combine_kernel(CombineArgs a, size_t total) {
     pdl_trigger();
     pdl_wait();
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = i / D;
-        const int c = (int)(i % D);
-        float v = add ? (row_gate ? delta[i] * row_gate[t] : delta[i]) : 0.f;
-        for (int k = 0; k < top; ++k) {
-            const int entry = pair_entry[t * top + k];
-            v = entry_score ? fmaf(entry_score[entry], y[(size_t)entry * D + c], v) : v + y[(size_t)entry * D + c];
+    struct __align__(4 * V) Vec { float f[V]; };
+    struct __align__(sizeof(T) * V) VecT { T f[V]; };
+    for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; i < total; i += (size_t)gridDim.x * blockDim.x * V) {
+        const size_t t = i / a.D;
+        const int c = (int)(i % a.D);
+        Vec v;
+        if (a.add) {
+            v = *reinterpret_cast<const Vec *>(a.delta + i);
+            if (a.row_gate) {
+                const float g = a.row_gate[t];
+#pragma unroll
+                for (int e = 0; e < V; ++e) v.f[e] *= g;
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) v.f[e] = 0.f;
         }
-        delta[i] = v;
+        for (int k = 0; k < a.top; ++k) {
+            const size_t pair = t * a.top + k;
+            const float s = a.out_scores ? a.out_scores[pair] : 1.f;
+            if (a.ids[pair] < a.E) {
+                const Vec u = *reinterpret_cast<const Vec *>(a.y + (size_t)a.pair_entry[pair] * a.D + c);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v.f[e] = fmaf(s, u.f[e], v.f[e]);
+            } else {
+                const VecT u = *reinterpret_cast<const VecT *>((const T *)a.h + i);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v.f[e] = fmaf(s, to_f32(u.f[e]), v.f[e]);
+            }
+        }
+        if (a.x != nullptr) {
+            Vec x = *reinterpret_cast<const Vec *>(a.x + i);
+            if (a.pend != nullptr) {
+                const Vec p = *reinterpret_cast<const Vec *>(a.pend + i);
+#pragma unroll
+                for (int e = 0; e < V; ++e) x.f[e] = fmaf(a.pend_scale, p.f[e], x.f[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) x.f[e] = fmaf(a.x_scale, v.f[e], x.f[e]);
+            *reinterpret_cast<Vec *>(a.x + i) = x;
+        } else {
+            *reinterpret_cast<Vec *>(a.delta + i) = v;
+        }
     }
 }
 
-// ints of workspace (`route`) that T rows need: counts [E], starts [E + 1], ids, entry_row, pair_entry [T top] and, as
-// floats, scores and entry_score [T top] and the rows' gates [T]
-JK_EXPORT long long jk_routed_experts_workspace(int T, int E, int top) { return 2LL * E + 1 + 5LL * T * top + T + 16; }
+// ints of workspace (`route`) that T rows need: counts [N], starts [N + 1], ids, entry_row, pair_entry [T top] and, as
+// floats, scores and entry_score [T top] and the rows' gates [T]; N counts the router's outputs
+JK_EXPORT long long jk_routed_experts_workspace(int T, int N, int top) { return 2LL * N + 1 + 5LL * T * top + T + 16; }
 
-// h [T, D] (type T) -> delta [T, D] float32 (add: on top of what is there).  entries [T top, D]-sized buffers: `act`
-// [T top, ff] of the activation type, `y` [T top, D] float32.
+// h [T, D] (type T) -> delta [T, D] float32 (add: on top of what is there), or into the stream x (x += x_scale * sum + pend_scale
+// * pend).  entries [T top, D]-sized buffers: `act` [T top, ff] of the activation type, `y` [T top, D] float32.
+// router [E + identity, D]; group_count 0: no groups.
 JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *w_gate_up, const void *w_down, float *delta, int add,
                                 int dtype, int T, int D, int ff, int E, int top, int actf, int *route, void *act, float *y,
-                                int score_form, float limit, const float *router_bias, const float *gate_w, cudaStream_t stream) {
+                                int score_form, float limit, const float *router_bias, const float *gate_w, int identity, int group_count,
+                                int group_keep, const float *correction, float *x, float x_scale, const float *pend, float pend_scale,
+                                cudaStream_t stream) {
     if (T == 0) return JK_OK;
+    const int N = E + identity;
     JK_REQUIRE(gate_w == nullptr || add, "routed_experts: a gate on a shared unit's output that is not there");
     JK_REQUIRE(h && router && w_gate_up && w_down && delta && route && act && y, "routed_experts: an argument is missing");
-    JK_REQUIRE(D > 0 && ff > 0 && E > 0 && top > 0 && top <= E, "routed_experts: %d experts, %d a row, sizes %d and %d", E, top, D, ff);
-    JK_REQUIRE((size_t)E * sizeof(float) <= 40 * 1024, "routed_experts: %d experts exceed the router's shared memory", E);
+    JK_REQUIRE(D > 0 && ff > 0 && E > 0 && identity >= 0 && top > 0 && top <= N, "routed_experts: %d + %d experts, %d a row, sizes %d and %d", E, identity, top, D, ff);
+    JK_REQUIRE(score_form >= 0 && score_form <= 2 && (identity == 0 || score_form != 0), "routed_experts: scores of form %d with %d identities", score_form, identity);
+    JK_REQUIRE(correction == nullptr || score_form == 2, "routed_experts: a correction of the choice with scores of form %d", score_form);
+    JK_REQUIRE(group_count == 0 || (group_count > 0 && N % group_count == 0 && group_keep > 0 && group_keep <= group_count && group_keep * (N / group_count) >= top),
+               "routed_experts: %d of %d groups of %d outputs for %d choices", group_keep, group_count, N, top);
+    JK_REQUIRE(pend == nullptr || x != nullptr, "routed_experts: a product that waits needs the stream");
+    const size_t route_smem = (2 * (size_t)N + 2 * (size_t)group_count) * sizeof(float);
+    JK_REQUIRE(route_smem <= 40 * 1024, "routed_experts: %d experts exceed the router's shared memory", N);
     const int pairs = T * top;
     int *counts = route, *starts = counts + E, *ids = starts + E + 1, *entry_row = ids + pairs, *pair_entry = entry_row + pairs;
     float *scores = (float *)(pair_entry + pairs), *entry_score = scores + pairs, *row_gate = gate_w ? entry_score + pairs : nullptr;
     if (cudaMemsetAsync(counts, 0, sizeof(int) * (size_t)E, stream) != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "routed_experts: clearing the counts failed");
-#define LAUNCH(TT) jk_launch(route_topk_kernel<TT>, dim3(T), dim3(128), (size_t)E * sizeof(float), stream, (const TT *)h, router, D, E, top, ids, scores, counts, score_form, router_bias, gate_w, row_gate)
+#define LAUNCH(TT) jk_launch(route_topk_kernel<TT>, dim3(T), dim3(128), route_smem, stream, (const TT *)h, router, D, N, E, top, ids, scores, counts, score_form, router_bias, gate_w, row_gate, correction, group_count, group_keep)
     BLOCKS_BY_DTYPE(dtype, "route_topk", LAUNCH);
 #undef LAUNCH
     JK_CHECK_LAUNCH("route_topk");
@@ -1635,8 +1939,8 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
               starts, entry_row, entry_score, pair_entry);
     JK_CHECK_LAUNCH("route_sort");
     // few rows: the experts' matrices stream past their entries (rows of 16-byte multiples); else tiles
-    // score_form 1: the score multiplies the unit's output (in the sum of a row's choices), not its input
-    const float *in_score = score_form == 1 ? nullptr : entry_score, *out_score = score_form == 1 ? entry_score : nullptr;
+    // score_form 1 and 2: the score multiplies the unit's output (in the sum of a row's choices), not its input
+    const float *in_score = score_form != 0 ? nullptr : entry_score, *out_scores = score_form != 0 ? scores : nullptr;
     const int per16 = dtype == JK_F32 ? 4 : 8;
     const bool stream_rows = pairs <= 64 && D % per16 == 0 && ff % per16 == 0 && (uintptr_t)w_gate_up % 16 == 0 && (uintptr_t)w_down % 16 == 0 &&
                              (size_t)ER_ROWS * std::max(D, ff) * 4 <= 160 * 1024;
@@ -1664,8 +1968,15 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
     JK_CHECK_LAUNCH("expert products");
     }
     const size_t total = (size_t)T * D;
-    jk_launch(expert_combine_kernel, dim3((int)std::min<size_t>((total + 255) / 256, 148 * 16)), dim3(256), 0, stream, (const float *)y,
-              (const int *)pair_entry, delta, D, top, add, total, out_score, (const float *)row_gate);
+    const CombineArgs ca{y, pair_entry, ids, out_scores, E, D, top, add, delta, row_gate, h, x, x_scale, pend, pend_scale};
+    const bool four = D % 4 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)delta % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)pend % 16 == 0;
+    const size_t threads = total / (four ? 4 : 1);
+    const int combine_blocks = (int)std::min<size_t>((threads + 255) / 256, 148 * 16);
+#define LAUNCH(TT)                                                                                            \
+    if (four) jk_launch(expert_combine_kernel<TT, 4>, dim3(combine_blocks), dim3(256), 0, stream, ca, total); \
+    else jk_launch(expert_combine_kernel<TT, 1>, dim3(combine_blocks), dim3(256), 0, stream, ca, total)
+    BLOCKS_BY_DTYPE(dtype, "expert_combine", LAUNCH);
+#undef LAUNCH
     JK_CHECK_LAUNCH("expert_combine");
     return JK_OK;
 }

@@ -140,6 +140,11 @@ static inline int jk_epilogue_gate(int epilogue) {
     return act == GATE_GELU_TANH ? GATE_GELU_TANH : (act == GATE_RELU ? GATE_RELU : GATE_SILU);
 }
 
+// ---- an output gate and a sink of a softmax attention ---------------------------------------------
+__device__ __forceinline__ float jk_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// The score of head h's sink in units of log2 (`sink_w` null: every head's is 0).
+__device__ __forceinline__ float jk_sink_log2(const float *sink_w, int h) { return sink_w != nullptr ? sink_w[h] * 1.4426950408889634f : 0.f; }
+
 // ---- the mask of a causal attention as one number --------------------------------------------
 // The first key that a query at position `pos` sees: `window` 0: every earlier key; W > 0: a sliding window of W keys
 // (pos - W + 1, not below 0); -C < 0: the keys of the query's own chunk of C positions, counted from position 0 of the

@@ -212,8 +212,9 @@ JK_EXPORT int jk_glu(const float *gu, void *out, int dtype, int ntok, int di, in
 //             (a cos(p f_i) - b sin(p f_i), b cos(p f_i) + a sin(p f_i)),  the angle p * f_i formed in float32
 // The projections before a portion's first row come from the request's tail: the last taps - 1 projected rows of its
 // sequence, tail[slot, s, c], s = taps - 2 the newest.  One block per row.  Queries go to q_out [T, nq]; keys (after
-// everything) and values (after the convolution) into their pages at the row's position.  `conv_tail_kernel` then
-// moves the tails forward; it runs after this kernel has read them.
+// everything) and values (after the convolution) into their pages at the row's position.  The tail of a request with one
+// row in the step moves forward here (a channel is one thread's); `conv_tail_kernel` does it for the others, after this
+// kernel has read them.
 // ---------------------------------------------------------------------------------------------------------------
 struct ConvQkvArgs {
     const float *u;             // [T, ld]
@@ -231,6 +232,7 @@ struct ConvQkvArgs {
                                 // 2: BEFORE the rotation every head of q and k passes an RMS norm whose weight (norm_q, norm_k:
                                 // [dk], shared by the heads) multiplies it; the whole-projection norm is then off
     const float *bias;          // [ld] or null: added to the projection's columns as they are read (no convolution then)
+    const float *temp;          // [heads] or null: head h's queries are multiplied by temp[h] after everything else
     const int *positions, *row_req, *req_start, *slot_ids, *block_table;
     int max_blocks, page_size;
     void *q_out, *k_pages, *v_pages;
@@ -247,7 +249,8 @@ __global__ void conv_qkv_kernel(ConvQkvArgs a) {
     const int req = a.row_req[t];
     const int back = t - a.req_start[req];          // rows of this portion before this one
     const int pos = a.positions[t];
-    const float *tail = a.tail ? a.tail + (size_t)a.slot_ids[req] * (a.taps - 1) * C : nullptr;
+    float *tail = a.tail ? a.tail + (size_t)a.slot_ids[req] * (a.taps - 1) * C : nullptr;
+    const bool only_row = tail != nullptr && a.req_start[req + 1] - a.req_start[req] == 1;
     float ssq = 0.f, ssk = 0.f;
     for (int c = threadIdx.x; c < C; c += blockDim.x) {
         int col;
@@ -266,6 +269,10 @@ __global__ void conv_qkv_kernel(ConvQkvArgs a) {
                 if (d <= back) uv = a.u[(size_t)(t - d) * a.ld + col];
                 else uv = tail[(size_t)(a.taps - 1 + back - d) * C + c];
                 acc = fmaf(w[j], uv, acc);
+            }
+            if (only_row) {
+                for (int s = 0; s + 2 < a.taps; ++s) tail[(size_t)s * C + c] = tail[(size_t)(s + 1) * C + c];
+                if (a.taps > 1) tail[(size_t)(a.taps - 2) * C + c] = a.u[(size_t)t * a.ld + col];
             }
         }
         y[c] = acc;
@@ -319,7 +326,7 @@ __global__ void conv_qkv_kernel(ConvQkvArgs a) {
                         val = first ? val * cs - other * sn : val * cs + other * sn;
                     }
                     const int c = hh * a.dk + e;
-                    if (c < a.nq) q_out[c] = from_f32<T>(val);
+                    if (c < a.nq) q_out[c] = from_f32<T>(a.temp ? val * a.temp[hh] : val);
                     else ((T *)a.k_pages)[(k_row + (size_t)((c - a.nq) / a.dk) * a.page_size) * a.dk + e] = from_f32<T>(val);
                 }
                 continue;
@@ -351,7 +358,7 @@ __global__ void conv_qkv_kernel(ConvQkvArgs a) {
                     val = first ? val * cs - other * sn : val * cs + other * sn;
                 }
                 const int c = hh * a.dk + e;
-                if (c < a.nq) q_out[c] = from_f32<T>(val * inv);
+                if (c < a.nq) q_out[c] = from_f32<T>(a.temp ? val * inv * a.temp[hh] : val * inv);
                 else ((T *)a.k_pages)[(k_row + (size_t)((c - a.nq) / a.dk) * a.page_size) * a.dk + e] = from_f32<T>(val * inv);
             }
         }
@@ -374,7 +381,7 @@ __global__ void conv_qkv_kernel(ConvQkvArgs a) {
                 const float other = y[a.rot_half ? (first ? c + half : c - half) : (first ? c + 1 : c - 1)];
                 val = first ? fmaf(val, cs, -other * sn) : fmaf(val, cs, other * sn);
             }
-            if (is_q) q_out[cc] = from_f32<T>(val);
+            if (is_q) q_out[cc] = from_f32<T>(a.temp ? val * a.temp[head] : val);
             else ((T *)a.k_pages)[(k_row + (size_t)head * a.page_size) * a.dk + e] = from_f32<T>(val);
         } else {
             const int cc = c - a.nq - a.nk;
@@ -395,6 +402,7 @@ __global__ void conv_tail_kernel(ConvQkvArgs a, int nreq) {
     if (idx >= nreq * C) return;
     const int req = idx / C, c = idx % C;
     const int first = a.req_start[req], n = a.req_start[req + 1] - first;
+    if (n == 1) return;         // moved forward by the row's own block
     int col;
     if (c < a.nq) col = a.q_off + c;
     else if (c < a.nq + a.nk) col = a.k_off + c - a.nq;
@@ -412,10 +420,11 @@ JK_EXPORT int jk_conv_qkv(const float *u, int ld, int q_off, int k_off, int v_of
                           const float *norm_q, const float *norm_k, float eps, const float *freq, int rot_dims, float *tail,
                           const int *positions, const int *row_req, const int *req_start, const int *slot_ids,
                           const int *block_table, int max_blocks, int page_size, void *q_out, void *k_pages, void *v_pages,
-                          int dtype, int T, int nreq, int rot_half, float rot_mag, int head_norm, const float *bias, cudaStream_t stream) {
+                          int dtype, int T, int nreq, int rot_half, float rot_mag, int head_norm, const float *bias, const float *temp,
+                          cudaStream_t stream) {
     if (T == 0) return JK_OK;
     ConvQkvArgs a;
-    a.bias = bias;
+    a.bias = bias; a.temp = temp;
     a.u = u; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
     a.nq = heads * dk; a.nk = has_kv ? kv_heads * dk : 0; a.nv = has_kv ? kv_heads * dv : 0;
     a.conv_q = conv_q; a.conv_k = conv_k; a.conv_v = conv_v; a.norm_q = norm_q; a.norm_k = norm_k; a.freq = freq; a.tail = tail;
@@ -445,7 +454,7 @@ JK_EXPORT int jk_conv_qkv(const float *u, int ld, int q_off, int k_off, int v_of
         JK_FAIL(JK_UNSUPPORTED, "conv_qkv: dtype %d", dtype);
     }
     JK_CHECK_LAUNCH("conv_qkv");
-    if (conv && taps > 1) {
+    if (conv && taps > 1 && T > nreq) {
         const int total = nreq * C;
         jk_launch(conv_tail_kernel, dim3((total + 127) / 128), dim3(128), 0, stream, a, nreq);
         JK_CHECK_LAUNCH("conv_tail");

@@ -271,18 +271,19 @@ int run_attention(Run &r, const RunnerOp &op) {
         // one warp per (row, head): float32, and every shape the tensor-core kernels are not built for
         RUN(attention, g_fns.attention_rows(q, op.k_pages, op.v_pages, o, r.env.dtype, r.st.positions, r.st.row_req, table,
                                             r.env.max_blocks, page, T, nh, nkvh, dh, op.softmax_scale, op.window, dv, op.sink, gate, op.ld,
-                                            op.cap, op.keep_first, r.stream));
+                                            op.cap, op.keep_first, op.sink_w, op.gated == 2, r.stream));
         return JK_OK;
     }
     if (n_tiles > 0) {
         if (tc)
             RUN(attention_tcgen05, g_fns.attention_tcgen05(q, op.k_pages, op.v_pages, o, tiles, n_tiles, T, r.st.req_start, r.st.req_pos,
                                                            table, r.env.max_blocks, op.num_pages, page, nh, nkvh, dh, op.softmax_scale,
-                                                           op.window, r.env.status, op.sink, gate, op.ld, op.cap, op.keep_first, r.stream));
+                                                           op.window, r.env.status, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w,
+                                                           op.gated == 2, r.stream));
         else
             RUN(attention, g_fns.attention_prefill(q, op.k_pages, op.v_pages, o, tiles, n_tiles, jk::TILE_ROWS, r.st.req_start,
                                                    r.st.req_pos, table, r.env.max_blocks, page, nh, nkvh, dh, op.softmax_scale,
-                                                   op.window, op.sink, gate, op.ld, op.cap, op.keep_first, r.stream));
+                                                   op.window, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w, op.gated == 2, r.stream));
     }
     if (n_short > 0) {
         const int context = r.st.context > 0 ? r.st.context : op.max_positions;
@@ -293,7 +294,7 @@ int run_attention(Run &r, const RunnerOp &op) {
             if (int rc = r.slot(SLOT_DECODE, need, &scratch, "the split-key attention's partial results")) return rc;
         RUN(attention, g_fns.attention_decode(q, op.k_pages, op.v_pages, o, (float *)scratch, short_rows, n_short, r.st.positions,
                                               r.st.row_req, table, r.env.max_blocks, page, nh, nkvh, dh, op.softmax_scale, op.window,
-                                              splits, op.sink, gate, op.ld, op.cap, op.keep_first, r.stream));
+                                              splits, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w, op.gated == 2, r.stream));
     }
     return JK_OK;
 }
@@ -395,6 +396,8 @@ int run_linear(Run &r, const RunnerOp &op) {
     if (rows == 0) return JK_OK;
     void *in, *out;
     if (int rc = r.slot(op.in_slot, (long long)r.elem() * rows * op.k * (op.in_part + 1), &in, "a product's activations")) return rc;
+    if (op.out_slot == SLOT_DELTA && !op.wanted_rows)       // a product that waits there goes into the stream first
+        if (int rc = flush_pending(r, rows, op.n)) return rc;
     in = (char *)in + (size_t)r.elem() * rows * op.k * op.in_part;
     if (op.ld > 0) {        // a column range of wider rows
         JK_REQUIRE(op.out_off >= 0 && op.out_off + op.n <= op.ld, "runner: a product writes columns %d .. %d of rows of %d", op.out_off, op.out_off + op.n, op.ld);
@@ -490,8 +493,8 @@ int run_conv_qkv(Run &r, const RunnerOp &op) {
     RUN(mixers, g_fns.conv_qkv((const float *)u, op.ld, op.q_off, op.k_off, op.v_off, op.heads, op.kv_heads, op.head_dim, dv, op.has_kv,
                                op.conv_q, op.conv_k, op.conv_v, op.taps, op.norm_q, op.norm_k, op.eps, op.freq, op.rot_dims, op.state,
                                r.st.positions, r.st.row_req, r.st.req_start, r.st.slot_ids, table, r.env.max_blocks, r.env.page_size, q,
-                               op.k_pages, op.v_pages, r.env.dtype, T, r.st.nreq, op.rot_half, op.rot_mag, op.head_norm, op.bias, r.stream));
-    if (op.taps > 1) ++g_launches;      // the tails' kernel
+                               op.k_pages, op.v_pages, r.env.dtype, T, r.st.nreq, op.rot_half, op.rot_mag, op.head_norm, op.bias, op.temp, r.stream));
+    if (op.taps > 1 && T > r.st.nreq) ++g_launches;      // the tails' kernel
     return JK_OK;
 }
 
@@ -562,6 +565,7 @@ int run_latent_qkv(Run &r, const RunnerOp &op) {
     const int T = r.st.ntok, H = op.heads, D = op.rank + op.rot_width;
     void *u, *q_full, *q_plain;
     if (int rc = r.slot(op.in_slot, 4LL * T * op.ld, &u, "the query and latent projection")) return rc;
+    const bool queries_only = op.k_off < 0;
     if (op.q_rank > 0) {        // the queries' own latent vector, normed; the heads' queries are made by the records that follow
         q_full = nullptr;
         if (int rc = r.slot(op.out2_slot, (long long)r.elem() * T * op.q_rank, &q_plain, "the queries' latent vector")) return rc;
@@ -569,11 +573,11 @@ int run_latent_qkv(Run &r, const RunnerOp &op) {
         if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * H * D, &q_full, "the queries")) return rc;
         if (int rc = r.slot(op.out2_slot, (long long)r.elem() * T * H * op.head_dim, &q_plain, "the queries' plain parts")) return rc;
     }
-    const int *table = r.st.block_tables[op.cache_group];
-    JK_REQUIRE(table != nullptr, "runner: a latent attention writes the cache of group %d, whose block table the step lacks", op.cache_group);
+    const int *table = queries_only ? nullptr : r.st.block_tables[op.cache_group];
+    JK_REQUIRE(table != nullptr || queries_only, "runner: a latent attention writes the cache of group %d, whose block table the step lacks", op.cache_group);
     RUN(blocks, g_fns.latent_qkv((const float *)u, op.ld, op.q_off, op.k_off, H, op.head_dim, op.rot_width, op.rank, op.rot_dims, op.freq,
                                  op.rot_mag, op.norm_k, op.eps, r.st.positions, r.st.row_req, table, r.env.max_blocks, r.env.page_size,
-                                 q_plain, q_full, op.k_pages, r.env.dtype, T, op.q_rank > 0 ? op.norm_q : nullptr, op.q_rank, r.stream));
+                                 q_plain, q_full, op.k_pages, r.env.dtype, T, op.q_rank > 0 ? op.norm_q : nullptr, op.q_rank, op.rot_half, r.stream));
     return JK_OK;
 }
 
@@ -589,7 +593,7 @@ int run_head_linear(Run &r, const RunnerOp &op) {
         if (int rc = r.slot(SLOT_TMP, 4LL * T * op.ld, &u, "the projection that holds the gate")) return rc;
         gate = (const float *)u + op.g_off;
     }
-    RUN(blocks, g_fns.head_linear(in, op.w, out, r.env.dtype, T, op.heads, op.n, op.k, op.out_hs, gate, op.ld, r.stream));
+    RUN(blocks, g_fns.head_linear(in, op.w, out, r.env.dtype, T, op.heads, op.n, op.k, op.out_hs, gate, op.ld, op.gated == 2, r.stream));
     return JK_OK;
 }
 
@@ -617,7 +621,7 @@ int run_latent_attention(Run &r, const RunnerOp &op) {
     if (splits > 1)
         if (int rc = r.slot(SLOT_DECODE, 4 * g_fns.latent_attention_scratch(T, H, op.rank, splits), &part, "the ranges of a latent attention")) return rc;
     RUN(blocks, g_fns.latent_attention(q, op.k_pages, o, (float *)part, r.env.dtype, r.st.positions, r.st.row_req, table, r.env.max_blocks,
-                                       r.env.page_size, T, H, op.rank, op.rot_width, op.softmax_scale, splits, r.st.req_start, r.st.nreq, op.window, r.stream));
+                                       r.env.page_size, T, H, op.rank, op.rot_width, op.softmax_scale, splits, r.st.req_start, r.st.nreq, op.window, op.sink_w, r.stream));
     if (splits > 1) ++g_launches;
     return JK_OK;
 }
@@ -660,17 +664,36 @@ int run_experts(Run &r, const RunnerOp &op) {
     void *h, *delta, *route, *act, *y;
     if (int rc = r.slot(op.in_slot, (long long)r.elem() * T * op.n, &h, "the experts' input")) return rc;
     if (int rc = r.slot(SLOT_DELTA, 4LL * T * op.n, &delta, "the experts' output")) return rc;
-    if (int rc = r.slot(SLOT_ROUTE, 4 * g_fns.routed_experts_workspace(T, op.experts, op.top), &route, "the rows' choice of experts")) return rc;
+    const bool adds = op.into_stream == 2;      // the sum goes into the stream by its own kernel, with a product that waits
+    if (int rc = r.slot(SLOT_ROUTE, 4 * g_fns.routed_experts_workspace(T, op.experts + op.identity, op.top), &route, "the rows' choice of experts")) return rc;
     if (int rc = r.slot(SLOT_ACT, (long long)r.elem() * T * op.top * op.ff, &act, "the experts' inner activations")) return rc;
     if (int rc = r.slot(SLOT_TMP, 4LL * T * op.top * op.n, &y, "the experts' results")) return rc;
-    JK_REQUIRE(!r.pending, "runner: routed experts while another product waits to be added");
+    JK_REQUIRE(!r.pending || (adds && !op.add), "runner: routed experts while another product waits to be added");
     RUN(blocks, g_fns.routed_experts(h, op.vec, op.w, op.w3, (float *)delta, op.add, r.env.dtype, T, op.n, op.ff, op.experts, op.top, op.act,
-                                     (int *)route, act, (float *)y, op.score_form, op.limit, op.router_bias, op.gate_w, r.stream));
+                                     (int *)route, act, (float *)y, op.score_form, op.limit, op.router_bias, op.gate_w, op.identity, op.group_count, op.group_keep,
+                                   op.correction, adds ? r.x() : nullptr, op.scale, r.pending ? (const float *)delta : nullptr, r.pending_scale, r.stream));
     g_launches += g_fns.routed_experts_launches() - 1;
-    if (op.into_stream) {       // a block without a norm on the sublayer's output: the next norm adds it
+    if (adds) {
+        r.pending = false;
+    } else if (op.into_stream) {       // a block without a norm on the sublayer's output: the next norm adds it
         r.pending = true;
         r.pending_scale = 1.f;
     }
+    return JK_OK;
+}
+
+int run_norm_pair(Run &r, const RunnerOp &op) {
+    JK_REQUIRE(g_fns.norm_pair != nullptr, "runner: a pair of norms needs the blocks module, which was not bound");
+    const int T = r.st.ntok;
+    void *h, *h2 = nullptr;
+    if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &h, "the first norm of a pair")) return rc;
+    if (op.out2_slot >= 0)
+        if (int rc = r.slot(op.out2_slot, (long long)r.elem() * T * op.n, &h2, "the second norm of a pair")) return rc;
+    JK_REQUIRE(op.bias == nullptr || (op.state != nullptr && r.st.slot_ids != nullptr), "runner: a token shift without its state slots");
+    if (int rc = flush_pending(r, T, op.n)) return rc;
+    RUN(blocks, g_fns.norm_pair(r.x(), op.vec, op.bias, op.eps, op.vec2, op.eps2, op.state, r.st.row_req, r.st.req_start, r.st.slot_ids, h, h2,
+                                r.env.dtype, T, r.st.nreq, op.n, r.stream));
+    if (op.bias != nullptr && T > r.st.nreq) ++g_launches;      // the kept rows of requests with several rows
     return JK_OK;
 }
 
@@ -845,6 +868,10 @@ JK_EXPORT int jk_runner_run(const RunnerEnv *envp, const RunnerOp *ops, int firs
                 rc = run_add_rows(r, op);
                 break;
             case OP_DELTA_RULE: rc = run_delta_rule(r, op); break;
+            case OP_NORM_PAIR:
+                hidden = op.n;
+                rc = run_norm_pair(r, op);
+                break;
             default:
                 JK_FAIL(JK_BAD_ARGUMENT, "runner_run: record %d has kind %d", i, op.kind);
         }
@@ -943,10 +970,14 @@ JK_EXPORT int jk_runner_slot_bytes(const RunnerEnv *env, const RunnerOp *ops, in
                 break;
             case OP_EXPERTS:
                 need(op.in_slot, e * rows * op.n); need(SLOT_DELTA, 4 * rows * op.n);
-                need(SLOT_ROUTE, 4 * (2LL * op.experts + 1 + 5 * rows * op.top + rows + 16));
+                need(SLOT_ROUTE, 4 * (2LL * (op.experts + op.identity) + 1 + 5 * rows * op.top + rows + 16));
                 need(SLOT_ACT, e * rows * op.top * op.ff); need(SLOT_TMP, 4 * rows * op.top * op.n);
                 break;
             case OP_SOFTCAP: need(op.in_slot, 4 * rows * op.n); break;
+            case OP_NORM_PAIR:
+                need(SLOT_X, 4 * rows * op.n); need(op.out_slot, e * rows * op.n);
+                if (op.out2_slot >= 0) need(op.out2_slot, e * rows * op.n);
+                break;
             case OP_ADD_ROWS: need(SLOT_X, 4 * rows * op.n); break;
             case OP_DELTA_RULE: {
                 const long long width = (long long)op.heads * op.v_head_dim;

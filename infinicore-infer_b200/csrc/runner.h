@@ -30,16 +30,17 @@ typedef int (*GemmTcgen05Fn)(const void *, const void *, void *, int, int, int, 
 typedef int (*GemmTcgen05QkvFn)(const void *, const void *, int, int, void *, void *, void *, const float *, const float *,
                                 const int *, const int *, const int *, int, int, int, int, int, int *, int, cudaStream_t);
 typedef int (*AttentionRowsFn)(const void *, const void *, const void *, void *, int, const int *, const int *, const int *, int,
-                               int, int, int, int, int, float, int, int, int, const float *, int, float, int, cudaStream_t);
+                               int, int, int, int, int, float, int, int, int, const float *, int, float, int, const float *, int,
+                               cudaStream_t);
 typedef int (*AttentionDecodeFn)(const void *, const void *, const void *, void *, float *, const int *, int, const int *,
                                  const int *, const int *, int, int, int, int, int, float, int, int, int, const float *, int, float, int,
-                                 cudaStream_t);
+                                 const float *, int, cudaStream_t);
 typedef int (*AttentionPrefillFn)(const void *, const void *, const void *, void *, const int *, int, int, const int *,
                                   const int *, const int *, int, int, int, int, int, float, int, int, const float *, int, float, int,
-                                  cudaStream_t);
+                                  const float *, int, cudaStream_t);
 typedef int (*AttentionTcgen05Fn)(const void *, const void *, const void *, void *, const int *, int, int, const int *,
                                   const int *, const int *, int, int, int, int, int, int, float, int, int *, int, const float *, int,
-                                  float, int, cudaStream_t);
+                                  float, int, const float *, int, cudaStream_t);
 typedef int (*SupportsFn)(int, int, int);
 typedef int (*LinearSmallPartsFn)(const void *, long long, const int *, int, const void *, void *, int, int, int, int, int, cudaStream_t);
 typedef int (*Supports1Fn)(int);
@@ -55,7 +56,7 @@ typedef int (*CastRowsFn)(const float *, void *, int, long long, cudaStream_t);
 typedef int (*GluFn)(const float *, void *, int, int, int, int, float, cudaStream_t);
 typedef int (*ConvQkvFn)(const float *, int, int, int, int, int, int, int, int, int, const float *, const float *, const float *, int,
                          const float *, const float *, float, const float *, int, float *, const int *, const int *, const int *,
-                         const int *, const int *, int, int, void *, void *, void *, int, int, int, int, float, int, const float *, cudaStream_t);
+                         const int *, const int *, int, int, void *, void *, void *, int, int, int, int, float, int, const float *, const float *, cudaStream_t);
 typedef int (*LinearScanFn)(const float *, int, int, int, int, int, int, int, int, float, const float *, const void *, int, const float *,
                             int, int, float, float *, const int *, const int *, int, int, float *, const int *, int, const int *, int,
                             const int *, int, float *, long long, int, const float *, int, int, cudaStream_t);
@@ -68,10 +69,10 @@ typedef int (*NormAddFn)(const float *, float *, const float *, float, const flo
 typedef int (*ConcatCastFn)(const float *, const float *, void *, int, int, int, cudaStream_t);
 typedef int (*AddBiasRowsFn)(float *, const float *, int, int, cudaStream_t);
 typedef int (*LatentQkvFn)(const float *, int, int, int, int, int, int, int, int, const float *, float, const float *, float, const int *,
-                           const int *, const int *, int, int, void *, void *, void *, int, int, const float *, int, cudaStream_t);
-typedef int (*HeadLinearFn)(const void *, const void *, void *, int, int, int, int, int, int, const float *, int, cudaStream_t);
+                           const int *, const int *, int, int, void *, void *, void *, int, int, const float *, int, int, cudaStream_t);
+typedef int (*HeadLinearFn)(const void *, const void *, void *, int, int, int, int, int, int, const float *, int, int, cudaStream_t);
 typedef int (*LatentAttentionFn)(const void *, const void *, void *, float *, int, const int *, const int *, const int *, int, int, int,
-                                 int, int, int, float, int, const int *, int, int, cudaStream_t);
+                                 int, int, int, float, int, const int *, int, int, const float *, cudaStream_t);
 typedef long long (*LatentScratchFn)(int, int, int, int);
 typedef int (*CausalConvFn)(const float *, int, int, int, const float *, const float *, int, int, float *, const int *, const int *,
                             const int *, float *, void *, int, int, int, cudaStream_t);
@@ -79,12 +80,15 @@ typedef int (*SelectiveScanFn)(const float *, const float *, int, int, int, int,
                                const float *, const float *, float *, const int *, const int *, int, void *, int, float *, int, int,
                                cudaStream_t);
 typedef int (*RoutedExpertsFn)(const void *, const float *, const void *, const void *, float *, int, int, int, int, int, int, int, int,
-                               int *, void *, float *, int, float, const float *, const float *, cudaStream_t);
+                               int *, void *, float *, int, float, const float *, const float *, int, int, int, const float *, float *, float,
+                               const float *, float, cudaStream_t);
 typedef long long (*RoutedWorkspaceFn)(int, int, int);
 typedef int (*CountFn)();
 typedef int (*SoftcapFn)(float *, float, long long, cudaStream_t);
 typedef int (*AddRowsFn)(float *, const void *, int, int, const int *, int, int, int, cudaStream_t);
 // csrc/mixers.cu
+typedef int (*NormPairFn)(const float *, const float *, const float *, float, const float *, float, float *, const int *, const int *, const int *,
+                          void *, void *, int, int, int, int, cudaStream_t);
 typedef int (*DeltaRuleFn)(const float *, int, int, int, int, const float *, int, int, int, const float *, const float *, int, int, int, int,
                            float, float, float *, const int *, const int *, int, float *, float *, int, cudaStream_t);
 typedef long long (*DeltaScratchFn)(int, int, int, int);
@@ -157,6 +161,7 @@ struct RunnerFns {
     AddRowsFn add_rows;
     DeltaRuleFn delta_rule;
     DeltaScratchFn delta_rule_scratch;
+    NormPairFn norm_pair;           // csrc/blocks.cu, bound with that module
 };
 
 // ---- records ---------------------------------------------------------------------------------------------------
@@ -179,6 +184,7 @@ enum RunnerSlot {
     SLOT_X0,            // float32 [T, hidden]: the embedding's output, for a model that feeds it in again later
     SLOT_ROUTE,         // int32 and float32: which experts each row chose, and the rows of each expert
     SLOT_SHIFT,         // activations [parts, T, width]: a row mixed with the row before it, once per projection that reads one
+    SLOT_H2,            // activations [T, hidden]: a second norm's output, for a sublayer beside the one that reads SLOT_H
     RUNNER_SLOTS
 };
 
@@ -222,6 +228,9 @@ enum RunnerOpKind {
     OP_DELTA_RULE,      // in: float32 rows [q | k | v] (after their convolutions), SLOT_TMP: the projection's rows with the write
                         // strength's and the decay's logits and the gate; S <- g S, S += k (beta (v - S^T k))^T, o = S^T q per head over
                         // each request's rows and its state slot; out = rmsnorm(o) * vec * act(gate)
+    OP_NORM_PAIR,       // two norms of the same stream: out2 = rmsnorm(stream) * vec2 (out2_slot < 0: not made), and out = h_t + (h_(t-1) -
+                        // h_t) * bias with h = rmsnorm(stream) * vec; the row before a portion's first row is kept in state [slots, n]
+                        // (bias null: out = h, no state)
 };
 
 enum RunnerAct { RUNNER_ACT_NONE = 0, RUNNER_ACT_SILU = 1, RUNNER_ACT_GELU_TANH = 2, RUNNER_ACT_SIGMOID = 3, RUNNER_ACT_RELU = 4,
@@ -314,6 +323,16 @@ struct RunnerOp {
     const float *bonus;         // LINEAR_ATTENTION: [heads, head_dim]; a row then reads the state before its own decay, its own key
                                 // times the bonus: o = (S + diag(bonus) k v^T)^T q, then S = diag(a) S + k v^T
     // ATTENTION: cap > 0 caps the scores, s <- cap tanh(s / cap).
+    // ---- what learned sinks, gates of another shape, identity experts in groups and pairs of norms add ------------------------------
+    int group_count, group_keep;        // EXPERTS: > 0: only experts of the best group_keep of group_count groups of neighbours are chosen
+    int identity;               // EXPERTS: so many router outputs behind the experts' stand for units that return their input
+    const float *sink_w;        // ATTENTION, LATENT_ATTENTION: [heads] the sinks' scores (null: 0; LATENT_ATTENTION: no sink)
+    const float *temp;          // CONV_QKV: [heads] head h's queries are multiplied by temp[h] after everything else, or null
+    const float *correction;    // EXPERTS: [experts + identity] added to the scores for the choice only, or null
+    // ATTENTION: gated 2: a gate per output element, sigmoid(SLOT_TMP[t, g_off + h dv + e]).  HEAD_LINEAR: gated 2: a gate per head.
+    // LATENT_QKV: k_off < 0 makes the heads' queries only, from rows [heads, head_dim + rot_width] at q_off (no cache row, no latent).
+    // EXPERTS: score_form 2: softmax over all router outputs, the chosen scores as they are, multiplying the units' outputs;
+    // into_stream 2: stream += scale * sum, by the sum's own kernel, which also adds a product that waits in SLOT_DELTA.
 };
 
 // What does not change from step to step and is no part's business.

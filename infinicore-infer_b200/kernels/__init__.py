@@ -441,7 +441,8 @@ def _sm_count(device) -> int:
 
 
 def _gate_args(gate: Optional[torch.Tensor], rows: int, nh: int):
-    """(pointer, leading dimension) of a float32 gate ``[rows, >= nh]`` (a view of wider rows is fine), or nulls."""
+    """(pointer, leading dimension) of a float32 gate ``[rows, >= nh]`` (a view of wider rows is fine), or nulls.  ``nh`` counts
+    columns: heads, or heads x value size for a gate per element."""
     if gate is None:
         return _ptr(None), _c_int(0)
     _need(gate, "gate", torch.float32, contiguous=False)
@@ -453,12 +454,14 @@ def _gate_args(gate: Optional[torch.Tensor], rows: int, nh: int):
 def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
                    positions: torch.Tensor, row_req: torch.Tensor, block_table: torch.Tensor, ntok: int,
                    nh: int, scale: float, window: int = 0, sink: bool = False,
-                   gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
+                   gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0,
+                   sink_w: Optional[torch.Tensor] = None, gate_elem: bool = False) -> torch.Tensor:
     """Causal attention of ``ntok`` query rows over the paged cache, one warp per (row, head).  Values may have
     another size than keys (``v_pages [..., dv]``, ``out [ntok, nh, dv]``); ``sink`` adds a key of score 0 without a
     value; ``gate`` (float32 ``[ntok, >= nh]``, a view of wider rows is fine) multiplies head h's output by
     sigmoid(gate[t, h]); ``cap`` > 0 caps the scores by cap tanh(s / cap); keys at positions below ``keep_first`` stay
-    visible when the window has passed them."""
+    visible when the window has passed them; ``sink_w`` (float32 [nh]): the sinks' scores instead of 0; ``gate_elem``: the gate
+    has a column for every output element (``[ntok, >= nh dv]``)."""
     _need(q, "q"); _need(k_pages, "k_pages"); _need(v_pages, "v_pages"); _need(out, "out")
     _need(positions, "positions", torch.int32); _need(row_req, "row_req", torch.int32)
     _need(block_table, "block_table", torch.int32)
@@ -471,7 +474,7 @@ def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     gate_ld = 0
     if gate is not None:
         _need(gate, "gate", torch.float32, contiguous=False)
-        if gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] < ntok or gate.shape[1] < nh:
+        if gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] < ntok or gate.shape[1] < nh * (dv if gate_elem else 1):
             raise KernelError("attention: gate must be [rows, heads] with unit stride along heads")
         gate_ld = gate.stride(0)
     lib = _build.load("attention")
@@ -479,7 +482,7 @@ def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _c_int(dtype_code(q.dtype)), _ptr(positions),
         _ptr(row_req), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(page_size), _c_int(ntok),
         _c_int(nh), _c_int(nkvh), _c_int(dh), _c_float(scale), _c_int(window or 0), _c_int(dv), _c_int(1 if sink else 0),
-        _ptr(gate), _c_int(gate_ld), _c_float(cap), _c_int(keep_first), _stream()))
+        _ptr(gate), _c_int(gate_ld), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
     return out
 
 
@@ -487,7 +490,8 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
                      rows: Optional[torch.Tensor], nrows: int, positions: torch.Tensor, row_req: torch.Tensor,
                      block_table: torch.Tensor, nh: int, scale: float, window: int, splits: int,
                      scratch: Optional[torch.Tensor] = None, sink: bool = False, gate: Optional[torch.Tensor] = None,
-                     cap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
+                     cap: float = 0.0, keep_first: int = 0, sink_w: Optional[torch.Tensor] = None,
+                     gate_elem: bool = False) -> torch.Tensor:
     """bfloat16 attention of rows that bring few queries per request (decoded tokens, short portions):
     the key range of every (row, key/value head) is cut into ``splits`` blocks whose partial results
     a second kernel merges.  ``rows`` lists the rows to work on (None: rows 0..nrows-1).  ``cap`` and ``keep_first``
@@ -512,7 +516,7 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(scratch if need else None), _ptr(rows), _c_int(nrows),
         _ptr(positions), _ptr(row_req), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(page_size),
         _c_int(nh), _c_int(nkvh), _c_int(dh), _c_float(scale), _c_int(window or 0), _c_int(splits), _c_int(1 if sink else 0),
-        *_gate_args(gate, 0, nh), _c_float(cap), _c_int(keep_first), _stream()))
+        *_gate_args(gate, 0, nh * (dh if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
     if need and splits > 1:
         global launch_count
         launch_count += 1          # the merge kernel
@@ -529,7 +533,8 @@ TILE_ROWS = _host.attention_tile_rows()      # rows of a query tile in the tile 
 def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
                       tiles: torch.Tensor, ntiles: int, req_start: torch.Tensor, req_pos: torch.Tensor,
                       block_table: torch.Tensor, nh: int, scale: float, window: int = 0, sink: bool = False,
-                      gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
+                      gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0,
+                      sink_w: Optional[torch.Tensor] = None, gate_elem: bool = False) -> torch.Tensor:
     """bfloat16 tensor-core (mma.sync) attention of requests that bring many rows: ``tiles[i] = (batch
     entry, first row)`` names TILE_ROWS-row tiles of query rows.  ``cap`` and ``keep_first`` as ``attention_rows`` takes
     them: the tiles of keys that hold kept keys and lie before the window's come first."""
@@ -544,8 +549,8 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
     _check("attention", lib.jk_attention_prefill(
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(tiles), _c_int(ntiles), _c_int(TILE_ROWS), _ptr(req_start),
         _ptr(req_pos), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(page_size), _c_int(nh), _c_int(nkvh),
-        _c_int(dh), _c_float(scale), _c_int(window or 0), _c_int(1 if sink else 0), *_gate_args(gate, 0, nh), _c_float(cap),
-        _c_int(keep_first), _stream()))
+        _c_int(dh), _c_float(scale), _c_int(window or 0), _c_int(1 if sink else 0), *_gate_args(gate, 0, nh * (dh if gate_elem else 1)), _c_float(cap),
+        _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
     return out
 
 
@@ -558,7 +563,8 @@ def attention_tcgen05_supports(dh: int, page_size: int) -> bool:
 def attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
                       tiles: torch.Tensor, ntiles: int, ntok: int, req_start: torch.Tensor, req_pos: torch.Tensor,
                       block_table: torch.Tensor, nh: int, scale: float, window: int = 0, sink: bool = False,
-                      gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
+                      gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0,
+                      sink_w: Optional[torch.Tensor] = None, gate_elem: bool = False) -> torch.Tensor:
     """The same attention of TILE_ROWS-row query tiles on the tcgen05 tensor cores (TMA operands, both
     products with accumulators in tensor memory); head sizes 64 and 128, pages that divide 128."""
     for name, t in (("q", q), ("k_pages", k_pages), ("v_pages", v_pages), ("out", out)):
@@ -573,7 +579,7 @@ def attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(tiles), _c_int(ntiles), _c_int(ntok), _ptr(req_start),
         _ptr(req_pos), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(num_pages), _c_int(page_size), _c_int(nh),
         _c_int(nkvh), _c_int(dh), _c_float(scale), _c_int(window or 0), _ptr(gemm_status(q.device)), _c_int(1 if sink else 0),
-        *_gate_args(gate, ntok, nh), _c_float(cap), _c_int(keep_first), _stream()))
+        *_gate_args(gate, ntok, nh * (dh if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
     return out
 
 
@@ -617,12 +623,13 @@ def glu(gate_up: torch.Tensor, out: torch.Tensor, act: int, limit: float = 0.0) 
 def conv_qkv(u: torch.Tensor, offsets, heads: int, kv_heads: int, dk: int, dv: int, has_kv: bool, convs, taps: int, norms, eps: float,
              freq: Optional[torch.Tensor], rot_dims: int, tail: Optional[torch.Tensor], positions, row_req, req_start, slot_ids,
              block_table: Optional[torch.Tensor], page_size: int, q_out: torch.Tensor, k_pages=None, v_pages=None,
-             rot_half: bool = False, rot_mag: float = 1.0, head_norm=False, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+             rot_half: bool = False, rot_mag: float = 1.0, head_norm=False, bias: Optional[torch.Tensor] = None,
+             temp: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Short convolution, whole-projection RMS norm, pair rotation and cache write of fused float32 projections ``u``
     ``[T, ld]`` (columns ``offsets = (q, k, v)``); ``convs = (q, k, v)`` taps ``[channels, taps]`` or None each;
     ``norms = (q, k)`` weights or None each; ``tail [slots, taps - 1, channels]`` is read and moved forward.  ``rot_half``
     pairs element i of a head with element i + rot_dims / 2, ``rot_mag`` multiplies cos and sin, ``head_norm`` divides each
-    head of q and k by its root mean square after the rotation."""
+    head of q and k by its root mean square after the rotation, ``temp`` [heads] multiplies the heads' queries."""
     _need(u, "u", torch.float32); _need(q_out, "q_out")
     T, nreq = u.shape[0], req_start.numel() - 1
     lib = _build.load("mixers")
@@ -632,7 +639,7 @@ def conv_qkv(u: torch.Tensor, offsets, heads: int, kv_heads: int, dk: int, dv: i
         _ptr(norms[0]), _ptr(norms[1]), _c_float(eps), _ptr(freq), _c_int(rot_dims), _ptr(tail), _ptr(positions), _ptr(row_req),
         _ptr(req_start), _ptr(slot_ids), _ptr(block_table), _c_int(block_table.shape[1] if block_table is not None else 0),
         _c_int(page_size), _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _c_int(dtype_code(q_out.dtype)), _c_int(T), _c_int(nreq),
-        _c_int(1 if rot_half else 0), _c_float(rot_mag), _c_int(int(head_norm)), _ptr(bias), _stream()))
+        _c_int(1 if rot_half else 0), _c_float(rot_mag), _c_int(int(head_norm)), _ptr(bias), _ptr(temp), _stream()))
     return q_out
 
 
@@ -716,36 +723,53 @@ def norm_add(delta: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: fl
     return x
 
 
+def norm_pair(x: torch.Tensor, weight: torch.Tensor, eps: float, h: torch.Tensor, mu: Optional[torch.Tensor] = None,
+              last: Optional[torch.Tensor] = None, row_req=None, req_start=None, slot_ids=None, weight2: Optional[torch.Tensor] = None,
+              eps2: float = 0.0, h2: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """h[t] = n_t + (n_(t-1) - n_t) * mu with n = rmsnorm(x) * weight (``mu`` None: n itself), the row before a request's first
+    row being ``last[slot]``, which then moves on to the n of its last row; h2 = rmsnorm(x) * weight2 if given."""
+    _need(x, "x", torch.float32); _need(weight, "weight", torch.float32); _need(h, "h")
+    lib = _build.load("blocks")
+    _check("blocks", lib.jk_norm_pair(_ptr(x), _ptr(weight), _ptr(mu), _c_float(eps), _ptr(weight2), _c_float(eps2), _ptr(last), _ptr(row_req),
+                                      _ptr(req_start), _ptr(slot_ids), _ptr(h), _ptr(h2), _c_int(dtype_code(h.dtype)), _c_int(x.shape[0]),
+                                      _c_int(req_start.numel() - 1 if req_start is not None else 1), _c_int(x.shape[1]), _stream()))
+    return h
+
+
 def latent_qkv(u: torch.Tensor, q_off: int, kv_off: int, heads: int, dn: int, dr: int, latent: int, rot_dims: int,
                freq: Optional[torch.Tensor], magnitude: float, norm_weight: torch.Tensor, eps: float, positions, row_req, block_table,
-               page_size: int, q_plain: torch.Tensor, q_full: Optional[torch.Tensor], pages: torch.Tensor, q_norm: Optional[torch.Tensor] = None,
-               q_rank: int = 0) -> None:
-    """Queries and cache rows of a latent attention from the fused float32 projection ``u`` (see csrc/blocks.cu)."""
-    _need(u, "u", torch.float32); _need(q_plain, "q_plain"); _need(pages, "pages")
+               page_size: int, q_plain: torch.Tensor, q_full: Optional[torch.Tensor], pages: Optional[torch.Tensor],
+               q_norm: Optional[torch.Tensor] = None, q_rank: int = 0, rot_half: bool = False) -> None:
+    """Queries and cache rows of a latent attention from the fused float32 projection ``u`` (see csrc/blocks.cu); ``kv_off`` < 0: the
+    queries only (``norm_weight``, ``block_table`` and ``pages`` may be None)."""
+    _need(u, "u", torch.float32); _need(q_plain, "q_plain")
     lib = _build.load("blocks")
     _check("blocks", lib.jk_latent_qkv(
         _ptr(u), _c_int(u.shape[1]), _c_int(q_off), _c_int(kv_off), _c_int(heads), _c_int(dn), _c_int(dr), _c_int(latent), _c_int(rot_dims),
         _ptr(freq), _c_float(magnitude), _ptr(norm_weight), _c_float(eps), _ptr(positions), _ptr(row_req), _ptr(block_table),
-        _c_int(block_table.shape[1]), _c_int(page_size), _ptr(q_plain), _ptr(q_full), _ptr(pages), _c_int(dtype_code(pages.dtype)),
-        _c_int(u.shape[0]), _ptr(q_norm), _c_int(q_rank), _stream()))
+        _c_int(block_table.shape[1] if block_table is not None else 1), _c_int(page_size), _ptr(q_plain), _ptr(q_full), _ptr(pages),
+        _c_int(dtype_code(q_plain.dtype)), _c_int(u.shape[0]), _ptr(q_norm), _c_int(q_rank), _c_int(1 if rot_half else 0), _stream()))
 
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_head_stride: int, gate: Optional[torch.Tensor] = None,
-                gate_ld: int = 0) -> torch.Tensor:
-    """out[t, h, :n] = x[t, h] w[h]^T for ``w [heads, n, k]``, times sigmoid(gate[t, h n + j]) if given (float32 rows ``gate_ld`` apart)."""
+                gate_ld: int = 0, gate_head: bool = False) -> torch.Tensor:
+    """out[t, h, :n] = x[t, h] w[h]^T for ``w [heads, n, k]``, times sigmoid(gate[t, h n + j]) if given (float32 rows ``gate_ld``
+    apart; ``gate_head``: sigmoid(gate[t, h]))."""
     _need(x, "x"); _need(w, "w"); _need(out, "out")
     H, n, k = w.shape
     lib = _build.load("blocks")
     _check("blocks", lib.jk_head_linear(_ptr(x), _ptr(w), _ptr(out), _c_int(dtype_code(x.dtype)), _c_int(x.shape[0]), _c_int(H), _c_int(n),
-                                        _c_int(k), _c_int(out_head_stride), _ptr(gate), _c_int(gate_ld), _stream()))
+                                        _c_int(k), _c_int(out_head_stride), _ptr(gate), _c_int(gate_ld), _c_int(1 if gate_head else 0), _stream()))
     return out
 
 
 def latent_attention(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, positions, row_req, block_table, heads: int, latent: int,
-                     dr: int, scale: float, splits: int = 1, req_start: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
+                     dr: int, scale: float, splits: int = 1, req_start: Optional[torch.Tensor] = None, window: int = 0,
+                     sink_w: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of ``heads`` query heads ``[T, heads, latent + dr]`` over the paged rows ``[pages, page, latent + dr]``;
     out ``[T, heads, latent]``.  ``splits`` > 1 cuts each row's keys into that many ranges.  With ``req_start`` (int32, the first
-    row of each request and the row count) bfloat16 rows run on the tensor cores."""
+    row of each request and the row count) bfloat16 rows run on the tensor cores.  ``sink_w`` (float32 [heads]): one more key per
+    softmax, of that score and without a value."""
     _need(q, "q"); _need(pages, "pages"); _need(out, "out")
     T = q.shape[0]
     lib = _build.load("blocks")
@@ -755,7 +779,7 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, po
     _check("blocks", lib.jk_latent_attention(_ptr(q), _ptr(pages), _ptr(out), _ptr(part), _c_int(dtype_code(q.dtype)), _ptr(positions),
                                              _ptr(row_req), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(pages.shape[-2]),
                                              _c_int(T), _c_int(heads), _c_int(latent), _c_int(dr), _c_float(scale), _c_int(splits), _ptr(req_start),
-                                             _c_int(req_start.numel() - 1 if req_start is not None else 0), _c_int(window), _stream()))
+                                             _c_int(req_start.numel() - 1 if req_start is not None else 0), _c_int(window), _ptr(sink_w), _stream()))
     return out
 
 
@@ -788,21 +812,26 @@ def selective_scan(x: torch.Tensor, low: torch.Tensor, dt_rank: int, states: int
 
 def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, delta: torch.Tensor, add: bool,
                    experts: int, top: int, act: int, score_form: int = 0, limit: float = 0.0, router_bias: Optional[torch.Tensor] = None,
-                   gate_w: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   gate_w: Optional[torch.Tensor] = None, identity: int = 0, groups=(0, 0), correction: Optional[torch.Tensor] = None,
+                   x: Optional[torch.Tensor] = None, x_scale: float = 1.0, pending: Optional[torch.Tensor] = None,
+                   pending_scale: float = 1.0) -> torch.Tensor:
     """delta (+)= sum over each row's ``top`` experts of largest sigmoid(router h) of expert(score * h); ``w_gate_up``
-    ``[experts * 2 ff, d]`` (an expert's gate rows, then its up rows), ``w_down [experts * d, ff]``."""
+    ``[experts * 2 ff, d]`` (an expert's gate rows, then its up rows), ``w_down [experts * d, ff]``.  ``identity``, ``groups``,
+    ``correction``: see csrc/blocks.cu (score_form 2).  With ``x`` (float32 ``[T, d]``) the sum goes there instead:
+    x += x_scale * sum + pending_scale * pending."""
     _need(h, "h"); _need(router, "router", torch.float32); _need(delta, "delta", torch.float32)
     T, d = h.shape
     ff = w_down.shape[1]
     lib = _build.load("blocks")
     lib.jk_routed_experts_workspace.restype = ctypes.c_longlong
-    route = torch.empty(int(lib.jk_routed_experts_workspace(_c_int(T), _c_int(experts), _c_int(top))), dtype=torch.int32, device=h.device)
+    route = torch.empty(int(lib.jk_routed_experts_workspace(_c_int(T), _c_int(experts + identity), _c_int(top))), dtype=torch.int32, device=h.device)
     act_buf = torch.empty(T * top, ff, dtype=h.dtype, device=h.device)
     y = torch.empty(T * top, d, dtype=torch.float32, device=h.device)
     _check("blocks", lib.jk_routed_experts(_ptr(h), _ptr(router), _ptr(w_gate_up), _ptr(w_down), _ptr(delta), _c_int(1 if add else 0),
                                            _c_int(dtype_code(h.dtype)), _c_int(T), _c_int(d), _c_int(ff), _c_int(experts), _c_int(top),
                                            _c_int(act), _ptr(route), _ptr(act_buf), _ptr(y), _c_int(score_form), _c_float(limit), _ptr(router_bias), _ptr(gate_w),
-                                           _stream()))
+                                           _c_int(identity), _c_int(groups[0]), _c_int(groups[1]), _ptr(correction), _ptr(x), _c_float(x_scale),
+                                           _ptr(pending), _c_float(pending_scale), _stream()))
     return delta
 
 

@@ -1,7 +1,9 @@
 """Softmax attention with a short convolution on its projections, whole-projection norms, partial rotation, a window,
 a sink and a gate per head, over the paged cache; optionally on another layer's keys and values.  Further options of the
 same records: a rotation that pairs the halves of a head's leading elements, with stretched frequencies; a division of
-every head of q and k by its root mean square after the rotation; capped scores; first positions that the window keeps.
+every head of q and k by its root mean square after the rotation; capped scores; first positions that the window keeps;
+a gate per output element instead of one per head; a factor per head on the scores (applied to the queries, in float32,
+before they are rounded); learned scores of the sinks.
 
 One fused product [q | k | v | gate] (or [q | gate] for a layer that borrows its keys) of the mixer's input in float32;
 ``conv_qkv`` (csrc/mixers.cu) convolves every channel over time (the taps - 1 projected rows before a portion come from
@@ -53,8 +55,12 @@ class ConvAttention:
                 decls[name + spec.norm_suffix] = TensorDecl((spec.head_dim,), VECTOR, init="ones")
             if spec.bias:
                 decls[name + spec.bias_suffix] = TensorDecl((n,), VECTOR, init="zeros")
-        if spec.head_gate:
-            decls[spec.gate_name] = TensorDecl((spec.num_heads, d))
+        if spec.head_gate or spec.element_gate:
+            decls[spec.gate_name] = TensorDecl((spec.num_heads * (spec.v_head_dim if spec.element_gate else 1), d))
+        if spec.temp_name:
+            decls[spec.temp_name] = TensorDecl((spec.num_heads,), VECTOR, init="ones")
+        if spec.sink_name:
+            decls[spec.sink_name] = TensorDecl((spec.num_heads,), VECTOR, init="taps")
         decls[spec.o_name] = TensorDecl((d, spec.num_heads * spec.v_head_dim))
         return decls
 
@@ -75,7 +81,8 @@ class ConvAttention:
     def __init__(self, spec, weights, prefix: str, runtime):
         self.spec, self.runtime = spec, runtime
         proj = self._projections(spec)
-        names = [n for n, _, _ in proj] + ([spec.gate_name] if spec.head_gate else [])
+        gated = spec.head_gate or spec.element_gate
+        names = [n for n, _, _ in proj] + ([spec.gate_name] if gated else [])
         self.w_in = weights.get_rows([prefix + n for n in names], MATRIX)
         self.w_o = weights.get(prefix + spec.o_name, MATRIX)
         get = lambda name: weights.get(prefix + name, VECTOR)
@@ -84,8 +91,14 @@ class ConvAttention:
             raise ValueError("an attention has a sliding window or chunks, not both")
         if spec.head_norm == "before_rotation" and spec.qk_norm:
             raise ValueError("a norm over the whole projection and one per head ahead of the rotation are not built together")
-        if spec.bias and (spec.conv_taps or spec.head_gate):
-            raise ValueError("biases beside a convolution or a gate per head are not built")
+        if spec.bias and (spec.conv_taps or gated):
+            raise ValueError("biases beside a convolution or a gate are not built")
+        if spec.head_gate and spec.element_gate:
+            raise ValueError("an attention has a gate per head or one per element, not both")
+        if spec.sink_name and not spec.sink:
+            raise ValueError("learned sinks of an attention without a sink")
+        self.temp = get(spec.temp_name) if spec.temp_name else None
+        self.sink_w = get(spec.sink_name) if spec.sink_name else None
         per_head = spec.qk_norm or spec.head_norm == "before_rotation"
         self.norms = {n: get(n + spec.norm_suffix) for n, _, normed in proj if normed} if per_head else {}
         self.bias = torch.cat([get(n + spec.bias_suffix) for n, _, _ in proj]).contiguous() if spec.bias else None
@@ -132,17 +145,17 @@ class ConvAttention:
                    conv_q=self.conv.get(s.q_name), conv_k=self.conv.get(s.k_name), conv_v=self.conv.get(s.v_name),
                    norm_q=self.norms.get(s.q_name), norm_k=self.norms.get(s.k_name), eps=s.qk_norm_eps, freq=self.freq, rot_dims=rot,
                    state=state, cache_group=view.group_index, k_pages=view.k_pages, v_pages=view.v_pages,
-                   num_pages=view.k_pages.shape[0], writes_cache=writes_cache, rot_mag=self.rot_mag, bias=self.bias,
+                   num_pages=view.k_pages.shape[0], writes_cache=writes_cache, rot_mag=self.rot_mag, bias=self.bias, temp=self.temp,
                    head_norm=2 if s.head_norm == "before_rotation" else int(bool(s.head_norm)),
                    rot_half=self.freq is not None and s.position.layout == "halves"),
             record("attention", "q", "o", heads=s.num_heads, kv_heads=s.num_kv_heads, head_dim=s.head_dim, v_head_dim=s.v_head_dim,
                    window=-int(s.chunk) if s.chunk else (s.window or 0), softmax_scale=s.softmax_scale, cache_group=view.group_index, list_short=short,
                    list_tiles=tiles, max_positions=program.max_blocks * program.page_size, k_pages=view.k_pages,
-                   v_pages=view.v_pages, num_pages=view.k_pages.shape[0], sink=s.sink, gated=s.head_gate, ld=ld, g_off=g_off,
+                   v_pages=view.v_pages, num_pages=view.k_pages.shape[0], sink=s.sink, sink_w=self.sink_w, gated=2 if s.element_gate else int(s.head_gate), ld=ld, g_off=g_off,
                    cap=float(s.score_cap or 0.0), keep_first=s.keep_first if s.window else 0),
             record("linear", "o", "delta", n=s.hidden_size, k=s.num_heads * s.v_head_dim, w=self.w_o) if into_stream is None else
             record("residual", "o", "x", n=s.hidden_size, k=s.num_heads * s.v_head_dim, w=self.w_o, scale=float(into_stream)),
-        ], keep=(self.w_in, self.w_o, self.conv, self.norms, self.freq, state, view.k_pages, view.v_pages, self.bias))
+        ], keep=(self.w_in, self.w_o, self.conv, self.norms, self.freq, state, view.k_pages, view.v_pages, self.bias, self.temp, self.sink_w))
 
     def forward(self, h: torch.Tensor, ctx, view, writes_cache: bool = True, state_view=None) -> torch.Tensor:
         """The part alone: its own records over ``h``; float32 ``[T, hidden]``."""

@@ -34,12 +34,18 @@ class GLU:
     def weight_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.w_gate_up, self.w_down))
 
-    def plan_delta(self, program) -> None:
-        """Two records: gate | up with the activation (h -> act), down into the delta slot."""
+    def plan(self, program, residual_scale: float = 1.0, in_slot: str = "h") -> None:
+        """The feed-forward in a block that adds its output to the stream itself."""
+        self.plan_delta(program, in_slot=in_slot, into_stream=residual_scale)
+
+    def plan_delta(self, program, in_slot: str = "h", into_stream=None) -> None:
+        """Two records: gate | up with the activation (h -> act), down into the delta slot (``into_stream`` s: added into the
+        stream times s)."""
         s = self.spec
         program.emit_records([
-            record("gate_up", "h", "act", n=s.intermediate_size, k=s.hidden_size, w=self.w_gate_up, act=ACT[s.act], limit=float(s.limit)),
-            record("linear", "act", "delta", n=s.hidden_size, k=s.intermediate_size, w=self.w_down),
+            record("gate_up", in_slot, "act", n=s.intermediate_size, k=s.hidden_size, w=self.w_gate_up, act=ACT[s.act], limit=float(s.limit)),
+            record("linear", "act", "delta", n=s.hidden_size, k=s.intermediate_size, w=self.w_down) if into_stream is None else
+            record("residual", "act", "x", n=s.hidden_size, k=s.intermediate_size, w=self.w_down, scale=float(into_stream)),
         ], keep=(self.w_gate_up, self.w_down))
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:

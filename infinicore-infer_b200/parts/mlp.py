@@ -31,15 +31,15 @@ class MLP:
     def weight_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down))
 
-    def plan(self, program, residual_scale: float = 1.0) -> None:
+    def plan(self, program, residual_scale: float = 1.0, in_slot: str = "h") -> None:
         """The feed-forward in a block that adds its output to the stream itself."""
-        self.plan_delta(program, into_stream=residual_scale)
+        self.plan_delta(program, into_stream=residual_scale, in_slot=in_slot)
 
-    def plan_delta(self, program, into_stream=None) -> None:
+    def plan_delta(self, program, into_stream=None, in_slot: str = "h") -> None:
         """Three records: up (h -> float32 rows), the activation (-> act), down into the delta slot or the stream."""
         s = self.spec
         program.emit_records([
-            record("linear", "h", "tmp", n=s.intermediate_size, k=s.hidden_size, w=self.w_up),
+            record("linear", in_slot, "tmp", n=s.intermediate_size, k=s.hidden_size, w=self.w_up),
             record("activate", "tmp", "act", n=s.intermediate_size, act=ACT[s.act]),
             record("linear", "act", "delta", n=s.hidden_size, k=s.intermediate_size, w=self.w_down) if into_stream is None else
             record("residual", "act", "x", n=s.hidden_size, k=s.intermediate_size, w=self.w_down, scale=float(into_stream)),

@@ -24,17 +24,17 @@ from ..kernels import host as _host
 
 _i, _f, _p, _ll = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_longlong
 
-SLOTS = ("x", "delta", "h", "q", "o", "act", "hw", "logits", "tmp", "decode", "mix", "scan", "x0", "route", "shift")       # RunnerSlot of csrc/runner.h
+SLOTS = ("x", "delta", "h", "q", "o", "act", "hw", "logits", "tmp", "decode", "mix", "scan", "x0", "route", "shift", "h2")       # RunnerSlot of csrc/runner.h
 SLOT = {name: i for i, name in enumerate(SLOTS)}
 OP_NAMES = {1: "embed", 2: "norm", 3: "qkv", 4: "attention", 5: "residual", 6: "gate_up", 7: "linear", 8: "cast",
             9: "layernorm", 10: "conv_qkv", 11: "linear_attention", 12: "norm_add", 13: "reinject", 14: "latent_qkv",
             15: "head_linear", 16: "latent_attention", 17: "causal_conv", 18: "selective_scan", 19: "experts", 20: "softcap",
-            21: "token_shift", 22: "activate", 23: "add_rows", 24: "delta_rule"}
+            21: "token_shift", 22: "activate", 23: "add_rows", 24: "delta_rule", 25: "norm_pair"}
 OP = {name: kind for kind, name in OP_NAMES.items()}                                # RunnerOpKind
 ACT = {"none": 0, "silu": 1, "gelu_tanh": 2, "sigmoid": 3, "relu": 4, "gelu_erf": 5, "swish_clamp": 6, "tanh": 7}    # RunnerAct
 _MIXERS_OPS = (OP["cast"], OP["layernorm"], OP["conv_qkv"], OP["linear_attention"], OP["token_shift"], OP["activate"], OP["delta_rule"])
 _BLOCKS_OPS = tuple(OP[n] for n in ("norm_add", "reinject", "latent_qkv", "head_linear", "latent_attention", "causal_conv",
-                                    "selective_scan", "experts", "softcap", "add_rows"))
+                                    "selective_scan", "experts", "softcap", "add_rows", "norm_pair"))
 MAX_GROUPS = 8
 MAX_LISTS = 8
 
@@ -62,7 +62,10 @@ class RunnerOp(ctypes.Structure):
                 # what learned positions, queries through a latent, the delta rule and a gated shared expert add
                 + [(n, _i) for n in ("fixed_row", "groups", "b_off", "a_off", "q_rank")]
                 + [("unit_eps", _f)]
-                + [(n, _p) for n in ("a_log", "dt_bias", "router_bias", "gate_w", "bonus")])
+                + [(n, _p) for n in ("a_log", "dt_bias", "router_bias", "gate_w", "bonus")]
+                # what learned sinks, gates of another shape, identity experts in groups and pairs of norms add
+                + [(n, _i) for n in ("group_count", "group_keep", "identity")]
+                + [(n, _p) for n in ("sink_w", "temp", "correction")])
 
 
 class Routing(ctypes.Structure):
@@ -95,7 +98,8 @@ class _Fns(ctypes.Structure):
         "linear_small_qkv_norm", "argmax", "sample", "err_sampling", "layernorm", "cast_rows", "glu", "conv_qkv", "linear_scan",
         "norm_gate", "token_shift", "act_rows", "err_mixers", "norm_add", "concat_cast", "add_bias_rows", "latent_qkv", "head_linear", "latent_attention",
         "latent_attention_scratch", "causal_conv", "selective_scan", "routed_experts", "routed_experts_workspace",
-        "routed_experts_launches", "softcap", "err_blocks", "linear_small_parts", "linear_small_parts_supports", "add_rows", "delta_rule", "delta_rule_scratch")]
+        "routed_experts_launches", "softcap", "err_blocks", "linear_small_parts", "linear_small_parts_supports", "add_rows", "delta_rule", "delta_rule_scratch",
+        "norm_pair")]
 
 
 def _addr(lib, name: str) -> int:
@@ -155,7 +159,8 @@ def runner_lib(gemm_tcgen05: bool = False, attention_tcgen05: bool = False, mixe
         err_blocks=get("blocks", "jk_blocks_last_error"),
         linear_small_parts=get("linear_small", "jk_linear_small_parts"),
         linear_small_parts_supports=get("linear_small", "jk_linear_small_parts_supports"),
-        add_rows=get("blocks", "jk_add_rows"), delta_rule=get("mixers", "jk_delta_rule"), delta_rule_scratch=get("mixers", "jk_delta_rule_scratch_floats"))
+        add_rows=get("blocks", "jk_add_rows"), delta_rule=get("mixers", "jk_delta_rule"), delta_rule_scratch=get("mixers", "jk_delta_rule_scratch_floats"),
+        norm_pair=get("blocks", "jk_norm_pair"))
     if lib.jk_runner_bind(ctypes.byref(fns)):
         from ..kernels import KernelError
         raise KernelError(lib.jk_runner_last_error().decode(errors="replace"))
