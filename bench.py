@@ -306,6 +306,25 @@ def fapenex_shape(width, ff, heads, kv_heads, dim, vocab, window):
             "logit_softcap": 30.0, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": [delta, att, lat, lat, delta, att]}
 
 
+def fupapel_shape(width, ff, heads, kv_heads, dim, vocab, window):
+    """Eight layers, mixers and feed-forwards side by side behind a token shift: attention with grouped heads of ``dim``, half of
+    each head rotated, chunks of ``window`` positions, a gate per output element; the same behind convolutions of three taps with
+    stretched frequencies, a factor and a learned sink per head, one such layer on another's keys and values; latent attention
+    with heads of ``dim`` plain and ``dim`` / 2 rotated elements, a latent vector of 4 dim, queries through a latent of 3/4 width.
+    Every layer has eight experts of ff / 4 and four identities in three groups, of which a row takes three from two groups."""
+    moe = {"kind": "moe", "router": {"experts": 8, "identity": 4, "top": 3, "groups": {"count": 3, "keep": 2}}, "expert": {"ff": ff // 4}}
+    heads_of = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window}}
+    att = {"type": "attention", "mlp": moe, "mixer": dict(heads_of, rot={"base": 1e4, "dims": dim // 2})}
+    conv = {"type": "attention_2", "mlp": moe,
+            "mixer": dict(heads_of, conv=3, rot={"base": 5e5, "dims": dim, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 1024}})}
+    borrows = {"type": "attention_2", "mlp": moe, "mixer": dict(conv["mixer"], kv_from=1)}
+    lat = {"type": "latent_attention", "mlp": moe,
+           "mixer": {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": 4 * dim, "q_rank": 3 * width // 4,
+                     "scale": (1.5 * dim) ** -0.5, "rot": {"base": 1e6, "dims": dim // 2}}}
+    return {"architecture": "Fupapel", "norm": {"eps": 1e-5}, "vocab": vocab, "width": width, "residual_mult": 0.5,
+            "layers": [att, conv, lat, lat, att, borrows, lat, att]}
+
+
 def decoder_shape(width, ff, heads, kv_heads, dim, vocab, layers=8):
     return dict(model_type="llama", num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv_heads,
                 head_dim=dim, intermediate_size=ff, vocab_size=vocab, max_position_embeddings=4096, rms_norm_eps=1e-5,
@@ -326,7 +345,8 @@ def record_cost(op, T, B, context, decode, page_bytes):
         reach = min(context, abs(op.window)) if op.window else context      # a negative window: chunks of that many positions
         keys = B * reach if decode else T       # cached rows that are read at least once
         seen = (B * reach) if decode else sum(min(t + 1, reach) for t in range(T))
-        return keys * op.kv_heads * (op.head_dim + dv) * 2 + 2 * T * op.heads * (op.head_dim + dv), 2.0 * seen * op.heads * (op.head_dim + dv)
+        gate = 4 * T * op.heads * (dv if op.gated == 2 else 1) if op.gated else 0
+        return keys * op.kv_heads * (op.head_dim + dv) * 2 + 2 * T * op.heads * (op.head_dim + dv) + gate, 2.0 * seen * op.heads * (op.head_dim + dv)
     if kind == "linear_attention":
         state = B * op.heads * op.head_dim * dv * 4 * 2
         return state + 4 * T * op.ld + 2 * T * op.heads * dv, 4.0 * T * op.heads * op.head_dim * dv
@@ -342,10 +362,14 @@ def record_cost(op, T, B, context, decode, page_bytes):
         return T * op.n * 6, 0.0
     if kind == "norm_add":
         return T * op.n * (4 + 4 + 4 + 2), 0.0
+    if kind == "norm_pair":
+        return T * op.n * (4 + 2 + (2 if op.out2_slot >= 0 else 0)) + B * op.n * 8, 0.0
     if kind == "reinject":
         return 2 * op.n * op.k + T * (8 * op.n + 2 * 2 * op.k + 8 * op.n), 2.0 * T * op.n * op.k
     if kind == "latent_qkv":
-        return 4 * T * op.ld + 2 * T * (op.heads * (op.head_dim + op.rot_width) + op.rank + op.rot_width), 0.0
+        queries = op.q_rank if op.q_rank else op.heads * (op.head_dim + op.rot_width)       # the queries' latent, or the heads' queries
+        row = op.rank + op.rot_width if op.k_off >= 0 else 0
+        return 4 * T * (queries + row) + 2 * T * (queries + row), 0.0
     if kind == "head_linear":
         return 2 * op.heads * op.n * op.k + 2 * T * op.heads * (op.k + op.n), 2.0 * T * op.heads * op.n * op.k
     if kind == "latent_attention":
@@ -364,18 +388,21 @@ def record_cost(op, T, B, context, decode, page_bytes):
     if kind == "add_rows":
         return T * op.n * (4 + 4 + 2), 0.0
     if kind == "experts":
-        used = min(op.experts, T * op.top)
-        return used * 3 * op.n * op.ff * 2 + T * op.n * (2 + 4) + T * op.top * (op.ff * 4 + op.n * 8), 2.0 * T * op.top * 3 * op.n * op.ff
+        pairs = T * op.top * op.experts / (op.experts + op.identity)         # random routers: choices of units with matrices, on average
+        used = min(op.experts, pairs)
+        return (used * 3 * op.n * op.ff * 2 + T * op.n * (2 + (8 if op.into_stream == 2 else 4)) + pairs * (op.ff * 4 + op.n * 8),
+                2.0 * pairs * 3 * op.n * op.ff)
     return 0, 0.0
 
 
 def run_design(args):
-    """Prefill and decode of another design (Sitelorn, Vunelix, Vipovik, Fapenex) at layer sizes of real models beside the decoder (llama graph) of
-    the same width, feed-forward, heads and layer count (Vipovik: also beside Sitelorn, Fapenex: also beside Vunelix, the designs closest to them), and every kind
+    """Prefill and decode of another design (Sitelorn, Vunelix, Vipovik, Fapenex, Fupapel) at layer sizes of real models beside the decoder (llama graph) of
+    the same width, feed-forward, heads and layer count (Vipovik: also beside Sitelorn, Fapenex: also beside Vunelix, Fupapel: also
+    beside Fapenex, the designs closest to them), and every kind
     of launch record of each timed alone against its roofline.  Prints one JSON line of its own kind; the default benchmark is
     untouched."""
     import torch
-    from infinicore_infer_b200.config import FapenexConfig, MiniCPMConfig, SitelornConfig, VipovikConfig, VunelixConfig
+    from infinicore_infer_b200.config import FapenexConfig, FupapelConfig, MiniCPMConfig, SitelornConfig, VipovikConfig, VunelixConfig
     from infinicore_infer_b200.engine import Engine, StepEntry
     from infinicore_infer_b200.parts import model_manifest
     from infinicore_infer_b200.parts.program import OP_NAMES
@@ -393,9 +420,12 @@ def run_design(args):
         for size in args.design_sizes.split(","):
             width, ff, heads, kv_heads, dim, vocab = DESIGN_SIZES[size]
             block = out["sizes"][size] = {"width": width, "ff": ff, "heads": heads, "kv_heads": kv_heads, "head_dim": dim, "layers": 8}
-            beside = {"vipovik": ("sitelorn",), "fapenex": ("vunelix",)}.get(args.design, ())
+            beside = {"vipovik": ("sitelorn",), "fapenex": ("vunelix",), "fupapel": ("fapenex",)}.get(args.design, ())
             for which in (args.design,) + beside + ("decoder",):
-                if which == "fapenex":
+                if which == "fupapel":
+                    cfg = FupapelConfig.from_dict(fupapel_shape(width, ff, heads, kv_heads, dim, vocab, args.design_window),
+                                                  max_tokens=max(4096, context + page))
+                elif which == "fapenex":
                     cfg = FapenexConfig.from_dict(fapenex_shape(width, ff, heads, kv_heads, dim, vocab, args.design_window),
                                                   max_tokens=max(4096, context + page))
                 elif which == "vipovik":
@@ -463,7 +493,7 @@ def run_design(args):
                     pos = engine.cache.length(ids[0])
                     for r in ids:
                         engine.cache.reserve(r, pos + 1)
-                    names = {}
+                    names, costs = {}, {}
                     for i in range(prog.count):
                         kind = OP_NAMES.get(prog.ops[i].kind)
                         if kind in ("embed",):
@@ -471,6 +501,11 @@ def run_design(args):
                         op = prog.ops[i]
                         key = f"{kind}:{op.n}x{op.k}" if kind in ("linear", "gate_up", "residual", "qkv", "head_linear") else \
                             (f"{kind}:{'projected' if op.rank else 'constant'}" if kind == "linear_attention" else kind)
+                        # records of one kind that move other amounts (two forms of it in one model) are rows of their own
+                        cost, base, n = record_cost(op, T, 1, T, False, page), key, 1
+                        while costs.setdefault(key, cost) != cost:
+                            n += 1
+                            key = f"{base}#{n}"
                         if not (op.wanted_rows and kind != "linear"):
                             names.setdefault(key, []).append(i)
                     kern = res["records"] = {key: {"count": len(idx)} for key, idx in names.items()}
@@ -516,7 +551,7 @@ def main():
                     help="run a few steps between cudaProfilerStart/Stop (for ncu --profile-from-start off) and exit")
     ap.add_argument("--shape", default="2b", choices=["2b", "1b", "8b"],
                     help="layer sizes: 2b is the headline configuration; the others are for profiles and side measurements")
-    ap.add_argument("--design", default=None, choices=["sitelorn", "vunelix", "vipovik", "fapenex"],
+    ap.add_argument("--design", default=None, choices=["sitelorn", "vunelix", "vipovik", "fapenex", "fupapel"],
                     help="instead of the benchmark: prefill and decode of this design at real layer sizes beside the decoder of equal size")
     ap.add_argument("--design-sizes", default="2k,4k", help="comma-separated names of " + ", ".join(sorted(DESIGN_SIZES)))
     ap.add_argument("--design-prompt", type=int, default=2048)

@@ -154,21 +154,64 @@ JK_EXPORT int jk_norm_add(const float *delta, float *x, const float *w, float ep
 // Two norms of one stream, the first with a token shift: with n_t = x[t] / sqrt(mean(x[t]^2) + eps) * w,
 //     h[t]  = T(n_t + (n_(t-1) - n_t) * mu)        (mu null: T(n_t))
 //     h2[t] = T(x[t] / sqrt(mean(x[t]^2) + eps2) * w2)        (h2 null: not made)
-// n_(t-1) of a portion's first row is last[slot] (float32; zeros when a request takes the slot).  A block takes RB rows in a
-// row: a thread keeps its elements of the row before, so a row is read once and the row ahead of the block's first once
-// more.  The kept row of a request with one row in the step moves on here (its elements are one thread's); of the others it
-// does in norm_pair_last, which makes the norm of their last row once more, after this kernel has read the slots.
+// n_(t-1) of a portion's first row is the row that the request's last step left (float32; zeros at position 0).  A block takes
+// RB rows, asks for all of them and the row ahead of them at once, and adds up their squares in one round.
+//
+// What is kept of a request is two rows that take turns, state[slot, 2, kept_floats(d)]: n, and behind it (the last word)
+// how many positions the sequence had when the row was written.  A step that starts at position p reads the row marked p and
+// leaves its last row, marked with the new length, in the other one, so the block with a request's first row and the block
+// with its last one never touch the same row (the marks start as 0 and the rows as zeros, which serves position 0).
 // ---------------------------------------------------------------------------------------------------------------
 struct NormPairArgs {
     const float *x, *w, *mu, *w2;
     float eps, eps2;
-    float *last;
-    const int *row_req, *req_start, *slot_ids;
+    float *state;
+    const int *row_req, *req_start, *req_pos, *slot_ids;
     void *h, *h2;
-    int T, d, RB;
+    int T, d;
 };
 
 constexpr int NP_THREADS = 512;
+
+__host__ __device__ __forceinline__ int norm_pair_kept_floats(int d) { return (d + 3) / 4 * 4 + 4; }
+JK_EXPORT int jk_norm_pair_kept_floats(int d) { return norm_pair_kept_floats(d); }
+
+// Row t in its request: whether it is the first or the last of the step, the kept row it reads (first) and the one it leaves
+// (last), and the mark that goes with the latter.  What this reads is read before the block's barrier, the mark written behind it.
+struct NormPairRow {
+    bool first, last;
+    float *from, *to;
+    int length;
+    __device__ __forceinline__ NormPairRow() : first(false), last(false), from(nullptr), to(nullptr), length(0) {}
+    __device__ __forceinline__ NormPairRow(const NormPairArgs &a, int t) : NormPairRow() {
+        if (a.mu == nullptr) return;
+        const int req = a.row_req[t], start = a.req_start[req], end = a.req_start[req + 1];
+        first = start == t;
+        last = end == t + 1;
+        if (!first && !last) return;
+        const int kept = norm_pair_kept_floats(a.d), pos = a.req_pos[req];
+        float *base = a.state + (size_t)a.slot_ids[req] * 2 * kept;
+        const bool second = *reinterpret_cast<const volatile int *>(base + kept - 1) != pos;      // the other row holds position pos
+        from = base + (second ? kept : 0);
+        to = base + (second ? 0 : kept);
+        length = pos + end - start;
+    }
+    __device__ __forceinline__ void mark(const NormPairArgs &a) const { reinterpret_cast<int *>(to)[norm_pair_kept_floats(a.d) - 1] = length; }
+};
+
+// n sums over a block at once: one barrier, every thread gets all of them.  scratch [n][32]
+template <int N>
+__device__ __forceinline__ void block_sums(float (&v)[N], float *scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = (blockDim.x + 31) >> 5;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        v[i] = warp_sum(v[i]);
+        if (lane == 0) scratch[i * 32 + warp] = v[i];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = warp_sum(lane < nwarp ? scratch[i * 32 + lane] : 0.f);
+}
 
 __device__ __forceinline__ float sumsq4(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
 __device__ __forceinline__ float4 scale4(float4 v, float s, float4 w) { return make_float4(v.x * s * w.x, v.y * s * w.y, v.z * s * w.z, v.w * s * w.w); }
@@ -176,64 +219,78 @@ __device__ __forceinline__ float4 mix4(float4 n, float4 before, float4 mu) {
     return make_float4(fmaf(before.x - n.x, mu.x, n.x), fmaf(before.y - n.y, mu.y, n.y), fmaf(before.z - n.z, mu.z, n.z), fmaf(before.w - n.w, mu.w, n.w));
 }
 
-template <typename T, int NV>       // NV vectors of four elements a thread
-__global__ void __launch_bounds__(NP_THREADS) norm_pair_kernel(NormPairArgs a) {
+// NV vectors of four elements a thread, RB rows a block.  The instances that take four rows are for steps of many: registers
+// for a full SM, since what a block waits for is the round trip of its loads and of its one barrier.
+template <typename T, int NV, int RB>
+__global__ void __launch_bounds__(NP_THREADS, RB == 4 ? 2 : 1) norm_pair_kernel(NormPairArgs a) {
     pdl_trigger();
-    __shared__ float scratch[33];
-    const int n4 = a.d / 4, t0 = blockIdx.x * a.RB, t1 = min(a.T, t0 + a.RB), step = blockDim.x;
+    __shared__ float scratch[(RB + 1) * 32];
+    constexpr bool EARLY = RB == 1;         // few rows: the weights are asked for ahead of the kernel before (no kernel writes them)
+    const int n4 = a.d / 4, t0 = blockIdx.x * RB, step = blockDim.x;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    float4 w[NV], w2[NV], mu[NV], before[NV], next[NV];
-    auto load = [&](float4 (&v)[NV], const float *row) {
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int c = threadIdx.x + i * step;
-            v[i] = c < n4 ? reinterpret_cast<const float4 *>(row)[c] : zero;
-        }
+    auto load = [&](const float *row, int c) { return row != nullptr && c < n4 ? reinterpret_cast<const float4 *>(row)[c] : zero; };
+    float4 w[NV], w2[NV], mu[NV];
+    auto load_weights = [&](int i) {
+        const int c = threadIdx.x + i * step;
+        w[i] = load(a.w, c);
+        w2[i] = load(a.h2 != nullptr ? a.w2 : nullptr, c);
+        mu[i] = load(a.mu, c);
     };
-    load(w, a.w);               // weights are there before any kernel of the step
-    if (a.h2 != nullptr) load(w2, a.w2);
-    if (a.mu != nullptr) load(mu, a.mu);
-    pdl_wait();
-    load(next, a.x + (size_t)t0 * a.d);
-    if (a.mu != nullptr && a.req_start[a.row_req[t0]] != t0) {
-        load(before, a.x + (size_t)(t0 - 1) * a.d);
-        float ss = 0.f;
+    if (EARLY) {
 #pragma unroll
-        for (int i = 0; i < NV; ++i) ss += sumsq4(before[i]);
-        const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
-#pragma unroll
-        for (int i = 0; i < NV; ++i) before[i] = scale4(before[i], inv, w[i]);
+        for (int i = 0; i < NV; ++i) load_weights(i);
     }
-    for (int t = t0; t < t1; ++t) {
-        float4 v[NV];
+    pdl_wait();
+    float4 v[RB + 1][NV];       // v[0]: the row ahead of the block's, or the kept row where the first starts a portion
 #pragma unroll
-        for (int i = 0; i < NV; ++i) v[i] = next[i];
-        if (t + 1 < t1) load(next, a.x + (size_t)(t + 1) * a.d);
-        float ss = 0.f;
+    for (int r = 0; r < RB; ++r)
 #pragma unroll
-        for (int i = 0; i < NV; ++i) ss += sumsq4(v[i]);
-        const float mean = block_sum(ss, scratch) / (float)a.d;
-        const float inv = 1.f / sqrtf(mean + a.eps), inv2 = 1.f / sqrtf(mean + a.eps2);
-        float *kept = nullptr;
-        bool only_row = false;
-        if (a.mu != nullptr) {
-            const int req = a.row_req[t];
-            if (a.req_start[req] == t) {
-                kept = a.last + (size_t)a.slot_ids[req] * a.d;
-                only_row = a.req_start[req + 1] == t + 1;
-                load(before, kept);
-            }
+        for (int i = 0; i < NV; ++i) v[r + 1][i] = load(t0 + r < a.T ? a.x + (size_t)(t0 + r) * a.d : nullptr, threadIdx.x + i * step);
+    NormPairRow at[RB];
+#pragma unroll
+    for (int r = 0; r < RB; ++r)
+        if (t0 + r < a.T) at[r] = NormPairRow(a, t0 + r);
+    const float *ahead = a.mu == nullptr ? nullptr : at[0].first ? at[0].from : a.x + (size_t)(t0 - 1) * a.d;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[0][i] = load(ahead, threadIdx.x + i * step);
+    float ss[RB + 1];
+#pragma unroll
+    for (int r = 0; r <= RB; ++r) {
+        ss[r] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss[r] += sumsq4(v[r][i]);
+    }
+    block_sums<RB + 1>(ss, scratch);
+    const bool norm_ahead = a.mu != nullptr && !at[0].first;        // the row ahead is one of this step: its norm, not the kept one's
+    float inv2[RB];
+#pragma unroll
+    for (int r = 0; r <= RB; ++r) {
+        const float mean = ss[r] / (float)a.d;
+        ss[r] = 1.f / sqrtf(mean + a.eps);
+        if (r > 0) inv2[r - 1] = 1.f / sqrtf(mean + a.eps2);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * step;
+        if (c >= n4) continue;
+        if (!EARLY) load_weights(i);
+        float4 before = norm_ahead ? scale4(v[0][i], ss[0], w[i]) : v[0][i];
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+            const int t = t0 + r;
+            if (t >= a.T) break;
+            if (r > 0 && at[r].first) before = load(at[r].from, c);
+            const float4 n = scale4(v[r + 1][i], ss[r + 1], w[i]);
+            store4((T *)a.h + (size_t)t * a.d + 4 * c, a.mu != nullptr ? mix4(n, before, mu[i]) : n);
+            if (a.h2 != nullptr) store4((T *)a.h2 + (size_t)t * a.d + 4 * c, scale4(v[r + 1][i], inv2[r], w2[i]));
+            if (at[r].last) reinterpret_cast<float4 *>(at[r].to)[c] = n;
+            before = n;
         }
+    }
+    if (threadIdx.x == 0) {
 #pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const int c = threadIdx.x + i * step;
-            if (c >= n4) continue;
-            const float4 n = scale4(v[i], inv, w[i]);
-            store4((T *)a.h + (size_t)t * a.d + 4 * c, a.mu != nullptr ? mix4(n, before[i], mu[i]) : n);
-            if (a.h2 != nullptr) store4((T *)a.h2 + (size_t)t * a.d + 4 * c, scale4(v[i], inv2, w2[i]));
-            if (only_row) reinterpret_cast<float4 *>(kept)[c] = n;
-            before[i] = n;
-        }
+        for (int r = 0; r < RB; ++r)
+            if (at[r].last) at[r].mark(a);
     }
 }
 
@@ -242,83 +299,61 @@ template <typename T>
 __global__ void __launch_bounds__(NP_THREADS) norm_pair_plain_kernel(NormPairArgs a) {
     pdl_trigger();
     pdl_wait();
-    __shared__ float scratch[33];
+    __shared__ float scratch[2 * 32];
     const int t = blockIdx.x;
-    const float *x = a.x + (size_t)t * a.d, *xb = nullptr;
-    float *kept = nullptr;
-    bool only_row = false;
-    if (a.mu != nullptr) {
-        const int req = a.row_req[t];
-        if (a.req_start[req] == t) {
-            kept = a.last + (size_t)a.slot_ids[req] * a.d;
-            only_row = a.req_start[req + 1] == t + 1;
-        } else {
-            xb = x - a.d;
-        }
-    }
-    float ss = 0.f, sb = 0.f;
+    const NormPairRow at(a, t);
+    const float *x = a.x + (size_t)t * a.d, *xb = a.mu != nullptr && !at.first ? x - a.d : nullptr;
+    float ss[2] = {0.f, 0.f};
     for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
-        ss += x[c] * x[c];
-        if (xb != nullptr) sb += xb[c] * xb[c];
+        ss[0] += x[c] * x[c];
+        if (xb != nullptr) ss[1] += xb[c] * xb[c];
     }
-    const float mean = block_sum(ss, scratch) / (float)a.d;
-    const float inv = 1.f / sqrtf(mean + a.eps), inv2 = 1.f / sqrtf(mean + a.eps2);
-    const float inv_b = xb != nullptr ? 1.f / sqrtf(block_sum(sb, scratch) / (float)a.d + a.eps) : 0.f;
+    block_sums<2>(ss, scratch);
+    const float mean = ss[0] / (float)a.d, inv = 1.f / sqrtf(mean + a.eps), inv2 = 1.f / sqrtf(mean + a.eps2);
+    const float inv_b = 1.f / sqrtf(ss[1] / (float)a.d + a.eps);
     for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
         const float n = x[c] * inv * a.w[c];
         float out = n;
         if (a.mu != nullptr) {
-            const float before = xb != nullptr ? xb[c] * inv_b * a.w[c] : kept[c];
+            const float before = xb != nullptr ? xb[c] * inv_b * a.w[c] : at.from[c];
             out = fmaf(before - n, a.mu[c], n);
-            if (only_row) kept[c] = n;
+            if (at.last) at.to[c] = n;
         }
         ((T *)a.h)[(size_t)t * a.d + c] = from_f32<T>(out);
         if (a.h2 != nullptr) ((T *)a.h2)[(size_t)t * a.d + c] = from_f32<T>(x[c] * inv2 * a.w2[c]);
     }
+    if (at.last && threadIdx.x == 0) at.mark(a);
 }
 
-// the kept rows of requests with several rows in the step
-__global__ void __launch_bounds__(NP_THREADS) norm_pair_last_kernel(NormPairArgs a) {
-    pdl_trigger();
-    pdl_wait();
-    __shared__ float scratch[33];
-    const int req = blockIdx.x, end = a.req_start[req + 1];
-    if (end - a.req_start[req] <= 1) return;
-    const float *x = a.x + (size_t)(end - 1) * a.d;
-    float *kept = a.last + (size_t)a.slot_ids[req] * a.d;
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < a.d; c += blockDim.x) ss += x[c] * x[c];
-    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
-    for (int c = threadIdx.x; c < a.d; c += blockDim.x) kept[c] = x[c] * inv * a.w[c];
-}
-
-JK_EXPORT int jk_norm_pair(const float *x, const float *w, const float *mu, float eps, const float *w2, float eps2, float *last,
-                           const int *row_req, const int *req_start, const int *slot_ids, void *h, void *h2, int dtype, int T, int nreq,
-                           int d, cudaStream_t stream) {
+JK_EXPORT int jk_norm_pair(const float *x, const float *w, const float *mu, float eps, const float *w2, float eps2, float *state,
+                           const int *row_req, const int *req_start, const int *req_pos, const int *slot_ids, void *h, void *h2, int dtype,
+                           int T, int d, cudaStream_t stream) {
     if (T == 0) return JK_OK;
     JK_REQUIRE(x && w && h && T > 0 && d > 0, "norm_pair: rows %d, width %d", T, d);
     JK_REQUIRE(h2 == nullptr || w2 != nullptr, "norm_pair: a second norm without its weight");
-    JK_REQUIRE(mu == nullptr || (last && row_req && req_start && slot_ids && nreq > 0), "norm_pair: a token shift without its kept rows");
+    JK_REQUIRE(mu == nullptr || (state && row_req && req_start && req_pos && slot_ids), "norm_pair: a token shift without its kept rows");
     const bool vec = d % 4 == 0 && d <= 4 * 4 * NP_THREADS && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)mu % 16 == 0 &&
-                     (uintptr_t)w2 % 16 == 0 && (uintptr_t)last % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)h2 % 16 == 0;
-    // rows a block: one where the rows do not fill the SMs four times over
-    const int RB = std::max(1, std::min(8, T / (4 * 148)));
-    NormPairArgs a{x, w, mu, w2, eps, eps2, last, row_req, req_start, slot_ids, h, h2, T, d, RB};
+                     (uintptr_t)w2 % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)h2 % 16 == 0;
+    const NormPairArgs a{x, w, mu, w2, eps, eps2, state, row_req, req_start, req_pos, slot_ids, h, h2, T, d};
+    // few rows: a thread takes one vector of a row; many: two, and several rows a block
     const int n4 = (d + 3) / 4;
-    const int threads = std::max(64, std::min(NP_THREADS, (n4 + 31) / 32 * 32));
+    const int NV = n4 <= (T <= 64 ? NP_THREADS : 128) ? 1 : (n4 <= 2 * NP_THREADS ? 2 : 4);
+    const int threads = vec ? std::max(64, ((n4 + NV - 1) / NV + 31) / 32 * 32) : std::max(64, std::min(NP_THREADS, (d + 31) / 32 * 32));
+    const int RB = NV == 4 ? (T >= 2 * 148 ? 2 : 1) : (T >= 4 * 148 ? 4 : (T >= 2 * 148 ? 2 : 1));
     const dim3 grid((T + RB - 1) / RB);
-#define LAUNCH(TT)                                                                                                   \
-    if (!vec) jk_launch(norm_pair_plain_kernel<TT>, dim3(T), dim3(threads), 0, stream, a);                           \
-    else if (n4 <= threads) jk_launch(norm_pair_kernel<TT, 1>, grid, dim3(threads), 0, stream, a);                   \
-    else if (n4 <= 2 * threads) jk_launch(norm_pair_kernel<TT, 2>, grid, dim3(threads), 0, stream, a);               \
-    else jk_launch(norm_pair_kernel<TT, 4>, grid, dim3(threads), 0, stream, a)
+#define LAUNCH_NV(TT, V)                                                                                            \
+    if (RB == 4 && V <= 2) jk_launch(norm_pair_kernel<TT, V, (V <= 2 ? 4 : 2)>, grid, dim3(threads), 0, stream, a); \
+    else if (RB == 2) jk_launch(norm_pair_kernel<TT, V, 2>, grid, dim3(threads), 0, stream, a);                     \
+    else jk_launch(norm_pair_kernel<TT, V, 1>, grid, dim3(threads), 0, stream, a)
+#define LAUNCH(TT)                                                                           \
+    if (!vec) jk_launch(norm_pair_plain_kernel<TT>, dim3(T), dim3(threads), 0, stream, a);   \
+    else if (NV == 1) { LAUNCH_NV(TT, 1); }                                                  \
+    else if (NV == 2) { LAUNCH_NV(TT, 2); }                                                  \
+    else { LAUNCH_NV(TT, 4); }
     BLOCKS_BY_DTYPE(dtype, "norm_pair", LAUNCH);
 #undef LAUNCH
+#undef LAUNCH_NV
     JK_CHECK_LAUNCH("norm_pair");
-    if (mu != nullptr && T > nreq) {
-        jk_launch(norm_pair_last_kernel, dim3(nreq), dim3(threads), 0, stream, a);
-        JK_CHECK_LAUNCH("norm_pair_last");
-    }
     return JK_OK;
 }
 

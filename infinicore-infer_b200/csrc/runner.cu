@@ -691,9 +691,8 @@ int run_norm_pair(Run &r, const RunnerOp &op) {
         if (int rc = r.slot(op.out2_slot, (long long)r.elem() * T * op.n, &h2, "the second norm of a pair")) return rc;
     JK_REQUIRE(op.bias == nullptr || (op.state != nullptr && r.st.slot_ids != nullptr), "runner: a token shift without its state slots");
     if (int rc = flush_pending(r, T, op.n)) return rc;
-    RUN(blocks, g_fns.norm_pair(r.x(), op.vec, op.bias, op.eps, op.vec2, op.eps2, op.state, r.st.row_req, r.st.req_start, r.st.slot_ids, h, h2,
-                                r.env.dtype, T, r.st.nreq, op.n, r.stream));
-    if (op.bias != nullptr && T > r.st.nreq) ++g_launches;      // the kept rows of requests with several rows
+    RUN(blocks, g_fns.norm_pair(r.x(), op.vec, op.bias, op.eps, op.vec2, op.eps2, op.state, r.st.row_req, r.st.req_start, r.st.req_pos, r.st.slot_ids,
+                                h, h2, r.env.dtype, T, op.n, r.stream));
     return JK_OK;
 }
 

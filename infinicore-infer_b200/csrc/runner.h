@@ -88,7 +88,7 @@ typedef int (*SoftcapFn)(float *, float, long long, cudaStream_t);
 typedef int (*AddRowsFn)(float *, const void *, int, int, const int *, int, int, int, cudaStream_t);
 // csrc/mixers.cu
 typedef int (*NormPairFn)(const float *, const float *, const float *, float, const float *, float, float *, const int *, const int *, const int *,
-                          void *, void *, int, int, int, int, cudaStream_t);
+                          const int *, void *, void *, int, int, int, cudaStream_t);
 typedef int (*DeltaRuleFn)(const float *, int, int, int, int, const float *, int, int, int, const float *, const float *, int, int, int, int,
                            float, float, float *, const int *, const int *, int, float *, float *, int, cudaStream_t);
 typedef long long (*DeltaScratchFn)(int, int, int, int);
@@ -229,7 +229,7 @@ enum RunnerOpKind {
                         // strength's and the decay's logits and the gate; S <- g S, S += k (beta (v - S^T k))^T, o = S^T q per head over
                         // each request's rows and its state slot; out = rmsnorm(o) * vec * act(gate)
     OP_NORM_PAIR,       // two norms of the same stream: out2 = rmsnorm(stream) * vec2 (out2_slot < 0: not made), and out = h_t + (h_(t-1) -
-                        // h_t) * bias with h = rmsnorm(stream) * vec; the row before a portion's first row is kept in state [slots, n]
+                        // h_t) * bias with h = rmsnorm(stream) * vec; the row before a portion's first row is kept in state (csrc/blocks.cu)
                         // (bias null: out = h, no state)
 };
 

@@ -723,16 +723,22 @@ def norm_add(delta: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: fl
     return x
 
 
+def norm_pair_kept_floats(width: int) -> int:
+    """Floats of one of the two rows that ``norm_pair`` keeps of a request: the row, and how long the sequence was then."""
+    return (width + 3) // 4 * 4 + 4
+
+
 def norm_pair(x: torch.Tensor, weight: torch.Tensor, eps: float, h: torch.Tensor, mu: Optional[torch.Tensor] = None,
-              last: Optional[torch.Tensor] = None, row_req=None, req_start=None, slot_ids=None, weight2: Optional[torch.Tensor] = None,
+              state: Optional[torch.Tensor] = None, row_req=None, req_start=None, req_pos=None, slot_ids=None, weight2: Optional[torch.Tensor] = None,
               eps2: float = 0.0, h2: Optional[torch.Tensor] = None) -> torch.Tensor:
     """h[t] = n_t + (n_(t-1) - n_t) * mu with n = rmsnorm(x) * weight (``mu`` None: n itself), the row before a request's first
-    row being ``last[slot]``, which then moves on to the n of its last row; h2 = rmsnorm(x) * weight2 if given."""
+    row being the one that ``state`` ``[slots, 2, norm_pair_kept_floats(width)]`` keeps of it, which then moves on to the n of its
+    last row; h2 = rmsnorm(x) * weight2 if given."""
     _need(x, "x", torch.float32); _need(weight, "weight", torch.float32); _need(h, "h")
     lib = _build.load("blocks")
-    _check("blocks", lib.jk_norm_pair(_ptr(x), _ptr(weight), _ptr(mu), _c_float(eps), _ptr(weight2), _c_float(eps2), _ptr(last), _ptr(row_req),
-                                      _ptr(req_start), _ptr(slot_ids), _ptr(h), _ptr(h2), _c_int(dtype_code(h.dtype)), _c_int(x.shape[0]),
-                                      _c_int(req_start.numel() - 1 if req_start is not None else 1), _c_int(x.shape[1]), _stream()))
+    _check("blocks", lib.jk_norm_pair(_ptr(x), _ptr(weight), _ptr(mu), _c_float(eps), _ptr(weight2), _c_float(eps2), _ptr(state), _ptr(row_req),
+                                      _ptr(req_start), _ptr(req_pos), _ptr(slot_ids), _ptr(h), _ptr(h2), _c_int(dtype_code(h.dtype)),
+                                      _c_int(x.shape[0]), _c_int(x.shape[1]), _stream()))
     return h
 
 

@@ -3,8 +3,8 @@
 Both norms read the stream as the layer found it, so one kernel makes both (``norm_pair``: the row and its mean square
 once), the first mixed with the row before it where the block has a token shift; the mixer reads its usual slot, the
 feed-forward a second one.  The mixer's output product then adds into the stream (or waits for it), and the feed-forward
-adds after it.  The row that the shift needs from the step before is kept per request in float32, beside whatever the
-mixer keeps.
+adds after it.  The row that the shift needs from the step before is kept per request in float32 (as two rows that take
+turns: a step reads one and leaves the other), beside whatever the mixer keeps.
 """
 from __future__ import annotations
 
@@ -12,6 +12,7 @@ import inspect
 from typing import Dict
 
 from ..cache import StateSlot, StateSlots
+from ..kernels import norm_pair_kept_floats
 from ..weights import VECTOR, TensorDecl
 from .base import part_class, register
 from .program import record
@@ -45,7 +46,7 @@ class ParallelBlock:
         mixer = ParallelBlock._mixer_state(spec, writes_cache)
         if not spec.shift_name:
             return mixer
-        own = (StateSlot((spec.mixer_norm.size,), "float32"),)
+        own = (StateSlot((2, norm_pair_kept_floats(spec.mixer_norm.size)), "float32"),)
         return StateSlots(own + (() if mixer is None else mixer.slots if isinstance(mixer, StateSlots) else (mixer,)))
 
     def __init__(self, spec, weights, prefix: str, runtime):
