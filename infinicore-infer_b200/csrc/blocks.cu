@@ -210,7 +210,15 @@ __device__ __forceinline__ void block_sums(float (&v)[N], float *scratch) {
     }
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = warp_sum(lane < nwarp ? scratch[i * 32 + lane] : 0.f);
+    for (int i = 0; i < N; ++i) {
+        if (nwarp <= 8) {
+            float t = 0.f;
+            for (int k = 0; k < nwarp; ++k) t += scratch[i * 32 + k];
+            v[i] = t;
+        } else {
+            v[i] = warp_sum(lane < nwarp ? scratch[i * 32 + lane] : 0.f);
+        }
+    }
 }
 
 __device__ __forceinline__ float sumsq4(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
@@ -219,10 +227,10 @@ __device__ __forceinline__ float4 mix4(float4 n, float4 before, float4 mu) {
     return make_float4(fmaf(before.x - n.x, mu.x, n.x), fmaf(before.y - n.y, mu.y, n.y), fmaf(before.z - n.z, mu.z, n.z), fmaf(before.w - n.w, mu.w, n.w));
 }
 
-// NV vectors of four elements a thread, RB rows a block.  The instances that take four rows are for steps of many: registers
-// for a full SM, since what a block waits for is the round trip of its loads and of its one barrier.
+// NV vectors of four elements a thread, RB rows a block: few threads with much of a row each, since the sums' shuffles are
+// what the kernel would otherwise spend its time on.
 template <typename T, int NV, int RB>
-__global__ void __launch_bounds__(NP_THREADS, RB == 4 ? 2 : 1) norm_pair_kernel(NormPairArgs a) {
+__global__ void __launch_bounds__(NP_THREADS) norm_pair_kernel(NormPairArgs a) {
     pdl_trigger();
     __shared__ float scratch[(RB + 1) * 32];
     constexpr bool EARLY = RB == 1;         // few rows: the weights are asked for ahead of the kernel before (no kernel writes them)
@@ -241,18 +249,18 @@ __global__ void __launch_bounds__(NP_THREADS, RB == 4 ? 2 : 1) norm_pair_kernel(
         for (int i = 0; i < NV; ++i) load_weights(i);
     }
     pdl_wait();
-    float4 v[RB + 1][NV];       // v[0]: the row ahead of the block's, or the kept row where the first starts a portion
+    float4 v[RB + 1][NV];       // v[0]: the row ahead of the block's
 #pragma unroll
-    for (int r = 0; r < RB; ++r)
+    for (int r = 0; r <= RB; ++r) {
+        const int t = t0 + r - 1;
+        const float *row = t < a.T && (r > 0 || (t >= 0 && a.mu != nullptr)) ? a.x + (size_t)t * a.d : nullptr;
 #pragma unroll
-        for (int i = 0; i < NV; ++i) v[r + 1][i] = load(t0 + r < a.T ? a.x + (size_t)(t0 + r) * a.d : nullptr, threadIdx.x + i * step);
+        for (int i = 0; i < NV; ++i) v[r][i] = load(row, threadIdx.x + i * step);
+    }
     NormPairRow at[RB];
 #pragma unroll
     for (int r = 0; r < RB; ++r)
         if (t0 + r < a.T) at[r] = NormPairRow(a, t0 + r);
-    const float *ahead = a.mu == nullptr ? nullptr : at[0].first ? at[0].from : a.x + (size_t)(t0 - 1) * a.d;
-#pragma unroll
-    for (int i = 0; i < NV; ++i) v[0][i] = load(ahead, threadIdx.x + i * step);
     float ss[RB + 1];
 #pragma unroll
     for (int r = 0; r <= RB; ++r) {
@@ -261,7 +269,6 @@ __global__ void __launch_bounds__(NP_THREADS, RB == 4 ? 2 : 1) norm_pair_kernel(
         for (int i = 0; i < NV; ++i) ss[r] += sumsq4(v[r][i]);
     }
     block_sums<RB + 1>(ss, scratch);
-    const bool norm_ahead = a.mu != nullptr && !at[0].first;        // the row ahead is one of this step: its norm, not the kept one's
     float inv2[RB];
 #pragma unroll
     for (int r = 0; r <= RB; ++r) {
@@ -274,12 +281,12 @@ __global__ void __launch_bounds__(NP_THREADS, RB == 4 ? 2 : 1) norm_pair_kernel(
         const int c = threadIdx.x + i * step;
         if (c >= n4) continue;
         if (!EARLY) load_weights(i);
-        float4 before = norm_ahead ? scale4(v[0][i], ss[0], w[i]) : v[0][i];
+        float4 before = scale4(v[0][i], ss[0], w[i]);
 #pragma unroll
         for (int r = 0; r < RB; ++r) {
             const int t = t0 + r;
             if (t >= a.T) break;
-            if (r > 0 && at[r].first) before = load(at[r].from, c);
+            if (at[r].first) before = load(at[r].from, c);         // the row that the step before left
             const float4 n = scale4(v[r + 1][i], ss[r + 1], w[i]);
             store4((T *)a.h + (size_t)t * a.d + 4 * c, a.mu != nullptr ? mix4(n, before, mu[i]) : n);
             if (a.h2 != nullptr) store4((T *)a.h2 + (size_t)t * a.d + 4 * c, scale4(v[r + 1][i], inv2[r], w2[i]));
@@ -335,15 +342,16 @@ JK_EXPORT int jk_norm_pair(const float *x, const float *w, const float *mu, floa
     const bool vec = d % 4 == 0 && d <= 4 * 4 * NP_THREADS && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)mu % 16 == 0 &&
                      (uintptr_t)w2 % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)h2 % 16 == 0;
     const NormPairArgs a{x, w, mu, w2, eps, eps2, state, row_req, req_start, req_pos, slot_ids, h, h2, T, d};
-    // few rows: a thread takes one vector of a row; many: two, and several rows a block
+    // few rows: a thread takes one vector of a row; many: four, and several rows a block (2,048 rows of 2,048 and of 4,096: 9.3
+    // and 17.2 us; with one vector a thread and a row a block 19.5 and 47.9)
     const int n4 = (d + 3) / 4;
-    const int NV = n4 <= (T <= 64 ? NP_THREADS : 128) ? 1 : (n4 <= 2 * NP_THREADS ? 2 : 4);
+    const int NV = T <= 64 ? (n4 <= NP_THREADS ? 1 : (n4 <= 2 * NP_THREADS ? 2 : 4)) : (n4 <= 64 ? 1 : (n4 <= 128 ? 2 : 4));
     const int threads = vec ? std::max(64, ((n4 + NV - 1) / NV + 31) / 32 * 32) : std::max(64, std::min(NP_THREADS, (d + 31) / 32 * 32));
-    const int RB = NV == 4 ? (T >= 2 * 148 ? 2 : 1) : (T >= 4 * 148 ? 4 : (T >= 2 * 148 ? 2 : 1));
+    const int RB = T >= 4 * 148 ? 4 : (T >= 2 * 148 ? 2 : 1);
     const dim3 grid((T + RB - 1) / RB);
-#define LAUNCH_NV(TT, V)                                                                                            \
-    if (RB == 4 && V <= 2) jk_launch(norm_pair_kernel<TT, V, (V <= 2 ? 4 : 2)>, grid, dim3(threads), 0, stream, a); \
-    else if (RB == 2) jk_launch(norm_pair_kernel<TT, V, 2>, grid, dim3(threads), 0, stream, a);                     \
+#define LAUNCH_NV(TT, V)                                                                        \
+    if (RB == 4) jk_launch(norm_pair_kernel<TT, V, 4>, grid, dim3(threads), 0, stream, a);      \
+    else if (RB == 2) jk_launch(norm_pair_kernel<TT, V, 2>, grid, dim3(threads), 0, stream, a); \
     else jk_launch(norm_pair_kernel<TT, V, 1>, grid, dim3(threads), 0, stream, a)
 #define LAUNCH(TT)                                                                           \
     if (!vec) jk_launch(norm_pair_plain_kernel<TT>, dim3(T), dim3(threads), 0, stream, a);   \
@@ -1549,15 +1557,37 @@ JK_EXPORT int jk_selective_scan(const float *x, const float *low, int ld_low, in
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// Routed experts.  route_topk: one block per row; logits z_e = router[e] . h in float32, scores sigmoid(z_e); the `top`
+// Routed experts.  route_topk: a block per row or per four rows; logits z_e = router[e] . h in float32, scores sigmoid(z_e); the `top`
 // experts of largest score (the lower index wins a tie) -> ids, scores [T, top], and the experts' counts.  route_sort:
-// one warp per expert lists its (row, choice) pairs in the order of the rows: entry -> source row, score; pair -> entry.
+// one block per expert lists its (row, choice) pairs in the order of the rows: entry -> source row, score; pair -> entry.
 // The experts' products then run over the entries, expert after expert, as tiles of the grouped kernels below; an
 // expert's input is score * h, which the first product applies to its sums (W (s h) = s (W h), in float32) before the
 // gate's activation.  expert_combine adds a row's `top` results in the order of its choices.
 // Options: a bias on the logits (`bias` [E]); a gate per row, sigmoid(gate_w . h), on what the sum is added to (a shared
 // unit's output that waits in delta).
 // ---------------------------------------------------------------------------------------------------------------
+template <typename T> struct Vec16;
+template <> struct Vec16<float> { static constexpr int N = 4; };
+template <> struct Vec16<__nv_bfloat16> { static constexpr int N = 8; };
+
+template <typename T>
+__device__ __forceinline__ void unpack16(const uint4 &v, float *f) {
+    if constexpr (Vec16<T>::N == 4) {
+        f[0] = __uint_as_float(v.x); f[1] = __uint_as_float(v.y); f[2] = __uint_as_float(v.z); f[3] = __uint_as_float(v.w);
+    } else {
+        const unsigned w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+    }
+}
+
+// eight elements of a row that starts on a 16-byte boundary
+__device__ __forceinline__ void load8(const float *p, float *f) {
+    *reinterpret_cast<float4 *>(f) = *reinterpret_cast<const float4 *>(p);
+    *reinterpret_cast<float4 *>(f + 4) = *reinterpret_cast<const float4 *>(p + 4);
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float *f) { unpack16<__nv_bfloat16>(*reinterpret_cast<const uint4 *>(p), f); }
+
 // The largest of n values (the lower index wins a tie) over a warp; every lane gets (value, index).  An index within the
 // list whatever the values are.
 __device__ __forceinline__ int warp_argmax(const float *v, int n, float *value) {
@@ -1579,70 +1609,83 @@ __device__ __forceinline__ int warp_argmax(const float *v, int n, float *value) 
 // N router outputs, of which the first E stand for experts with matrices and the rest for units that return their input.
 // score_form 0: sigmoid; 1: softmax over all, the chosen ones' scores divided by their sum; 2: softmax over all, as they are.
 // Forms 0 and 1 choose by the logits, form 2 by score + correction; with groups only outputs of the `group_keep` groups
-// (of N / group_count neighbours) whose best choice score is largest can be chosen.
-template <typename T>
-__global__ void route_topk_kernel(const T *__restrict__ h, const float *__restrict__ router, int D, int N, int E, int top, int *__restrict__ ids,
-                                  float *__restrict__ scores, int *__restrict__ counts, int score_form, const float *__restrict__ bias,
-                                  const float *__restrict__ gate_w, float *__restrict__ row_gate, const float *__restrict__ correction,
-                                  int group_count, int group_keep) {
+// (of N / group_count neighbours) whose best choice score is largest can be chosen.  A block takes R rows: a warp one output
+// at a time for all of them (a router row is read once a block), then a warp a row for the choice.
+struct RouteArgs {
+    const float *router, *bias, *gate_w, *correction;
+    int T, D, N, E, top, score_form, group_count, group_keep;
+    int *ids, *counts;
+    float *scores, *row_gate;
+};
+
+template <typename T, int R>
+__global__ void route_topk_kernel(const T *__restrict__ h, RouteArgs a) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ float z[];        // [N] logits, then scores; [N] choice scores; [group_count] best of a group; [group_count] kept
-    float *choice = z + N, *group_best = choice + N, *group_kept = group_best + group_count;
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
-    const T *row = h + (size_t)t * D;
-    const bool vec = D % 8 == 0 && (uintptr_t)row % 16 == 0 && (uintptr_t)router % 16 == 0;
-    for (int e = warp; e < N; e += nwarp) {
-        const float *w = router + (size_t)e * D;
-        float dot = 0.f;
+    extern __shared__ float route_smem[];       // per row: [N] logits, then scores; [N] choice scores; [group_count] best of a group, kept
+    const int N = a.N, D = a.D, row_floats = 2 * N + 2 * a.group_count;
+    const int t0 = blockIdx.x * R, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+    const bool vec = D % 8 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)a.router % 16 == 0 && (uintptr_t)a.gate_w % 16 == 0;
+    // output N: the row's gate on what the experts' sum is added to
+    for (int e = warp; e < (a.gate_w != nullptr ? N + 1 : N); e += nwarp) {
+        const float *w = e < N ? a.router + (size_t)e * D : a.gate_w;
+        float dot[R];
+#pragma unroll
+        for (int r = 0; r < R; ++r) dot[r] = 0.f;
         if (vec) {          // eight elements a lane a pass, the passes' loads independent of one another
 #pragma unroll 4
             for (int c = lane * 8; c < D; c += 256) {
-                const float4 w0 = *reinterpret_cast<const float4 *>(w + c), w1 = *reinterpret_cast<const float4 *>(w + c + 4);
-                float x[8];
+                float wv[8];
+                load8(w + c, wv);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) x[i] = to_f32(row[c + i]);
-                dot = fmaf(w0.x, x[0], dot); dot = fmaf(w0.y, x[1], dot); dot = fmaf(w0.z, x[2], dot); dot = fmaf(w0.w, x[3], dot);
-                dot = fmaf(w1.x, x[4], dot); dot = fmaf(w1.y, x[5], dot); dot = fmaf(w1.z, x[6], dot); dot = fmaf(w1.w, x[7], dot);
+                for (int r = 0; r < R; ++r) {
+                    float x[8];
+                    load8(h + (size_t)min(t0 + r, a.T - 1) * D + c, x);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) dot[r] = fmaf(wv[i], x[i], dot[r]);
+                }
             }
         } else {
-            for (int c = lane; c < D; c += 32) dot = fmaf(w[c], to_f32(row[c]), dot);
+            for (int c = lane; c < D; c += 32)
+#pragma unroll
+                for (int r = 0; r < R; ++r) dot[r] = fmaf(w[c], to_f32(h[(size_t)min(t0 + r, a.T - 1) * D + c]), dot[r]);
         }
-        dot = warp_sum(dot);
-        if (lane == 0) z[e] = dot + (bias ? bias[e] : 0.f);
-    }
-    if (gate_w != nullptr && warp == nwarp - 1) {       // the row's gate on what the experts' sum is added to: sigmoid(gate_w . h)
-        float dot = 0.f;
-        for (int c = lane; c < D; c += 32) dot = fmaf(gate_w[c], to_f32(row[c]), dot);
-        dot = warp_sum(dot);
-        if (lane == 0) row_gate[t] = sigmoid_f(dot);
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            dot[r] = warp_sum(dot[r]);
+            if (lane != 0) continue;
+            if (e < N) route_smem[r * row_floats + e] = dot[r] + (a.bias ? a.bias[e] : 0.f);
+            else if (t0 + r < a.T) a.row_gate[t0 + r] = sigmoid_f(dot[r]);
+        }
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int t = t0 + warp;
+    if (warp >= R || t >= a.T) return;
+    float *z = route_smem + warp * row_floats, *choice = z + N, *group_best = choice + N, *group_kept = group_best + a.group_count;
     float zmax = -INFINITY, total = 0.f, unused;
-    if (score_form != 0) {
+    if (a.score_form != 0) {
         for (int e = lane; e < N; e += 32) zmax = fmaxf(zmax, z[e]);
         zmax = warp_max(zmax);
         for (int e = lane; e < N; e += 32) total += expf(z[e] - zmax);
         total = warp_sum(total);
     }
     for (int e = lane; e < N; e += 32) {        // a lane's own outputs: no other lane touches them before the barrier
-        const float logit = z[e], s = score_form != 0 ? expf(logit - zmax) / total : sigmoid_f(logit);
-        choice[e] = score_form == 2 ? s + (correction ? correction[e] : 0.f) : logit;
+        const float logit = z[e], s = a.score_form != 0 ? expf(logit - zmax) / total : sigmoid_f(logit);
+        choice[e] = a.score_form == 2 ? s + (a.correction ? a.correction[e] : 0.f) : logit;
         z[e] = s;
     }
     __syncwarp();
-    if (group_count > 0) {
-        const int size = N / group_count;
-        for (int g = lane; g < group_count; g += 32) {
+    if (a.group_count > 0) {
+        const int size = N / a.group_count;
+        for (int g = lane; g < a.group_count; g += 32) {
             float b = -INFINITY;
             for (int i = 0; i < size; ++i) b = fmaxf(b, choice[g * size + i]);
             group_best[g] = b;
             group_kept[g] = 0.f;
         }
         __syncwarp();
-        for (int k = 0; k < group_keep; ++k) {
-            const int g = warp_argmax(group_best, group_count, &unused);
+        for (int k = 0; k < a.group_keep; ++k) {
+            const int g = warp_argmax(group_best, a.group_count, &unused);
             __syncwarp();
             if (lane == 0) { group_best[g] = -INFINITY; group_kept[g] = 1.f; }
             __syncwarp();
@@ -1652,59 +1695,67 @@ __global__ void route_topk_kernel(const T *__restrict__ h, const float *__restri
         __syncwarp();
     }
     float chosen = 0.f;
-    for (int k = 0; k < top; ++k) {
+    int *ids = a.ids + (size_t)t * a.top;
+    float *scores = a.scores + (size_t)t * a.top;
+    for (int k = 0; k < a.top; ++k) {
         const int best = warp_argmax(choice, N, &unused);
         const float sc = z[best];
         chosen += sc;
         __syncwarp();
         if (lane == 0) {
-            ids[(size_t)t * top + k] = best;
-            scores[(size_t)t * top + k] = sc;
-            if (best < E) atomicAdd(&counts[best], 1);
+            ids[k] = best;
+            scores[k] = sc;
+            if (best < a.E) atomicAdd(&a.counts[best], 1);
             choice[best] = -INFINITY;
         }
         __syncwarp();
     }
-    if (score_form == 1)
-        for (int k = lane; k < top; k += 32) scores[(size_t)t * top + k] /= chosen + 1e-20f;
+    if (a.score_form == 1)
+        for (int k = lane; k < a.top; k += 32) scores[k] /= chosen + 1e-20f;
 }
 
-// entry_row[pos], entry_score[pos] for pos in [starts[e], starts[e + 1]); pair_entry[pair] = pos
+// entry_row[pos], entry_score[pos] for pos in [starts[e], starts[e + 1]); pair_entry[pair] = pos.  A block an expert; each of its
+// warps takes a stretch of the pairs: it counts the expert's among them, and behind the barrier lists them from where the
+// warps before it end, so the entries are in the order of the rows.
+constexpr int RS_WARPS = 32;
+
 __global__ void route_sort_kernel(const int *__restrict__ ids, const float *__restrict__ scores, const int *__restrict__ counts, int pairs,
                                   int E, int top, int *__restrict__ starts, int *__restrict__ entry_row, float *__restrict__ entry_score,
                                   int *__restrict__ pair_entry) {
     pdl_trigger();
     pdl_wait();
-    const int lane = threadIdx.x & 31;
-    const int e = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (e >= E) return;
+    __shared__ int found[RS_WARPS];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5, e = blockIdx.x;
     int start = 0;
-    for (int i = 0; i < e; ++i) start += counts[i];
-    if (lane == 0) {
+    for (int i = lane; i < e; i += 32) start += counts[i];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) start += __shfl_xor_sync(0xffffffffu, start, o);
+    if (threadIdx.x == 0) {
         starts[e] = start;
         if (e == E - 1) starts[E] = start + counts[e];
     }
+    const int stretch = ((pairs + nwarp - 1) / nwarp + 31) / 32 * 32, first = warp * stretch, end = min(pairs, first + stretch);
+    int mine = 0;
+#pragma unroll 4
+    for (int p = first + lane; p < end; p += 32) mine += ids[p] == e ? 1 : 0;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mine += __shfl_xor_sync(0xffffffffu, mine, o);
+    if (lane == 0) found[warp] = mine;
+    __syncthreads();
     int at = start;
-    for (int p0 = 0; p0 < pairs; p0 += 128) {          // four passes of 32 pairs, their loads asked for together
-        int id[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int p = p0 + 32 * i + lane;
-            id[i] = p < pairs ? ids[p] : -1;
+    for (int i = 0; i < warp; ++i) at += found[i];
+    if (mine == 0) return;
+    for (int p0 = first; p0 < end; p0 += 32) {
+        const int p = p0 + lane;
+        const bool hit = p < end && ids[p] == e;
+        const unsigned ballot = __ballot_sync(0xffffffffu, hit);
+        if (hit) {
+            const int pos = at + __popc(ballot & ((1u << lane) - 1u));
+            entry_row[pos] = p / top;
+            entry_score[pos] = scores[p];
+            pair_entry[p] = pos;
         }
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int p = p0 + 32 * i + lane;
-            const bool mine = id[i] == e;
-            const unsigned ballot = __ballot_sync(0xffffffffu, mine);
-            if (mine) {
-                const int pos = at + __popc(ballot & ((1u << lane) - 1u));
-                entry_row[pos] = p / top;
-                entry_score[pos] = scores[p];
-                pair_entry[p] = pos;
-            }
-            at += __popc(ballot);
-        }
+        at += __popc(ballot);
     }
 }
 
@@ -1772,21 +1823,6 @@ __global__ void __launch_bounds__(256) expert_down_kernel(const T *__restrict__ 
 // per pass, all loads of a row asked for before the sums start.  Float32 sums on the CUDA cores, in the order of K per
 // lane and then across lanes, whatever else the step holds.
 constexpr int ER_ROWS = 8, ER_FEATURES = 32;        // entries at a time; output features a block
-
-template <typename T> struct Vec16;
-template <> struct Vec16<float> { static constexpr int N = 4; };
-template <> struct Vec16<__nv_bfloat16> { static constexpr int N = 8; };
-
-template <typename T>
-__device__ __forceinline__ void unpack16(const uint4 &v, float *f) {
-    if constexpr (Vec16<T>::N == 4) {
-        f[0] = __uint_as_float(v.x); f[1] = __uint_as_float(v.y); f[2] = __uint_as_float(v.z); f[3] = __uint_as_float(v.w);
-    } else {
-        const unsigned w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
-    }
-}
 
 // the features of one block against ROWS staged entries (the caller picks the smallest ROWS that holds them)
 template <typename T, bool GLU, int ROWS>
@@ -1966,11 +2002,16 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
     int *counts = route, *starts = counts + E, *ids = starts + E + 1, *entry_row = ids + pairs, *pair_entry = entry_row + pairs;
     float *scores = (float *)(pair_entry + pairs), *entry_score = scores + pairs, *row_gate = gate_w ? entry_score + pairs : nullptr;
     if (cudaMemsetAsync(counts, 0, sizeof(int) * (size_t)E, stream) != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "routed_experts: clearing the counts failed");
-#define LAUNCH(TT) jk_launch(route_topk_kernel<TT>, dim3(T), dim3(128), route_smem, stream, (const TT *)h, router, D, N, E, top, ids, scores, counts, score_form, router_bias, gate_w, row_gate, correction, group_count, group_keep)
+    const RouteArgs ra{router, router_bias, gate_w, correction, T, D, N, E, top, score_form, group_count, group_keep, ids, counts, scores, row_gate};
+    // few rows: a block a row with a warp for every output; many: four rows a block
+    const int many = T >= 512 && 4 * route_smem <= 40 * 1024, warps = many ? 8 : std::min(32, std::max(4, N));
+#define LAUNCH(TT)                                                                                                          \
+    if (many) jk_launch(route_topk_kernel<TT, 4>, dim3((T + 3) / 4), dim3(32 * warps), 4 * route_smem, stream, (const TT *)h, ra); \
+    else jk_launch(route_topk_kernel<TT, 1>, dim3(T), dim3(32 * warps), route_smem, stream, (const TT *)h, ra)
     BLOCKS_BY_DTYPE(dtype, "route_topk", LAUNCH);
 #undef LAUNCH
     JK_CHECK_LAUNCH("route_topk");
-    jk_launch(route_sort_kernel, dim3((E + 3) / 4), dim3(128), 0, stream, (const int *)ids, (const float *)scores, (const int *)counts, pairs, E, top,
+    jk_launch(route_sort_kernel, dim3(E), dim3(32 * std::max(1, std::min(RS_WARPS, pairs / 64))), 0, stream, (const int *)ids, (const float *)scores, (const int *)counts, pairs, E, top,
               starts, entry_row, entry_score, pair_entry);
     JK_CHECK_LAUNCH("route_sort");
     // few rows: the experts' matrices stream past their entries (rows of 16-byte multiples); else tiles
