@@ -65,7 +65,6 @@ struct AtArgs {
     float cap_raw;            // a cap on the scores divided by the softmax scale: raw s <- cap tanh(s / cap) (0: none)
     int keep_first;           // with a window: keys at positions below this stay visible when the window has passed them
     const float *sink_w;
-    int gate_elem;            // 1: the gate has one column per output element, gate[t, h dh + e]
 };
 
 // ---- PTX wrappers (see gemm_tcgen05.cu for the same set) -----------------------------------------
@@ -229,7 +228,9 @@ template <int DH> struct AtSmem {
     unsigned tmem_base;
 };
 
-template <int DH>
+// ELEM: the gate, if there is one, has a column per output element (an instance of its own, so that the others carry neither
+// its code nor its registers)
+template <int DH, bool ELEM>
 __global__ void __launch_bounds__(AT_THREADS, DH <= 64 ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, AtArgs a) {
@@ -509,9 +510,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const float w_mine = ex2(m_ref - m_all), w_other = ex2(other.x - m_all);
             // a sink adds its term 2^(sink - m_all); a gate multiplies the row's output
             float inv = 1.f / (l * w_mine + other.y * w_other + (a.sink ? exp2f(jk_sink_log2(a.sink_w, h) - m_all) : 0.f));
-            const float *gate = a.gate != nullptr && row < nrows ? a.gate + (size_t)(row0 + row) * a.gate_ld : nullptr;
-            if (gate != nullptr && !a.gate_elem) { inv *= jk_sigmoid(gate[h]); gate = nullptr; }
-            if (gate != nullptr) gate += (size_t)h * DH + half * (DH / 2);         // the gates of this thread's columns
+            if (!ELEM && a.gate != nullptr && row < nrows) inv *= jk_sigmoid(a.gate[(size_t)(row0 + row) * a.gate_ld + h]);
+            const float *gate = ELEM && row < nrows ? a.gate + (size_t)(row0 + row) * a.gate_ld + (size_t)h * DH + half * (DH / 2) : nullptr;   // of this thread's columns
             const float w0 = (half ? w_other : w_mine) * inv, w1 = (half ? w_mine : w_other) * inv;
             // this thread writes columns [half * DH / 2, + DH / 2) of its row
             __nv_bfloat16 *dst = a.out + ((size_t)(row0 + row) * a.nh + h) * DH + half * (DH / 2);
@@ -525,8 +525,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
                         unsigned w[4];
-                        float z[8];
-                        if (gate != nullptr) {
+                        float z[ELEM ? 8 : 1];
+                        if constexpr (ELEM) {
                             const float *g = gate + c * 32 + j;
                             if ((uintptr_t)g % 16 == 0) {
                                 *reinterpret_cast<float4 *>(z) = *reinterpret_cast<const float4 *>(g);
@@ -540,7 +540,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                         for (int q = 0; q < 4; ++q) {
                             float lo = __uint_as_float(o0[j + 2 * q]) * w0 + __uint_as_float(o1[j + 2 * q]) * w1;
                             float hi = __uint_as_float(o0[j + 2 * q + 1]) * w0 + __uint_as_float(o1[j + 2 * q + 1]) * w1;
-                            if (gate != nullptr) { lo *= jk_sigmoid(z[2 * q]); hi *= jk_sigmoid(z[2 * q + 1]); }
+                            if constexpr (ELEM) { lo *= jk_sigmoid(z[2 * q]); hi *= jk_sigmoid(z[2 * q + 1]); }
                             const __nv_bfloat162 b = __floats2bfloat162_rn(lo, hi);
                             w[q] = *reinterpret_cast<const unsigned *>(&b);
                         }
@@ -609,12 +609,12 @@ JK_EXPORT int jk_attention_tcgen05_supports(int dh, int page_size) {
     return (dh == 64 || dh == 128) && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64 || page_size == 128);
 }
 
-template <int DH>
+template <int DH, bool ELEM>
 static int launch_at(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const AtArgs &a, cudaStream_t stream) {
     const size_t smem = sizeof(AtSmem<DH>);
-    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<DH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<DH, ELEM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "attention_tcgen05: %s", cudaGetErrorString(e));
-    jk_launch(attention_tcgen05_kernel<DH>, dim3(a.nh, a.ntiles), dim3(AT_THREADS), smem, stream, mq, mk, mv, a);
+    jk_launch(attention_tcgen05_kernel<DH, ELEM>, dim3(a.nh, a.ntiles), dim3(AT_THREADS), smem, stream, mq, mk, mv, a);
     JK_CHECK_LAUNCH("attention_tcgen05");
     return JK_OK;
 }
@@ -635,8 +635,9 @@ JK_EXPORT int jk_attention_tcgen05(const void *q, const void *k_pages, const voi
     if (int rc = tensor_map(v_pages, (long long)num_pages * nkvh * page_size, dh, page_size, &mv)) return rc;
     AtArgs a{(__nv_bfloat16 *)out, tiles, req_start, req_pos, block_table, status,
              ntiles, nh, nkvh, page_size, max_blocks, window, scale * 1.4426950408889634f, sink, gate, gate_ld,
-             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w, gate_elem};
+             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w};
     JK_REQUIRE(cap >= 0.f && keep_first >= 0 && scale > 0.f, "attention_tcgen05: cap %g, %d kept keys, scale %g", cap, keep_first, scale);
-    if (dh == 64) return launch_at<64>(mq, mk, mv, a, stream);
-    return launch_at<128>(mq, mk, mv, a, stream);
+    const bool elem = gate != nullptr && gate_elem;
+    if (dh == 64) return elem ? launch_at<64, true>(mq, mk, mv, a, stream) : launch_at<64, false>(mq, mk, mv, a, stream);
+    return elem ? launch_at<128, true>(mq, mk, mv, a, stream) : launch_at<128, false>(mq, mk, mv, a, stream);
 }
