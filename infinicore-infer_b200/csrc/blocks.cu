@@ -15,6 +15,9 @@
 //   selective_scan      S <- exp(dt A) S + dt x B, y = S C + D x per channel, with dt = softplus(W low + b) formed here
 //   route_topk, route_sort, expert products, expert_combine      experts chosen per token by their scores
 //   softcap             cap * tanh(logits / cap)
+//   embed_pair          embedding plus a vector per pair of neighbouring tokens, normed
+//   join_parts          the outputs of sublayers side by side, each normed or not, added into the stream
+//   gated_recurrence    S <- a S + sqrt(1 - a^2) i u per channel with gates from block-diagonal maps of u
 //
 // Everything that the design wants in float32 is float32 here: norms, angles, scores and softmax weights, routers, the
 // scan's state, decays, step sizes and gates.  Products take operands of the activation type T (float or bfloat16) and
@@ -63,7 +66,8 @@ __device__ __forceinline__ float expert_inner(int act, float s, float g, float u
 
 // ---------------------------------------------------------------------------------------------------------------
 // x[r] += delta[r] / sqrt(mean(delta[r]^2) + eps) * w;  then, if `out` is given,
-// out[r] = T(x[r] / sqrt(mean(x[r]^2) + eps2) * w_next)   (w_next null: out[r] = T(x[r])).
+// out[r] = T(x[r] / sqrt(mean(x[r]^2) + eps2) * w_next)   (w_next null: out[r] = T(x[r])), and with out2 the same with the weight
+// w_next2 (two sublayers side by side read the same stream).
 // One block per row; the row stays in shared memory between the passes.
 // ---------------------------------------------------------------------------------------------------------------
 __device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
@@ -77,7 +81,8 @@ __device__ __forceinline__ void store4(__nv_bfloat16 *p, float4 v) {
 // VEC: the width is a multiple of four and every operand starts on a 16-byte boundary: four elements move at a time
 template <typename T, bool VEC>
 __global__ void norm_add_kernel(const float *__restrict__ delta, float *__restrict__ x, const float *__restrict__ w, float eps,
-                                const float *__restrict__ w_next, float eps2, T *__restrict__ out, int d) {
+                                const float *__restrict__ w_next, float eps2, T *__restrict__ out, const float *__restrict__ w_next2,
+                                T *__restrict__ out2, int d) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float row_buf[];
@@ -120,27 +125,34 @@ __global__ void norm_add_kernel(const float *__restrict__ delta, float *__restri
             const float4 v = *reinterpret_cast<const float4 *>(row_buf + c);
             const float4 wv = w_next != nullptr ? *reinterpret_cast<const float4 *>(w_next + c) : make_float4(1.f, 1.f, 1.f, 1.f);
             store4(out + base + c, w_next != nullptr ? make_float4(v.x * inv2 * wv.x, v.y * inv2 * wv.y, v.z * inv2 * wv.z, v.w * inv2 * wv.w) : v);
+            if (out2 != nullptr) {
+                const float4 w2 = *reinterpret_cast<const float4 *>(w_next2 + c);
+                store4(out2 + base + c, make_float4(v.x * inv2 * w2.x, v.y * inv2 * w2.y, v.z * inv2 * w2.z, v.w * inv2 * w2.w));
+            }
         } else {
             out[base + c] = from_f32<T>(w_next != nullptr ? row_buf[c] * inv2 * w_next[c] : row_buf[c]);
+            if (out2 != nullptr) out2[base + c] = from_f32<T>(row_buf[c] * inv2 * w_next2[c]);
         }
     }
 }
 
 JK_EXPORT int jk_norm_add(const float *delta, float *x, const float *w, float eps, const float *w_next, float eps2, void *out,
-                          int dtype, int rows, int d, cudaStream_t stream) {
+                          const float *w_next2, void *out2, int dtype, int rows, int d, cudaStream_t stream) {
     if (rows == 0) return JK_OK;
     JK_REQUIRE(delta && x && w && rows > 0 && d > 0, "norm_add: rows %d, width %d", rows, d);
     const size_t smem = (size_t)d * sizeof(float);
     JK_REQUIRE(smem <= 200 * 1024, "norm_add: width %d does not fit shared memory", d);
+    JK_REQUIRE(out2 == nullptr || (out && w_next && w_next2), "norm_add: a second norm without the first or without its weight");
     const bool vec = d % 4 == 0 && (uintptr_t)delta % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
-                     (w_next == nullptr || (uintptr_t)w_next % 16 == 0) && (out == nullptr || (uintptr_t)out % 16 == 0);
+                     (w_next == nullptr || (uintptr_t)w_next % 16 == 0) && (out == nullptr || (uintptr_t)out % 16 == 0) &&
+                     (uintptr_t)w_next2 % 16 == 0 && (uintptr_t)out2 % 16 == 0;
     // a step of few rows has few blocks: then a thread takes one vector of the row, so that a pass is one round of loads
     int threads = d >= 4096 ? 512 : (d >= 1024 ? 256 : 128);
     if (rows <= 64 && vec) threads = std::min(1024, std::max(threads, (d / 4 + 31) / 32 * 32));
 #define LAUNCH_V(T, V)                                                                                                              \
     do {                                                                                                                            \
         if (smem > 48 * 1024) cudaFuncSetAttribute(norm_add_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        jk_launch(norm_add_kernel<T, V>, dim3(rows), dim3(threads), smem, stream, delta, x, w, eps, w_next, eps2, (T *)out, d);   \
+        jk_launch(norm_add_kernel<T, V>, dim3(rows), dim3(threads), smem, stream, delta, x, w, eps, w_next, eps2, (T *)out, w_next2, (T *)out2, d);   \
     } while (0)
 #define LAUNCH(T) if (vec) LAUNCH_V(T, true); else LAUNCH_V(T, false)
     BLOCKS_BY_DTYPE(dtype, "norm_add", LAUNCH);
@@ -684,35 +696,55 @@ __device__ __forceinline__ void tile_product(const __nv_bfloat16 *__restrict__ A
 }
 
 // C = A W^T for a float32 A and a bfloat16 W on the tensor cores without rounding A: every element of A is cut into two
-// bfloat16 halves (a = hi + lo, which keeps 16 bits of its mantissa) and both halves meet the same weights.
-__device__ __forceinline__ void tile_product_split(const float *__restrict__ A, size_t lda, int M, const __nv_bfloat16 *__restrict__ W, size_t ldw,
-                                                   int N, int K, int m0, int n0, float (&acc)[16]) {
+// bfloat16 halves (a = hi + lo, which keeps 16 bits of its mantissa) and both halves meet the same weights.  With TWO a second
+// weight tile runs along.  The next step of K is on its way in registers while the tensor cores work on this one.
+template <bool TWO>
+__device__ __forceinline__ void tile_product_split(const float *__restrict__ A, size_t lda, int M, const __nv_bfloat16 *__restrict__ W,
+                                                   const __nv_bfloat16 *__restrict__ W2, size_t ldw, int N, int K, int m0, int n0,
+                                                   float (&acc)[16], float (&acc2)[16]) {
     __shared__ __align__(16) __nv_bfloat16 Ah[GT_M * TC_LD];
     __shared__ __align__(16) __nv_bfloat16 Al[GT_M * TC_LD];
     __shared__ __align__(16) __nv_bfloat16 Ws[GT_N * TC_LD];
+    __shared__ __align__(16) __nv_bfloat16 W2s[TWO ? GT_N * TC_LD : 8];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int lr = tid / 4, lk = (tid % 4) * 8;
     const int am = m0 + lr, wn = n0 + lr;
     const float *arow = am < M ? A + (size_t)am * lda : nullptr;
     const __nv_bfloat16 *wrow = wn < N ? W + (size_t)wn * ldw : nullptr;
-    const bool vec_w = ldw % 8 == 0 && (uintptr_t)W % 16 == 0;
+    const __nv_bfloat16 *w2row = (TWO && wn < N) ? W2 + (size_t)wn * ldw : nullptr;
+    const bool vec_w = ldw % 8 == 0 && (uintptr_t)W % 16 == 0 && (!TWO || (uintptr_t)W2 % 16 == 0);
+    const bool vec_a = lda % 4 == 0 && (uintptr_t)A % 16 == 0;
 #pragma unroll
-    for (int e = 0; e < 16; ++e) acc[e] = 0.f;
+    for (int e = 0; e < 16; ++e) { acc[e] = 0.f; acc2[e] = 0.f; }
     const int a_row = (warp & 3) * 16 + (lane & 15), a_col = (lane >> 4) * 8;
     const int b_row = (warp >> 2) * 32 + (lane >> 4) * 8 + (lane & 7), b_col = ((lane >> 3) & 1) * 8;
+    __align__(16) float av[8];
+    uint4 wv, w2v = make_uint4(0u, 0u, 0u, 0u);
+    auto fetch = [&](int k0) {
+        if (vec_a && arow != nullptr && k0 + lk + 8 <= K) {
+            *reinterpret_cast<float4 *>(av) = *reinterpret_cast<const float4 *>(arow + k0 + lk);
+            *reinterpret_cast<float4 *>(av + 4) = *reinterpret_cast<const float4 *>(arow + k0 + lk + 4);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) av[i] = (arow != nullptr && k0 + lk + i < K) ? arow[k0 + lk + i] : 0.f;
+        }
+        wv = fetch8(wrow, k0 + lk, K, vec_w);
+        if (TWO) w2v = fetch8(w2row, k0 + lk, K, vec_w);
+    };
+    fetch(0);
     for (int k0 = 0; k0 < K; k0 += TC_K) {
-        __nv_bfloat16 h8[8], l8[8];
+        __align__(16) __nv_bfloat16 h8[8], l8[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            const int k = k0 + lk + i;
-            const float v = (arow && k < K) ? arow[k] : 0.f;
-            h8[i] = __float2bfloat16_rn(v);
-            l8[i] = __float2bfloat16_rn(v - __bfloat162float(h8[i]));
+            h8[i] = __float2bfloat16_rn(av[i]);
+            l8[i] = __float2bfloat16_rn(av[i] - __bfloat162float(h8[i]));
         }
         *reinterpret_cast<uint4 *>(Ah + lr * TC_LD + lk) = *reinterpret_cast<const uint4 *>(h8);
         *reinterpret_cast<uint4 *>(Al + lr * TC_LD + lk) = *reinterpret_cast<const uint4 *>(l8);
-        *reinterpret_cast<uint4 *>(Ws + lr * TC_LD + lk) = fetch8(wrow, k0 + lk, K, vec_w);
+        *reinterpret_cast<uint4 *>(Ws + lr * TC_LD + lk) = wv;
+        if (TWO) *reinterpret_cast<uint4 *>(W2s + lr * TC_LD + lk) = w2v;
         __syncthreads();
+        if (k0 + TC_K < K) fetch(k0 + TC_K);
 #pragma unroll
         for (int kk = 0; kk < TC_K; kk += 16) {
             unsigned h0, h1, h2, h3, l0, l1, l2, l3;
@@ -726,6 +758,13 @@ __device__ __forceinline__ void tile_product_split(const float *__restrict__ A, 
                 mma_bf16_16816(acc + (2 * p + 1) * 4, l0, l1, l2, l3, b2, b3);
                 mma_bf16_16816(acc + (2 * p) * 4, h0, h1, h2, h3, b0, b1);
                 mma_bf16_16816(acc + (2 * p + 1) * 4, h0, h1, h2, h3, b2, b3);
+                if (TWO) {
+                    ldmatrix_x4(b0, b1, b2, b3, W2s + (b_row + p * 16) * TC_LD + kk + b_col);
+                    mma_bf16_16816(acc2 + (2 * p) * 4, l0, l1, l2, l3, b0, b1);
+                    mma_bf16_16816(acc2 + (2 * p + 1) * 4, l0, l1, l2, l3, b2, b3);
+                    mma_bf16_16816(acc2 + (2 * p) * 4, h0, h1, h2, h3, b0, b1);
+                    mma_bf16_16816(acc2 + (2 * p + 1) * 4, h0, h1, h2, h3, b2, b3);
+                }
             }
         }
         __syncthreads();
@@ -1279,8 +1318,9 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
 // ---------------------------------------------------------------------------------------------------------------
 // A short causal convolution over time on each of C channels, with bias and activation:
 //     y_t[c] = act(bias[c] + sum_j taps[c, j] * u_(t - J + 1 + j)[c])          zeros before the sequence starts
-// u is a column range of float32 rows [T, ld].  The J - 1 rows before a portion come from the request's tail
-// [slots, J - 1, C] (s = J - 2 the newest), which conv_tails then moves forward.  y goes out as float32 (what a
+// u is a column range of float32 rows [T, ld], with in_bias[c] added (the projection's bias; not before the sequence starts).  The
+// J - 1 rows before a portion come from the request's tail [slots, J - 1, C] (s = J - 2 the newest; in_bias included), which moves
+// forward: that of a request with one row in the step in the row's own pass (a channel is one thread's), the others' by conv_tails.  y goes out as float32 (what a
 // recurrence reads) and in the activation type (what a product reads).
 // ---------------------------------------------------------------------------------------------------------------
 struct ConvArgs {
@@ -1291,6 +1331,7 @@ struct ConvArgs {
     const int *row_req, *req_start, *slot_ids;
     float *y32;
     void *yT;
+    const float *in_bias;
 };
 
 template <typename T>
@@ -1302,12 +1343,17 @@ __global__ void causal_conv_kernel(ConvArgs a, int rows) {
         const int t = (int)(i / a.C), c = (int)(i % a.C);
         const int req = a.row_req[t];
         const int back = t - a.req_start[req];
-        const float *tail = a.J > 1 ? a.tail + (size_t)a.slot_ids[req] * (a.J - 1) * a.C : nullptr;
-        float acc = a.bias ? a.bias[c] : 0.f;
+        float *tail = a.J > 1 ? a.tail + (size_t)a.slot_ids[req] * (a.J - 1) * a.C : nullptr;
+        float acc = a.bias ? a.bias[c] : 0.f, uv = 0.f;
+        const float in_bias = a.in_bias ? a.in_bias[c] : 0.f;
         for (int j = 0; j < a.J; ++j) {
             const int d = a.J - 1 - j;          // rows back
-            const float uv = d <= back ? a.u[(size_t)(t - d) * a.ld + a.off + c] : tail[(size_t)(a.J - 1 + back - d) * a.C + c];
+            uv = d <= back ? a.u[(size_t)(t - d) * a.ld + a.off + c] + in_bias : tail[(size_t)(a.J - 1 + back - d) * a.C + c];
             acc = fmaf(a.taps[(size_t)c * a.J + j], uv, acc);
+        }
+        if (tail != nullptr && a.req_start[req + 1] - a.req_start[req] == 1) {
+            for (int s = 0; s + 2 < a.J; ++s) tail[(size_t)s * a.C + c] = tail[(size_t)(s + 1) * a.C + c];
+            tail[(size_t)(a.J - 2) * a.C + c] = uv;          // the row's own input
         }
         const float y = block_act(a.act, acc);
         if (a.y32) a.y32[i] = y;
@@ -1324,28 +1370,30 @@ __global__ void conv_tails_kernel(ConvArgs a, int nreq) {
     if (idx >= nreq * a.C) return;
     const int req = idx / a.C, c = idx % a.C;
     const int first = a.req_start[req], n = a.req_start[req + 1] - first;
+    if (n == 1) return;         // moved forward by the row's own thread
     float *tail = a.tail + (size_t)a.slot_ids[req] * (a.J - 1) * a.C;
+    const float in_bias = a.in_bias ? a.in_bias[c] : 0.f;
     for (int s = 0; s < a.J - 1; ++s) {
         const int off = n - (a.J - 1) + s;
-        const float v = off >= 0 ? a.u[(size_t)(first + off) * a.ld + a.off + c] : tail[(size_t)(s + n) * a.C + c];
+        const float v = off >= 0 ? a.u[(size_t)(first + off) * a.ld + a.off + c] + in_bias : tail[(size_t)(s + n) * a.C + c];
         tail[(size_t)s * a.C + c] = v;
     }
 }
 
 JK_EXPORT int jk_causal_conv(const float *u, int ld, int off, int C, const float *taps, const float *bias, int J, int act, float *tail,
                              const int *row_req, const int *req_start, const int *slot_ids, float *y32, void *yT, int dtype, int T,
-                             int nreq, cudaStream_t stream) {
+                             int nreq, const float *in_bias, cudaStream_t stream) {
     if (T == 0) return JK_OK;
     JK_REQUIRE(u && taps && row_req && req_start && C > 0 && J >= 1 && (y32 || yT), "causal_conv: an argument is missing");
     JK_REQUIRE(J == 1 || (tail && slot_ids), "causal_conv: %d taps without the tails' state", J);
-    ConvArgs a{u, ld, off, C, J, act, taps, bias, tail, row_req, req_start, slot_ids, y32, yT};
+    ConvArgs a{u, ld, off, C, J, act, taps, bias, tail, row_req, req_start, slot_ids, y32, yT, in_bias};
     const size_t total = (size_t)T * C;
     const int blocks = (int)std::min<size_t>((total + 255) / 256, 148 * 16);
 #define LAUNCH(TT) jk_launch(causal_conv_kernel<TT>, dim3(blocks), dim3(256), 0, stream, a, T)
     BLOCKS_BY_DTYPE(dtype, "causal_conv", LAUNCH);
 #undef LAUNCH
     JK_CHECK_LAUNCH("causal_conv");
-    if (J > 1) {
+    if (J > 1 && T > nreq) {
         jk_launch(conv_tails_kernel, dim3((nreq * C + 127) / 128), dim3(128), 0, stream, a, nreq);
         JK_CHECK_LAUNCH("conv_tails");
     }
@@ -1387,11 +1435,10 @@ __global__ void __launch_bounds__(256) scan_steps_kernel(const float *__restrict
     pdl_trigger();
     pdl_wait();
     const int m0 = blockIdx.x * GT_M, n0 = blockIdx.y * GT_N;
-    float acc[16];
+    float acc[16], unused[16];
     if constexpr (OnTensorCores<TW>::value) {
-        tile_product_split(low, (size_t)ld_low, rows, Wdt, (size_t)K, E, K, m0, n0, acc);
+        tile_product_split<false>(low, (size_t)ld_low, rows, Wdt, (const TW *)nullptr, (size_t)K, E, K, m0, n0, acc, unused);
     } else {
-        float unused[16];
         tile_product<false>(low, (size_t)ld_low, nullptr, rows, Wdt, (const float *)nullptr, (size_t)K, E, K, m0, n0, acc, unused);
     }
 #pragma unroll
@@ -1607,7 +1654,7 @@ __device__ __forceinline__ int warp_argmax(const float *v, int n, float *value) 
 }
 
 // N router outputs, of which the first E stand for experts with matrices and the rest for units that return their input.
-// score_form 0: sigmoid; 1: softmax over all, the chosen ones' scores divided by their sum; 2: softmax over all, as they are.
+// score_form 0: sigmoid; 1: softmax over all, the chosen ones' scores divided by their sum, times score_scale; 2: softmax over all, as they are.
 // Forms 0 and 1 choose by the logits, form 2 by score + correction; with groups only outputs of the `group_keep` groups
 // (of N / group_count neighbours) whose best choice score is largest can be chosen.  A block takes R rows: a warp one output
 // at a time for all of them (a router row is read once a block), then a warp a row for the choice.
@@ -1616,6 +1663,7 @@ struct RouteArgs {
     int T, D, N, E, top, score_form, group_count, group_keep;
     int *ids, *counts;
     float *scores, *row_gate;
+    float score_scale;          // form 1: factor of the renormalised scores
 };
 
 template <typename T, int R>
@@ -1711,7 +1759,7 @@ __global__ void route_topk_kernel(const T *__restrict__ h, RouteArgs a) {
         __syncwarp();
     }
     if (a.score_form == 1)
-        for (int k = lane; k < a.top; k += 32) scores[k] /= chosen + 1e-20f;
+        for (int k = lane; k < a.top; k += 32) scores[k] = scores[k] / (chosen + 1e-20f) * a.score_scale;
 }
 
 // entry_row[pos], entry_score[pos] for pos in [starts[e], starts[e + 1]); pair_entry[pair] = pos.  A block an expert; each of its
@@ -1985,7 +2033,7 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
                                 int dtype, int T, int D, int ff, int E, int top, int actf, int *route, void *act, float *y,
                                 int score_form, float limit, const float *router_bias, const float *gate_w, int identity, int group_count,
                                 int group_keep, const float *correction, float *x, float x_scale, const float *pend, float pend_scale,
-                                cudaStream_t stream) {
+                                float score_scale, cudaStream_t stream) {
     if (T == 0) return JK_OK;
     const int N = E + identity;
     JK_REQUIRE(gate_w == nullptr || add, "routed_experts: a gate on a shared unit's output that is not there");
@@ -1996,13 +2044,14 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
     JK_REQUIRE(group_count == 0 || (group_count > 0 && N % group_count == 0 && group_keep > 0 && group_keep <= group_count && group_keep * (N / group_count) >= top),
                "routed_experts: %d of %d groups of %d outputs for %d choices", group_keep, group_count, N, top);
     JK_REQUIRE(pend == nullptr || x != nullptr, "routed_experts: a product that waits needs the stream");
+    JK_REQUIRE(score_scale == 1.f || score_form == 1, "routed_experts: a factor of scores of form %d", score_form);
     const size_t route_smem = (2 * (size_t)N + 2 * (size_t)group_count) * sizeof(float);
     JK_REQUIRE(route_smem <= 40 * 1024, "routed_experts: %d experts exceed the router's shared memory", N);
     const int pairs = T * top;
     int *counts = route, *starts = counts + E, *ids = starts + E + 1, *entry_row = ids + pairs, *pair_entry = entry_row + pairs;
     float *scores = (float *)(pair_entry + pairs), *entry_score = scores + pairs, *row_gate = gate_w ? entry_score + pairs : nullptr;
     if (cudaMemsetAsync(counts, 0, sizeof(int) * (size_t)E, stream) != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "routed_experts: clearing the counts failed");
-    const RouteArgs ra{router, router_bias, gate_w, correction, T, D, N, E, top, score_form, group_count, group_keep, ids, counts, scores, row_gate};
+    const RouteArgs ra{router, router_bias, gate_w, correction, T, D, N, E, top, score_form, group_count, group_keep, ids, counts, scores, row_gate, score_scale};
     // few rows: a block a row with a warp for every output; many: four rows a block
     const int many = T >= 512 && 4 * route_smem <= 40 * 1024, warps = many ? 8 : std::min(32, std::max(4, N));
 #define LAUNCH(TT)                                                                                                          \
@@ -2101,5 +2150,451 @@ JK_EXPORT int jk_softcap(float *x, float cap, long long n, cudaStream_t stream) 
     JK_REQUIRE(x && n > 0 && cap > 0.f, "softcap: %lld values, cap %f", n, (double)cap);
     jk_launch(softcap_kernel, dim3((int)std::min<long long>((n + 255) / 256, 148 * 16)), dim3(256), 0, stream, x, cap, (size_t)n);
     JK_CHECK_LAUNCH("softcap");
+    return JK_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Embedding with a vector per pair of neighbouring tokens and a norm:
+//     v_t = scale * table[token_t] + pairs[r_t],   r_t = (prev_t * mul_prev + token_t * mul_cur) mod buckets, or `buckets` at position 0
+//     x_t = v_t / sqrt(mean(v_t^2) + eps) * w        (w null: x_t = v_t; pairs null: no second vector)
+// prev_t of a portion's first row is the last token of the request's step before.  What is kept of a request is two marked tokens
+// that take turns, state[slot, 2] of (positions the sequence had then, token): a step that starts at position p reads the one marked
+// p and leaves its last token, marked with the new length, in the other, so the block with a request's first row and the one with
+// its last never touch the same (the scheme of norm_pair's kept rows).  One block per row.
+// ---------------------------------------------------------------------------------------------------------------
+struct EmbedPairArgs {
+    const int *tokens, *positions, *row_req, *req_start, *req_pos, *slot_ids;
+    const void *table, *pairs;
+    int buckets;
+    long long mul_prev, mul_cur;
+    float scale;
+    int *state;             // [slots, 2, 2]
+    const float *w;
+    float eps;
+    float *x;
+    int d;
+};
+
+template <typename TW>
+__global__ void embed_pair_kernel(EmbedPairArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float row_buf[];
+    __shared__ float scratch[33];
+    __shared__ int pair_row;
+    const int t = blockIdx.x, token = a.tokens[t];
+    const TW *src = (const TW *)a.table + (size_t)token * a.d;
+    if (a.pairs != nullptr && threadIdx.x == 0) {
+        const int req = a.row_req[t], start = a.req_start[req], end = a.req_start[req + 1], pos = a.req_pos[req];
+        int row = a.buckets;
+        int *kept = nullptr;
+        bool second = false;
+        if (t == start || t + 1 == end) {
+            kept = a.state + (size_t)a.slot_ids[req] * 4;
+            second = *reinterpret_cast<volatile int *>(kept) != pos;        // the other one is marked with position pos
+        }
+        if (a.positions[t] > 0) {
+            const int prev = t > start ? a.tokens[t - 1] : kept[second ? 3 : 1];
+            row = (int)(((long long)prev * a.mul_prev + (long long)token * a.mul_cur) % a.buckets);
+        }
+        if (t + 1 == end) {
+            int *to = kept + (second ? 0 : 2);
+            to[1] = token;
+            to[0] = pos + end - start;
+        }
+        pair_row = row;
+    }
+    __syncthreads();
+    const TW *add = a.pairs != nullptr ? (const TW *)a.pairs + (size_t)pair_row * a.d : nullptr;
+    float *dst = a.x + (size_t)t * a.d;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
+        float v = a.scale * to_f32(src[c]);
+        if (add != nullptr) v += to_f32(add[c]);
+        if (a.w == nullptr) dst[c] = v;
+        else row_buf[c] = v;
+        ss += v * v;
+    }
+    if (a.w == nullptr) return;
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) dst[c] = row_buf[c] * inv * a.w[c];
+}
+
+// tables of type `dtype`; pairs [buckets + 1, d]
+JK_EXPORT int jk_embed_pair(const int *tokens, const int *positions, const int *row_req, const int *req_start, const int *req_pos, const int *slot_ids,
+                            const void *table, const void *pairs, int dtype, int buckets, int mul_prev, int mul_cur, float scale, int *state,
+                            const float *w, float eps, float *x, int T, int d, cudaStream_t stream) {
+    if (T == 0) return JK_OK;
+    JK_REQUIRE(tokens && table && x && d > 0, "embed_pair: an argument is missing");
+    JK_REQUIRE(pairs == nullptr || (positions && row_req && req_start && req_pos && slot_ids && state && buckets > 0 && mul_prev >= 0 && mul_cur >= 0),
+               "embed_pair: a table of pairs of %d rows without the requests' last tokens", buckets);
+    const size_t smem = w != nullptr ? (size_t)d * sizeof(float) : 0;
+    JK_REQUIRE(smem <= 200 * 1024, "embed_pair: width %d does not fit shared memory", d);
+    const EmbedPairArgs a{tokens, positions, row_req, req_start, req_pos, slot_ids, table, pairs, buckets, mul_prev, mul_cur, scale, state, w, eps, x, d};
+    const int threads = T <= 64 ? std::min(1024, std::max(128, (d / 2 + 31) / 32 * 32)) : (d >= 1024 ? 256 : 128);
+#define LAUNCH(TT)                                                                                                                     \
+    do {                                                                                                                               \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(embed_pair_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+        jk_launch(embed_pair_kernel<TT>, dim3(T), dim3(threads), smem, stream, a);                                                     \
+    } while (0)
+    BLOCKS_BY_DTYPE(dtype, "embed_pair", LAUNCH);
+#undef LAUNCH
+    JK_CHECK_LAUNCH("embed_pair");
+    return JK_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// What several sublayers side by side leave, into the stream by one kernel:
+//     x[r] += f(p1[r], w1) + f(p2[r], w2) + p3[r],   f(p, w) = p / sqrt(mean(p^2) + eps) * w, or p where w is null
+// (p2, p3 null: absent), and out[r] = T(x[r]) if `out` is given.  One block per row.
+// ---------------------------------------------------------------------------------------------------------------
+struct JoinArgs {
+    float *x;
+    const float *p1, *w1, *p2, *w2, *p3;
+    float eps1, eps2;
+    void *out;
+    int d;
+};
+
+template <typename T, bool VEC>
+__global__ void join_parts_kernel(JoinArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[64];
+    constexpr int S = VEC ? 4 : 1;
+    struct __align__(4 * S) Vec { float f[S]; };
+    const size_t base = (size_t)blockIdx.x * a.d;
+    float ss[2] = {0.f, 0.f};
+    if (a.w1 != nullptr || a.w2 != nullptr) {
+        for (int c = threadIdx.x * S; c < a.d; c += blockDim.x * S) {
+            const Vec v = *reinterpret_cast<const Vec *>(a.p1 + base + c);
+#pragma unroll
+            for (int e = 0; e < S; ++e) ss[0] += v.f[e] * v.f[e];
+            if (a.p2 != nullptr) {
+                const Vec u = *reinterpret_cast<const Vec *>(a.p2 + base + c);
+#pragma unroll
+                for (int e = 0; e < S; ++e) ss[1] += u.f[e] * u.f[e];
+            }
+        }
+        block_sums<2>(ss, scratch);
+    }
+    const float inv1 = a.w1 != nullptr ? 1.f / sqrtf(ss[0] / (float)a.d + a.eps1) : 1.f;
+    const float inv2 = a.w2 != nullptr ? 1.f / sqrtf(ss[1] / (float)a.d + a.eps2) : 1.f;
+    for (int c = threadIdx.x * S; c < a.d; c += blockDim.x * S) {        // the row again: it comes from the caches
+        Vec x = *reinterpret_cast<const Vec *>(a.x + base + c), v = *reinterpret_cast<const Vec *>(a.p1 + base + c), w;
+        if (a.w1 != nullptr) {
+            w = *reinterpret_cast<const Vec *>(a.w1 + c);
+#pragma unroll
+            for (int e = 0; e < S; ++e) v.f[e] *= inv1 * w.f[e];
+        }
+        if (a.p2 != nullptr) {
+            const Vec u = *reinterpret_cast<const Vec *>(a.p2 + base + c);
+            if (a.w2 != nullptr) w = *reinterpret_cast<const Vec *>(a.w2 + c);
+#pragma unroll
+            for (int e = 0; e < S; ++e) v.f[e] += a.w2 != nullptr ? u.f[e] * inv2 * w.f[e] : u.f[e];
+        }
+        if (a.p3 != nullptr) {
+            const Vec u = *reinterpret_cast<const Vec *>(a.p3 + base + c);
+#pragma unroll
+            for (int e = 0; e < S; ++e) v.f[e] += u.f[e];
+        }
+#pragma unroll
+        for (int e = 0; e < S; ++e) x.f[e] += v.f[e];
+        *reinterpret_cast<Vec *>(a.x + base + c) = x;
+        if (a.out != nullptr) {
+            if constexpr (VEC) store4((T *)a.out + base + c, make_float4(x.f[0], x.f[1], x.f[2], x.f[3]));
+            else ((T *)a.out)[base + c] = from_f32<T>(x.f[0]);
+        }
+    }
+}
+
+JK_EXPORT int jk_join_parts(float *x, const float *p1, const float *w1, float eps1, const float *p2, const float *w2, float eps2, const float *p3,
+                            void *out, int dtype, int rows, int d, cudaStream_t stream) {
+    if (rows == 0) return JK_OK;
+    JK_REQUIRE(x && p1 && rows > 0 && d > 0 && (w2 == nullptr || p2 != nullptr), "join_parts: an argument is missing");
+    const bool vec = d % 4 == 0 && ((uintptr_t)x | (uintptr_t)p1 | (uintptr_t)w1 | (uintptr_t)p2 | (uintptr_t)w2 | (uintptr_t)p3 | (uintptr_t)out) % 16 == 0;
+    const JoinArgs a{x, p1, w1, p2, w2, p3, eps1, eps2, out, d};
+    int threads = d >= 4096 ? 512 : (d >= 1024 ? 256 : 128);
+    if (rows <= 64 && vec) threads = std::min(1024, std::max(threads, (d / 4 + 31) / 32 * 32));
+#define LAUNCH(T)                                                                                      \
+    if (vec) jk_launch(join_parts_kernel<T, true>, dim3(rows), dim3(threads), 0, stream, a);           \
+    else jk_launch(join_parts_kernel<T, false>, dim3(rows), dim3(threads), 0, stream, a)
+    BLOCKS_BY_DTYPE(dtype, "join_parts", LAUNCH);
+#undef LAUNCH
+    JK_CHECK_LAUNCH("join_parts");
+    return JK_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// A real-gated linear recurrence, per channel c of C over a request's rows in order:
+//     r = sigmoid(R u_t + rb)[c],  i = sigmoid(I u_t + ib)[c],  log a = rate[c] r,  a = exp(log a)
+//     S <- a S + sqrt(1 - a^2) i u_t[c];      out_t[c] = T(S * act(y_t[c] + yb[c]))
+// u float32 [T, C].  R and I are block-diagonal: C is cut into `blocks` equal parts of n channels, each with its own n x n matrices
+// (w_r, w_i [blocks, n, n], rows are outputs); rate[c] is negative (so a < 1), and y is a column range of float32 rows.  The state
+// S lives in state[slot, c], float32.  Everything is float32; in bfloat16 mode the float32 rows u meet the stored weights on the
+// tensor cores as two bfloat16 halves each, so that nothing of them is rounded away.
+//
+// Three ways:
+//   every request brings one row      gated_rows: gates, state and output of 8 rows x 16 channels a block
+//   else                              gated_pairs makes (a, sqrt(1 - a^2) i u) of every row as one tiled product per part;
+//                                     gated_scan then walks the work items: a request of at most SCAN_PIECE rows from its slot and
+//                                     back; of a longer one, cut into pieces, the first piece from the slot (its rows leave at
+//                                     once), the others from zeros (leaving their end state and the product of their decays);
+//                                     gated_finish gives the other pieces their start state, the pieces before them joined in
+//                                     order, and walks them again; the last one leaves the slot.  Nothing is divided by a decay.
+// ---------------------------------------------------------------------------------------------------------------
+struct GatedArgs {
+    const float *u;
+    const void *w_r, *w_i;
+    const float *b_r, *b_i, *rate;
+    const float *y;             // y_t[c] = y[t * ld_y + c]
+    int ld_y;
+    const float *y_bias;
+    int act;
+    float *state;
+    const int *req_start, *slot_ids;
+    void *out;                  // [T, C]
+    int T, C, blocks, n;
+    float *a, *b;               // [T, C] each: the recurrence's pairs
+    float *piece_end, *piece_prod;      // [n_pieces, C]
+    const int *direct, *pieces, *piece_reqs;
+    int n_direct, n_pieces, n_piece_reqs;
+};
+
+// (a, sqrt(1 - a^2) i u) from the two gates' sums
+__device__ __forceinline__ void gated_pair(float zr, float zi, float rate, float u, float *a, float *b) {
+    const float la = rate * sigmoid_f(zr);
+    *a = expf(la);
+    *b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi) * u;
+}
+
+template <typename TW>
+__global__ void __launch_bounds__(256) gated_pairs_kernel(GatedArgs g) {
+    pdl_trigger();
+    pdl_wait();
+    const int blk = blockIdx.z, m0 = blockIdx.x * GT_M, n0 = blockIdx.y * GT_N, n = g.n;
+    const float *A = g.u + (size_t)blk * n;
+    const TW *wr = (const TW *)g.w_r + (size_t)blk * n * n, *wi = (const TW *)g.w_i + (size_t)blk * n * n;
+    float zr[16], zi[16];
+    if constexpr (OnTensorCores<TW>::value) tile_product_split<true>(A, (size_t)g.C, g.T, wr, wi, (size_t)n, n, n, m0, n0, zr, zi);
+    else tile_product<true>(A, (size_t)g.C, nullptr, g.T, wr, wi, (size_t)n, n, n, m0, n0, zr, zi);
+#pragma unroll
+    for (int e = 0; e < 16; ++e) {
+        int r, k;
+        tile_at<TW>(e, &r, &k);
+        const int t = m0 + r;
+        if (t >= g.T || n0 + k >= n) continue;
+        const int c = blk * n + n0 + k;
+        const size_t at = (size_t)t * g.C + c;
+        gated_pair(zr[e] + g.b_r[c], zi[e] + g.b_i[c], g.rate[c], g.u[at], g.a + at, g.b + at);
+    }
+}
+
+constexpr int GS_THREADS = 128, GS_AHEAD = 8;
+
+// rows [first, last) of channel c from state s; OUT: their outputs; else the product of their decays into *prod
+template <typename T, bool OUT>
+__device__ __forceinline__ float gated_walk(const GatedArgs &g, int c, int first, int last, float s, float *prod) {
+    const float yb = OUT && g.y_bias != nullptr ? g.y_bias[c] : 0.f;
+    float p = 1.f;
+    for (int t0 = first; t0 < last; t0 += GS_AHEAD) {
+        float a[GS_AHEAD], b[GS_AHEAD], y[GS_AHEAD];
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j) {
+            const size_t t = min(t0 + j, last - 1);
+            a[j] = g.a[t * g.C + c];
+            b[j] = g.b[t * g.C + c];
+            y[j] = OUT ? g.y[t * g.ld_y + c] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j) {
+            if (t0 + j >= last) break;
+            s = fmaf(a[j], s, b[j]);
+            if (OUT) ((T *)g.out)[(size_t)(t0 + j) * g.C + c] = from_f32<T>(s * block_act(g.act, y[j] + yb));
+            else p *= a[j];
+        }
+    }
+    if (!OUT) *prod = p;
+    return s;
+}
+
+// whose piece p is: (the request's first piece, its pieces, the request)
+__device__ __forceinline__ int3 gated_piece_of(const GatedArgs &g, int p) {
+    for (int i = 0; i < g.n_piece_reqs; ++i) {
+        const int first = g.piece_reqs[3 * i + 1], n = g.piece_reqs[3 * i + 2];
+        if (p >= first && p < first + n) return make_int3(first, n, g.piece_reqs[3 * i]);
+    }
+    return make_int3(p, 1, 0);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(GS_THREADS) gated_scan_kernel(GatedArgs g) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * GS_THREADS + threadIdx.x, item = blockIdx.y;
+    if (c >= g.C) return;
+    if (item < g.n_direct) {
+        const int req = g.direct ? g.direct[item] : item;
+        float *S = g.state + (size_t)g.slot_ids[req] * g.C + c;
+        *S = gated_walk<T, true>(g, c, g.req_start[req], g.req_start[req + 1], *S, nullptr);
+        return;
+    }
+    const int p = item - g.n_direct, first = g.pieces[2 * p], last = first + g.pieces[2 * p + 1];
+    const int3 of = gated_piece_of(g, p);
+    if (p == of.x) {
+        float *S = g.state + (size_t)g.slot_ids[of.z] * g.C + c;
+        const float s = gated_walk<T, true>(g, c, first, last, *S, nullptr);
+        g.piece_end[(size_t)p * g.C + c] = s;
+        if (of.y == 1) *S = s;
+    } else {
+        float prod;
+        g.piece_end[(size_t)p * g.C + c] = gated_walk<T, false>(g, c, first, last, 0.f, &prod);
+        g.piece_prod[(size_t)p * g.C + c] = prod;
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(GS_THREADS) gated_finish_kernel(GatedArgs g) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * GS_THREADS + threadIdx.x, p = blockIdx.y;
+    if (c >= g.C) return;
+    const int3 of = gated_piece_of(g, p);
+    if (p == of.x) return;
+    float s = g.piece_end[(size_t)of.x * g.C + c];
+    for (int q0 = of.x + 1; q0 < p; q0 += GS_AHEAD) {
+        float e[GS_AHEAD], d[GS_AHEAD];
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j) {
+            const size_t q = min(q0 + j, p - 1);
+            e[j] = g.piece_end[q * g.C + c];
+            d[j] = g.piece_prod[q * g.C + c];
+        }
+#pragma unroll
+        for (int j = 0; j < GS_AHEAD; ++j)
+            if (q0 + j < p) s = fmaf(d[j], s, e[j]);
+    }
+    const int first = g.pieces[2 * p], last = first + g.pieces[2 * p + 1];
+    s = gated_walk<T, true>(g, c, first, last, s, nullptr);
+    if (p == of.x + of.y - 1) g.state[(size_t)g.slot_ids[of.z] * g.C + c] = s;
+}
+
+// One row a request (row t is request t's): GR_ROWS rows and GR_CHANNELS channels of one part a block.  The rows' inputs wait in
+// shared memory; a warp takes a channel at a time, its lanes the row of both matrices; then lane r does row r's step.
+constexpr int GR_ROWS = 8, GR_CHANNELS = 16;
+
+template <typename T, int ROWS>
+__device__ __forceinline__ void gated_rows_body(const GatedArgs &g, const float *rows_u, int t0, int live, int blk, int c_first) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = g.n;
+    constexpr int V = Vec16<T>::N;
+    const bool vec = n % V == 0 && n % 4 == 0 && ((uintptr_t)g.w_r | (uintptr_t)g.w_i) % 16 == 0;
+    for (int k = c_first + warp; k < min(n, c_first + GR_CHANNELS); k += 8) {
+        const T *wr = (const T *)g.w_r + ((size_t)blk * n + k) * n, *wi = (const T *)g.w_i + ((size_t)blk * n + k) * n;
+        float zr[ROWS], zi[ROWS];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) { zr[r] = 0.f; zi[r] = 0.f; }
+        if (vec) {
+#pragma unroll 2
+            for (int j = lane * V; j < n; j += 32 * V) {
+                float fr[V], fi[V];
+                unpack16<T>(*reinterpret_cast<const uint4 *>(wr + j), fr);
+                unpack16<T>(*reinterpret_cast<const uint4 *>(wi + j), fi);
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+                    for (int v = 0; v < V; v += 4) {
+                        const float4 x = *reinterpret_cast<const float4 *>(rows_u + (size_t)r * n + j + v);
+                        zr[r] = fmaf(fr[v + 3], x.w, fmaf(fr[v + 2], x.z, fmaf(fr[v + 1], x.y, fmaf(fr[v], x.x, zr[r]))));
+                        zi[r] = fmaf(fi[v + 3], x.w, fmaf(fi[v + 2], x.z, fmaf(fi[v + 1], x.y, fmaf(fi[v], x.x, zi[r]))));
+                    }
+            }
+        } else {
+            for (int j = lane; j < n; j += 32)
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) {
+                    zr[r] = fmaf(to_f32(wr[j]), rows_u[(size_t)r * n + j], zr[r]);
+                    zi[r] = fmaf(to_f32(wi[j]), rows_u[(size_t)r * n + j], zi[r]);
+                }
+        }
+        float mr = 0.f, mi = 0.f;       // lane r: row r's sums
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const float a = warp_sum(zr[r]), b = warp_sum(zi[r]);
+            if (lane == r) { mr = a; mi = b; }
+        }
+        if (lane < live) {
+            const int t = t0 + lane, c = blk * n + k;
+            float a, b;
+            gated_pair(mr + g.b_r[c], mi + g.b_i[c], g.rate[c], rows_u[(size_t)lane * n + k], &a, &b);
+            float *S = g.state + (size_t)g.slot_ids[t] * g.C + c;
+            const float s = fmaf(a, *S, b);
+            *S = s;
+            ((T *)g.out)[(size_t)t * g.C + c] = from_f32<T>(s * block_act(g.act, g.y[(size_t)t * g.ld_y + c] + (g.y_bias ? g.y_bias[c] : 0.f)));
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) gated_rows_kernel(GatedArgs g) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float rows_u[];     // [rows][n], rows 1, 2, 4 or 8
+    const int blk = blockIdx.y, t0 = blockIdx.z * GR_ROWS, live = min(GR_ROWS, g.T - t0), n = g.n;
+    const int rows = live <= 1 ? 1 : (live <= 2 ? 2 : (live <= 4 ? 4 : 8));
+    for (int i = threadIdx.x; i < rows * n; i += 256) {
+        const int r = i / n;
+        rows_u[i] = r < live ? g.u[(size_t)(t0 + r) * g.C + (size_t)blk * n + i - r * n] : 0.f;
+    }
+    __syncthreads();
+    const int c_first = blockIdx.x * GR_CHANNELS;
+    if (rows == 1) gated_rows_body<T, 1>(g, rows_u, t0, live, blk, c_first);
+    else if (rows == 2) gated_rows_body<T, 2>(g, rows_u, t0, live, blk, c_first);
+    else if (rows == 4) gated_rows_body<T, 4>(g, rows_u, t0, live, blk, c_first);
+    else gated_rows_body<T, 8>(g, rows_u, t0, live, blk, c_first);
+}
+
+// floats of scratch that a step of T rows with n_pieces pieces needs
+JK_EXPORT long long jk_gated_recurrence_scratch_floats(int T, int C, int n_pieces) { return 2LL * T * C + 2LL * n_pieces * C; }
+// kernels that a call launches
+JK_EXPORT int jk_gated_recurrence_launches(int T, int nreq, int n, int n_pieces) {
+    return T == nreq && T <= 64 && (size_t)n * GR_ROWS * 4 <= 200 * 1024 ? 1 : (n_pieces > 0 ? 3 : 2);
+}
+
+JK_EXPORT int jk_gated_recurrence(const float *u, const void *w_r, const void *w_i, const float *b_r, const float *b_i, const float *rate, const float *y,
+                                  int ld_y, const float *y_bias, int act, float *state, const int *req_start, const int *slot_ids, int nreq, void *out,
+                                  int dtype, int T, int C, int blocks, const int *direct, int n_direct, const int *pieces, int n_pieces,
+                                  const int *piece_reqs, int n_piece_reqs, float *scratch, long long scratch_floats, cudaStream_t stream) {
+    if (T == 0 || nreq == 0) return JK_OK;
+    JK_REQUIRE(u && w_r && w_i && b_r && b_i && rate && y && state && req_start && slot_ids && out, "gated_recurrence: an argument is missing");
+    JK_REQUIRE(C > 0 && blocks > 0 && C % blocks == 0 && blocks <= 65535, "gated_recurrence: %d channels in %d parts", C, blocks);
+    GatedArgs g{u, w_r, w_i, b_r, b_i, rate, y, ld_y, y_bias, act, state, req_start, slot_ids, out, T, C, blocks, C / blocks,
+                nullptr, nullptr, nullptr, nullptr, direct, pieces, piece_reqs, n_direct, n_pieces, n_piece_reqs};
+    if (jk_gated_recurrence_launches(T, nreq, g.n, n_pieces) == 1) {
+        const size_t smem = sizeof(float) * (size_t)(T <= 1 ? 1 : (T <= 2 ? 2 : (T <= 4 ? 4 : 8))) * g.n;
+        const dim3 grid((g.n + GR_CHANNELS - 1) / GR_CHANNELS, blocks, (T + GR_ROWS - 1) / GR_ROWS);
+#define LAUNCH(TT)                                                                                                                     \
+    do {                                                                                                                               \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(gated_rows_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+        jk_launch(gated_rows_kernel<TT>, grid, dim3(256), smem, stream, g);                                                            \
+    } while (0)
+        BLOCKS_BY_DTYPE(dtype, "gated_rows", LAUNCH);
+#undef LAUNCH
+        JK_CHECK_LAUNCH("gated_rows");
+        return JK_OK;
+    }
+    if (n_pieces == 0 && direct == nullptr && n_direct <= 0) g.n_direct = nreq;       // no lists: every request is one item
+    JK_REQUIRE(g.n_direct >= 0 && n_pieces >= 0 && g.n_direct + n_pieces > 0 && g.n_direct + n_pieces <= 65535, "gated_recurrence: %d and %d work items", n_direct, n_pieces);
+    JK_REQUIRE(n_pieces == 0 || (pieces && piece_reqs && n_piece_reqs > 0), "gated_recurrence: pieces without their lists");
+    JK_REQUIRE(scratch && scratch_floats >= jk_gated_recurrence_scratch_floats(T, C, n_pieces), "gated_recurrence: %lld floats of scratch are too few", scratch_floats);
+    g.a = scratch; g.b = g.a + (size_t)T * C; g.piece_end = g.b + (size_t)T * C; g.piece_prod = g.piece_end + (size_t)n_pieces * C;
+    const dim3 tiles((T + GT_M - 1) / GT_M, (g.n + GT_N - 1) / GT_N, blocks);
+    const int groups = (C + GS_THREADS - 1) / GS_THREADS;
+#define LAUNCH(TT)                                                                                                                   \
+    jk_launch(gated_pairs_kernel<TT>, tiles, dim3(256), 0, stream, g);                                                               \
+    jk_launch(gated_scan_kernel<TT>, dim3(groups, g.n_direct + n_pieces), dim3(GS_THREADS), 0, stream, g);                           \
+    if (n_pieces > 0) jk_launch(gated_finish_kernel<TT>, dim3(groups, n_pieces), dim3(GS_THREADS), 0, stream, g)
+    BLOCKS_BY_DTYPE(dtype, "gated_recurrence", LAUNCH);
+#undef LAUNCH
+    JK_CHECK_LAUNCH("gated_recurrence");
     return JK_OK;
 }

@@ -1011,7 +1011,7 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
 // or head by head with one weight of dv shared by the heads), times act(gate), into the activation type.
 //     out[t, c] = o[t, c] / sqrt(mean_scope(o^2) + eps) * w[c or c % dv] * act(u[t, g_off + c])
 // One block per row; a warp per head in the per-head forms (per_head 1: one weight of dv shared by the heads; 2: the mean
-// per head, a weight of heads * dv).
+// per head, a weight of heads * dv).  w null: no weight.
 // ---------------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ u, int ld, int g_off, const float *__restrict__ w,
@@ -1030,20 +1030,20 @@ __global__ void norm_gate_kernel(const float *__restrict__ o, const float *__res
             for (int e = lane; e < dv; e += 32) { const float x = orow[h * dv + e]; ss += x * x; }
             const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
             for (int e = lane; e < dv; e += 32)
-                dst[h * dv + e] = from_f32<T>(orow[h * dv + e] * inv * w[per_head == 2 ? h * dv + e : e] * apply_act(gate_act, grow[h * dv + e]));
+                dst[h * dv + e] = from_f32<T>(orow[h * dv + e] * inv * (w ? w[per_head == 2 ? h * dv + e : e] : 1.f) * apply_act(gate_act, grow[h * dv + e]));
         }
     } else {
         float ss = 0.f;
         for (int c = threadIdx.x; c < n; c += blockDim.x) { const float x = orow[c]; ss += x * x; }
         const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
-        for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = from_f32<T>(orow[c] * inv * w[c] * apply_act(gate_act, grow[c]));
+        for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = from_f32<T>(orow[c] * inv * (w ? w[c] : 1.f) * apply_act(gate_act, grow[c]));
     }
 }
 
 JK_EXPORT int jk_norm_gate(const float *o, const float *u, int ld, int g_off, const float *w, float eps, int heads, int dv,
                            int per_head, int gate_act, void *out, int dtype, int T, cudaStream_t stream) {
     if (T == 0) return JK_OK;
-    JK_REQUIRE(o && u && w && out && heads > 0 && dv > 0, "norm_gate: an argument is missing");
+    JK_REQUIRE(o && u && out && heads > 0 && dv > 0, "norm_gate: an argument is missing");
     const int n = heads * dv;
     const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);
     if (dtype == JK_F32)
@@ -1161,11 +1161,20 @@ JK_EXPORT int jk_token_shift(const void *h, const float *mu, float *last, const 
 
 // ---------------------------------------------------------------------------------------------------------------
 // An activation between two products of a feed-forward without a gate: out[t, c] = T(act(u[t, c])), u float32 rows `ld` apart.
+// With a table: times table[tokens[t], off + c] (rows of `ld` elements of type T), a vector of the row's own token.
 // ---------------------------------------------------------------------------------------------------------------
+struct ActTable {
+    const void *rows;           // null: no factor
+    const int *tokens;
+    long long ld;
+    int off;
+};
+
 template <typename T>
-__global__ void act_rows_kernel(const float *__restrict__ u, int ld, T *__restrict__ out, int n, size_t total, int act, int vec) {
+__global__ void act_rows_kernel(const float *__restrict__ u, int ld, T *__restrict__ out, int n, size_t total, int act, int vec, ActTable table) {
     pdl_trigger();
     pdl_wait();
+    const T *rows = (const T *)table.rows;
     if (vec) {          // four neighbouring columns of a row at a time (n and ld multiples of four, both bases aligned)
         const size_t quads = total / 4;
         const int per_row = n / 4;
@@ -1173,8 +1182,13 @@ __global__ void act_rows_kernel(const float *__restrict__ u, int ld, T *__restri
             const size_t t = i / per_row;
             const int c = (int)(i - t * per_row) * 4;
             const float4 x = *reinterpret_cast<const float4 *>(u + t * ld + c);
-            __align__(16) T o[4] = {from_f32<T>(apply_act(act, x.x)), from_f32<T>(apply_act(act, x.y)), from_f32<T>(apply_act(act, x.z)),
-                      from_f32<T>(apply_act(act, x.w))};
+            float y[4] = {apply_act(act, x.x), apply_act(act, x.y), apply_act(act, x.z), apply_act(act, x.w)};
+            if (rows != nullptr) {
+                const T *e = rows + (size_t)table.tokens[t] * table.ld + table.off + c;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) y[k] *= to_f32(e[k]);
+            }
+            __align__(16) T o[4] = {from_f32<T>(y[0]), from_f32<T>(y[1]), from_f32<T>(y[2]), from_f32<T>(y[3])};
             if (sizeof(T) == 2) *reinterpret_cast<uint2 *>(out + t * n + c) = *reinterpret_cast<const uint2 *>(o);
             else *reinterpret_cast<uint4 *>(out + t * n + c) = *reinterpret_cast<const uint4 *>(o);
         }
@@ -1183,23 +1197,73 @@ __global__ void act_rows_kernel(const float *__restrict__ u, int ld, T *__restri
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / n;
         const int c = (int)(i - t * n);
-        out[i] = from_f32<T>(apply_act(act, u[t * ld + c]));
+        const float e = rows != nullptr ? to_f32(rows[(size_t)table.tokens[t] * table.ld + table.off + c]) : 1.f;
+        out[i] = from_f32<T>(apply_act(act, u[t * ld + c]) * e);
     }
 }
 
-JK_EXPORT int jk_act_rows(const float *u, int ld, void *out, int dtype, int T, int n, int act, cudaStream_t stream) {
+// `table` (may be null): rows of `table_ld` elements of the activation type, one per token id; columns off .. off + n multiply the row
+JK_EXPORT int jk_act_rows(const float *u, int ld, void *out, int dtype, int T, int n, int act, const void *table, long long table_ld, int off,
+                          const int *tokens, cudaStream_t stream) {
     if (T == 0) return JK_OK;
     JK_REQUIRE(u && out && n > 0 && ld >= n, "act_rows: an argument is missing");
+    JK_REQUIRE(table == nullptr || (tokens && off >= 0 && off + n <= table_ld), "act_rows: columns %d .. %d of a table of %lld", off, off + n, table_ld);
     const size_t total = (size_t)T * n;
     const int vec = n % 4 == 0 && ld % 4 == 0 && (uintptr_t)u % 16 == 0 && (uintptr_t)out % 16 == 0;
     const int blocks = (int)std::min<size_t>(((vec ? total / 4 : total) + 255) / 256, 148 * 16);
+    const ActTable tab{table, tokens, table_ld, off};
     if (dtype == JK_F32)
-        jk_launch(act_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, u, ld, (float *)out, n, total, act, vec);
+        jk_launch(act_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, u, ld, (float *)out, n, total, act, vec, tab);
     else if (dtype == JK_BF16)
-        jk_launch(act_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, u, ld, (__nv_bfloat16 *)out, n, total, act, vec);
+        jk_launch(act_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, u, ld, (__nv_bfloat16 *)out, n, total, act, vec, tab);
     else
         JK_FAIL(JK_UNSUPPORTED, "act_rows: dtype %d", dtype);
     JK_CHECK_LAUNCH("act_rows");
+    return JK_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Rotation of queries and keys that lie in float32 rows u [T, ld], in place: the first `rot_dims` elements of each of `heads`
+// heads of dk at column q_off, and of as many at k_off (< 0: none), in pairs by the angle positions[t] * freq[i], formed in float32:
+// (a, b) -> (a cos - b sin, b cos + a sin), cos and sin times `mag`.  half: element i pairs with i + rot_dims / 2, else 2i with
+// 2i + 1.  One block per row; a row's angles are formed once for all heads.
+// ---------------------------------------------------------------------------------------------------------------
+__global__ void rotate_rows_kernel(float *__restrict__ u, int ld, int q_off, int k_off, int heads, int dk, const float *__restrict__ freq,
+                                   int rot_dims, int half_layout, float mag, const int *__restrict__ positions) {
+    extern __shared__ float2 angle[];       // [rot_dims / 2] (cos, sin)
+    pdl_trigger();
+    pdl_wait();
+    const int pairs = rot_dims >> 1, t = blockIdx.x;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+        float sn, cs;
+        sincosf(pos * freq[i], &sn, &cs);
+        angle[i] = make_float2(cs * mag, sn * mag);
+    }
+    __syncthreads();
+    float *row = u + (size_t)t * ld;
+    const int each = heads * pairs, total = k_off < 0 ? each : 2 * each;
+    for (int j = threadIdx.x; j < total; j += blockDim.x) {
+        const int jj = j < each ? j : j - each, h = jj / pairs, i = jj - h * pairs;
+        float *head = row + (j < each ? q_off : k_off) + h * dk;
+        float *pa = head + (half_layout ? i : 2 * i), *pb = head + (half_layout ? i + pairs : 2 * i + 1);
+        const float2 cs = angle[i];
+        const float a = *pa, b = *pb;
+        *pa = a * cs.x - b * cs.y;
+        *pb = b * cs.x + a * cs.y;
+    }
+}
+
+JK_EXPORT int jk_rotate_rows(float *u, int ld, int q_off, int k_off, int heads, int dk, const float *freq, int rot_dims, int half_layout, float mag,
+                             const int *positions, int T, cudaStream_t stream) {
+    if (T == 0 || rot_dims == 0) return JK_OK;
+    JK_REQUIRE(u && freq && positions && heads > 0 && dk > 0 && q_off >= 0, "rotate_rows: an argument is missing");
+    JK_REQUIRE(rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= dk && rot_dims <= 8192, "rotate_rows: rotation of %d of %d elements", rot_dims, dk);
+    JK_REQUIRE(q_off + heads * dk <= ld && (k_off < 0 || k_off + heads * dk <= ld), "rotate_rows: %d heads of %d beyond rows of %d", heads, dk, ld);
+    const int work = heads * rot_dims, threads = std::min(T <= 64 ? 1024 : 256, std::max(64, (work + 31) / 32 * 32));
+    jk_launch(rotate_rows_kernel, dim3(T), dim3(threads), sizeof(float2) * (size_t)(rot_dims / 2), stream, u, ld, q_off, k_off, heads, dk, freq, rot_dims,
+              half_layout, mag > 0.f ? mag : 1.f, positions);
+    JK_CHECK_LAUNCH("rotate_rows");
     return JK_OK;
 }
 

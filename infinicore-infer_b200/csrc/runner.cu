@@ -538,7 +538,10 @@ int run_norm_add(Run &r, const RunnerOp &op) {
     if (op.out_slot >= 0)
         if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &h, "the next sublayer's input")) return rc;
     JK_REQUIRE(!r.pending, "runner: a norm over a sublayer's output while another product waits to be added");
-    RUN(blocks, g_fns.norm_add((const float *)delta, r.x(), op.vec, op.eps, op.vec2, op.eps2, h, r.env.dtype, T, op.n, r.stream));
+    void *h2 = nullptr;
+    if (op.out2_slot >= 0)
+        if (int rc = r.slot(op.out2_slot, (long long)r.elem() * T * op.n, &h2, "the input of the sublayer beside the next")) return rc;
+    RUN(blocks, g_fns.norm_add((const float *)delta, r.x(), op.vec, op.eps, op.vec2, op.eps2, h, op.vec3, h2, r.env.dtype, T, op.n, r.stream));
     return JK_OK;
 }
 
@@ -637,8 +640,8 @@ int run_causal_conv(Run &r, const RunnerOp &op) {
         if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &yT, "a convolution's output")) return rc;
     JK_REQUIRE(r.st.slot_ids != nullptr || op.taps <= 1, "runner: a convolution keeps tails, but the step names no state slots");
     RUN(blocks, g_fns.causal_conv((const float *)u, op.ld, op.q_off, op.n, op.conv_q, op.bias, op.taps, op.act, op.state, r.st.row_req,
-                                  r.st.req_start, r.st.slot_ids, (float *)y32, yT, r.env.dtype, T, r.st.nreq, r.stream));
-    if (op.taps > 1) ++g_launches;
+                                  r.st.req_start, r.st.slot_ids, (float *)y32, yT, r.env.dtype, T, r.st.nreq, op.in_bias, r.stream));
+    if (op.taps > 1 && T > r.st.nreq) ++g_launches;
     return JK_OK;
 }
 
@@ -671,7 +674,8 @@ int run_experts(Run &r, const RunnerOp &op) {
     JK_REQUIRE(!r.pending || (adds && !op.add), "runner: routed experts while another product waits to be added");
     RUN(blocks, g_fns.routed_experts(h, op.vec, op.w, op.w3, (float *)delta, op.add, r.env.dtype, T, op.n, op.ff, op.experts, op.top, op.act,
                                      (int *)route, act, (float *)y, op.score_form, op.limit, op.router_bias, op.gate_w, op.identity, op.group_count, op.group_keep,
-                                   op.correction, adds ? r.x() : nullptr, op.scale, r.pending ? (const float *)delta : nullptr, r.pending_scale, r.stream));
+                                   op.correction, adds ? r.x() : nullptr, op.scale, r.pending ? (const float *)delta : nullptr, r.pending_scale,
+                                   op.score_scale > 0.f ? op.score_scale : 1.f, r.stream));
     g_launches += g_fns.routed_experts_launches() - 1;
     if (adds) {
         r.pending = false;
@@ -715,7 +719,7 @@ int run_activate(Run &r, const RunnerOp &op) {
     void *u, *out;
     if (int rc = r.slot(op.in_slot, 4LL * T * ld, &u, "an activation's input")) return rc;
     if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &out, "an activation's output")) return rc;
-    RUN(mixers, g_fns.act_rows((const float *)u, ld, out, r.env.dtype, T, op.n, op.act, r.stream));
+    RUN(mixers, g_fns.act_rows((const float *)u, ld, out, r.env.dtype, T, op.n, op.act, op.w, op.k, op.g_off, r.st.tokens, r.stream));
     return JK_OK;
 }
 
@@ -750,6 +754,66 @@ int run_delta_rule(Run &r, const RunnerOp &op) {
     ++g_launches;       // the rows' preparation
     RUN(mixers, g_fns.norm_gate((const float *)mix, (const float *)u, op.r_off, op.g_off, op.vec, op.eps, op.heads, dv, op.per_head_norm,
                                 op.gate_act, out, r.env.dtype, T, r.stream));
+    return JK_OK;
+}
+
+int run_embed_pair(Run &r, const RunnerOp &op) {
+    JK_REQUIRE(g_fns.embed_pair != nullptr, "runner: an embedding with pairs or a norm needs the blocks module, which was not bound");
+    void *out;
+    if (int rc = r.slot(op.out_slot, 4LL * r.st.ntok * op.n, &out, "the embedding")) return rc;
+    JK_REQUIRE(op.w3 == nullptr || (r.st.slot_ids != nullptr && op.state != nullptr), "runner: pairs of tokens without the requests' last tokens");
+    RUN(blocks, g_fns.embed_pair(r.st.tokens, r.st.positions, r.st.row_req, r.st.req_start, r.st.req_pos, r.st.slot_ids, op.w, op.w3, op.w_dtype,
+                                 op.buckets, op.mul_prev, op.mul_cur, op.scale, (int *)op.state, op.vec, op.eps, (float *)out, r.st.ntok, op.n, r.stream));
+    return JK_OK;
+}
+
+int run_join(Run &r, const RunnerOp &op) {
+    JK_REQUIRE(g_fns.join_parts != nullptr, "runner: joining sublayers' outputs needs the blocks module, which was not bound");
+    const int T = r.st.ntok;
+    void *p1, *p2 = nullptr, *p3 = nullptr, *h = nullptr;
+    if (int rc = r.slot(op.in_slot, 4LL * T * op.n, &p1, "a sublayer's output")) return rc;
+    if (op.in2_slot >= 0)
+        if (int rc = r.slot(op.in2_slot, 4LL * T * op.n, &p2, "a second sublayer's output")) return rc;
+    if (op.add) {
+        if (int rc = r.slot(SLOT_DELTA, 4LL * T * op.n, &p3, "a third sublayer's output")) return rc;
+        JK_REQUIRE(!r.pending, "runner: sublayers' outputs join while another product waits to be added");
+    } else if (int rc = flush_pending(r, T, op.n)) {
+        return rc;
+    }
+    if (op.out_slot >= 0)
+        if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &h, "the stream as activations")) return rc;
+    RUN(blocks, g_fns.join_parts(r.x(), (const float *)p1, op.vec, op.eps, (const float *)p2, op.vec2, op.eps2, (const float *)p3, h, r.env.dtype, T,
+                                 op.n, r.stream));
+    return JK_OK;
+}
+
+int run_rotate(Run &r, const RunnerOp &op) {
+    JK_REQUIRE(g_fns.rotate_rows != nullptr, "runner: a rotation in place needs the mixers module, which was not bound");
+    void *u;
+    if (int rc = r.slot(op.in_slot, 4LL * r.st.ntok * op.ld, &u, "the rows of a rotation")) return rc;
+    RUN(mixers, g_fns.rotate_rows((float *)u, op.ld, op.q_off, op.k_off, op.heads, op.head_dim, op.freq, op.rot_dims, op.rot_half, op.rot_mag,
+                                  r.st.positions, r.st.ntok, r.stream));
+    return JK_OK;
+}
+
+int run_gated_recurrence(Run &r, const RunnerOp &op) {
+    JK_REQUIRE(g_fns.gated_recurrence != nullptr, "runner: a gated recurrence needs the blocks module, which was not bound");
+    const int T = r.st.ntok, n_pieces = r.st.list_n[op.list_tiles];
+    void *u, *y, *out, *scratch = nullptr;
+    if (int rc = r.slot(op.in_slot, 4LL * T * op.n, &u, "a recurrence's input")) return rc;
+    if (int rc = r.slot(SLOT_TMP, 4LL * T * op.ld, &y, "the projection that holds a recurrence's branch")) return rc;
+    if (int rc = r.slot(op.out_slot, (long long)r.elem() * T * op.n, &out, "a recurrence's output")) return rc;
+    JK_REQUIRE(r.st.slot_ids != nullptr && op.state != nullptr, "runner: a recurrence without its state slots");
+    JK_REQUIRE(op.blocks > 0, "runner: a recurrence in %d parts", op.blocks);
+    const int launches = g_fns.gated_recurrence_launches(T, r.st.nreq, op.n / op.blocks, n_pieces);
+    const long long floats = launches > 1 ? g_fns.gated_recurrence_scratch(T, op.n, n_pieces) : 0;
+    if (floats > 0)
+        if (int rc = r.slot(SLOT_SCAN, 4 * floats, &scratch, "a recurrence's pairs and pieces")) return rc;
+    RUN(blocks, g_fns.gated_recurrence((const float *)u, op.w, op.w3, op.b1, op.b2, op.decay, (const float *)y + op.g_off, op.ld, op.bias, op.act,
+                                       op.state, r.st.req_start, r.st.slot_ids, r.st.nreq, out, r.env.dtype, T, op.n, op.blocks,
+                                       r.st.lists[op.list_short], r.st.list_n[op.list_short], r.st.lists[op.list_tiles], n_pieces,
+                                       r.st.lists[op.list_aux], r.st.list_n[op.list_aux], (float *)scratch, floats, r.stream));
+    g_launches += launches - 1;
     return JK_OK;
 }
 
@@ -871,6 +935,16 @@ JK_EXPORT int jk_runner_run(const RunnerEnv *envp, const RunnerOp *ops, int firs
                 hidden = op.n;
                 rc = run_norm_pair(r, op);
                 break;
+            case OP_EMBED_PAIR:
+                hidden = op.n;
+                rc = run_embed_pair(r, op);
+                break;
+            case OP_JOIN:
+                hidden = op.n;
+                rc = run_join(r, op);
+                break;
+            case OP_ROTATE: rc = run_rotate(r, op); break;
+            case OP_GATED_RECURRENCE: rc = run_gated_recurrence(r, op); break;
             default:
                 JK_FAIL(JK_BAD_ARGUMENT, "runner_run: record %d has kind %d", i, op.kind);
         }
@@ -939,6 +1013,7 @@ JK_EXPORT int jk_runner_slot_bytes(const RunnerEnv *env, const RunnerOp *ops, in
             case OP_NORM_ADD:
                 need(SLOT_X, 4LL * max_rows * op.n); need(op.in_slot, 4 * rows * op.n);
                 if (op.out_slot >= 0) need(op.out_slot, e * rows * op.n);
+                if (op.out2_slot >= 0) need(op.out2_slot, e * rows * op.n);
                 break;
             case OP_REINJECT: need(SLOT_X, 4 * rows * op.n); need(op.in_slot, 4 * rows * op.n); need(SLOT_ACT, e * rows * op.k); break;
             case OP_LATENT_QKV:
@@ -986,6 +1061,18 @@ JK_EXPORT int jk_runner_slot_bytes(const RunnerEnv *env, const RunnerOp *ops, in
                 need(op.out_slot, e * rows * width);
                 break;
             }
+            case OP_EMBED_PAIR: need(op.out_slot, 4 * rows * op.n); break;
+            case OP_JOIN:
+                need(SLOT_X, 4 * rows * op.n); need(op.in_slot, 4 * rows * op.n);
+                if (op.in2_slot >= 0) need(op.in2_slot, 4 * rows * op.n);
+                if (op.add) need(SLOT_DELTA, 4 * rows * op.n);
+                if (op.out_slot >= 0) need(op.out_slot, e * rows * op.n);
+                break;
+            case OP_ROTATE: need(op.in_slot, 4 * rows * op.ld); break;
+            case OP_GATED_RECURRENCE:
+                need(op.in_slot, 4 * rows * op.n); need(SLOT_TMP, 4 * rows * op.ld); need(op.out_slot, e * rows * op.n);
+                need(SLOT_SCAN, 4 * 2 * op.n * (rows + jk::scan_max_pieces(rows)));
+                break;
             default: JK_FAIL(JK_BAD_ARGUMENT, "runner_slot_bytes: record %d has kind %d", i, op.kind);
         }
     }

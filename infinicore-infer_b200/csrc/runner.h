@@ -63,9 +63,10 @@ typedef int (*LinearScanFn)(const float *, int, int, int, int, int, int, int, in
 typedef int (*NormGateFn)(const float *, const float *, int, int, const float *, float, int, int, int, int, void *, int, int, cudaStream_t);
 typedef int (*TokenShiftFn)(const void *, const float *, float *, const int *, const int *, const int *, void *, int, int, int, int, int,
                             cudaStream_t);
-typedef int (*ActRowsFn)(const float *, int, void *, int, int, int, int, cudaStream_t);
+typedef int (*ActRowsFn)(const float *, int, void *, int, int, int, int, const void *, long long, int, const int *, cudaStream_t);
+typedef int (*RotateRowsFn)(float *, int, int, int, int, int, const float *, int, int, float, const int *, int, cudaStream_t);
 // csrc/blocks.cu
-typedef int (*NormAddFn)(const float *, float *, const float *, float, const float *, float, void *, int, int, int, cudaStream_t);
+typedef int (*NormAddFn)(const float *, float *, const float *, float, const float *, float, void *, const float *, void *, int, int, int, cudaStream_t);
 typedef int (*ConcatCastFn)(const float *, const float *, void *, int, int, int, cudaStream_t);
 typedef int (*AddBiasRowsFn)(float *, const float *, int, int, cudaStream_t);
 typedef int (*LatentQkvFn)(const float *, int, int, int, int, int, int, int, int, const float *, float, const float *, float, const int *,
@@ -75,13 +76,13 @@ typedef int (*LatentAttentionFn)(const void *, const void *, void *, float *, in
                                  int, int, int, float, int, const int *, int, int, const float *, cudaStream_t);
 typedef long long (*LatentScratchFn)(int, int, int, int);
 typedef int (*CausalConvFn)(const float *, int, int, int, const float *, const float *, int, int, float *, const int *, const int *,
-                            const int *, float *, void *, int, int, int, cudaStream_t);
+                            const int *, float *, void *, int, int, int, const float *, cudaStream_t);
 typedef int (*SelectiveScanFn)(const float *, const float *, int, int, int, int, const float *, int, const void *, const float *,
                                const float *, const float *, float *, const int *, const int *, int, void *, int, float *, int, int,
                                cudaStream_t);
 typedef int (*RoutedExpertsFn)(const void *, const float *, const void *, const void *, float *, int, int, int, int, int, int, int, int,
                                int *, void *, float *, int, float, const float *, const float *, int, int, int, const float *, float *, float,
-                               const float *, float, cudaStream_t);
+                               const float *, float, float, cudaStream_t);
 typedef long long (*RoutedWorkspaceFn)(int, int, int);
 typedef int (*CountFn)();
 typedef int (*SoftcapFn)(float *, float, long long, cudaStream_t);
@@ -92,6 +93,16 @@ typedef int (*NormPairFn)(const float *, const float *, const float *, float, co
 typedef int (*DeltaRuleFn)(const float *, int, int, int, int, const float *, int, int, int, const float *, const float *, int, int, int, int,
                            float, float, float *, const int *, const int *, int, float *, float *, int, cudaStream_t);
 typedef long long (*DeltaScratchFn)(int, int, int, int);
+// csrc/blocks.cu
+typedef int (*EmbedPairFn)(const int *, const int *, const int *, const int *, const int *, const int *, const void *, const void *, int, int, int,
+                           int, float, int *, const float *, float, float *, int, int, cudaStream_t);
+typedef int (*JoinPartsFn)(float *, const float *, const float *, float, const float *, const float *, float, const float *, void *, int, int, int,
+                           cudaStream_t);
+typedef int (*GatedRecurrenceFn)(const float *, const void *, const void *, const float *, const float *, const float *, const float *, int,
+                                 const float *, int, float *, const int *, const int *, int, void *, int, int, int, int, const int *, int,
+                                 const int *, int, const int *, int, float *, long long, cudaStream_t);
+typedef long long (*GatedScratchFn)(int, int, int);
+typedef int (*GatedLaunchesFn)(int, int, int, int);
 typedef int (*ArgmaxFn)(const float *, long long, int, int, int *, void *, cudaStream_t);
 typedef int (*SampleFn)(const float *, long long, int, int, const float *, const int *, const float *, const float *, int *,
                         cudaStream_t);
@@ -162,6 +173,13 @@ struct RunnerFns {
     DeltaRuleFn delta_rule;
     DeltaScratchFn delta_rule_scratch;
     NormPairFn norm_pair;           // csrc/blocks.cu, bound with that module
+    // csrc/blocks.cu, and the rotation of csrc/mixers.cu; bound with their modules
+    EmbedPairFn embed_pair;
+    JoinPartsFn join_parts;
+    GatedRecurrenceFn gated_recurrence;
+    GatedScratchFn gated_recurrence_scratch;
+    GatedLaunchesFn gated_recurrence_launches;
+    RotateRowsFn rotate_rows;
 };
 
 // ---- records ---------------------------------------------------------------------------------------------------
@@ -185,6 +203,8 @@ enum RunnerSlot {
     SLOT_ROUTE,         // int32 and float32: which experts each row chose, and the rows of each expert
     SLOT_SHIFT,         // activations [parts, T, width]: a row mixed with the row before it, once per projection that reads one
     SLOT_H2,            // activations [T, hidden]: a second norm's output, for a sublayer beside the one that reads SLOT_H
+    SLOT_PART1,         // float32 [T, hidden]: the outputs of mixers side by side, which a norm of their own or another sublayer's
+    SLOT_PART2,         // output still has to meet before they join the stream
     RUNNER_SLOTS
 };
 
@@ -231,6 +251,12 @@ enum RunnerOpKind {
     OP_NORM_PAIR,       // two norms of the same stream: out2 = rmsnorm(stream) * vec2 (out2_slot < 0: not made), and out = h_t + (h_(t-1) -
                         // h_t) * bias with h = rmsnorm(stream) * vec; the row before a portion's first row is kept in state (csrc/blocks.cu)
                         // (bias null: out = h, no state)
+    OP_EMBED_PAIR,      // out = rmsnorm(scale * w[token] + w3[row of (previous token, token)]) * vec (vec null: no norm; w3 null: no pairs)
+    OP_JOIN,            // stream += rmsnorm(in) * vec + rmsnorm(in2) * vec2 (vec, vec2 null: unnormed; in2 < 0: absent) + SLOT_DELTA (add);
+                        // out = activations(stream) if out_slot >= 0
+    OP_ROTATE,          // in place: in's float32 rows `ld` apart, the first rot_dims elements of `heads` heads of head_dim at q_off and k_off
+    OP_GATED_RECURRENCE,// in: float32 [T, n]; gates sigmoid(w in + b1), sigmoid(w3 in + b2) of block-diagonal maps, S = a S + sqrt(1 - a^2) i in
+                        // per channel over each request's rows and its state slot; out = S * act(SLOT_TMP[t, g_off + c] + bias[c])
 };
 
 enum RunnerAct { RUNNER_ACT_NONE = 0, RUNNER_ACT_SILU = 1, RUNNER_ACT_GELU_TANH = 2, RUNNER_ACT_SIGMOID = 3, RUNNER_ACT_RELU = 4,
@@ -329,6 +355,15 @@ struct RunnerOp {
     const float *sink_w;        // ATTENTION, LATENT_ATTENTION: [heads] the sinks' scores (null: 0; LATENT_ATTENTION: no sink)
     const float *temp;          // CONV_QKV: [heads] head h's queries are multiplied by temp[h] after everything else, or null
     const float *correction;    // EXPERTS: [experts + identity] added to the scores for the choice only, or null
+    // ---- what pairs of tokens, joined parts, real-gated recurrences and a token's own vectors add ------------------------------------
+    int buckets, mul_prev, mul_cur;     // EMBED_PAIR: row (previous * mul_prev + token * mul_cur) mod buckets of w3 [buckets + 1, n]
+    int blocks;                 // GATED_RECURRENCE: parts of the block-diagonal maps
+    float score_scale;          // EXPERTS: factor of the renormalised scores of score_form 1 (0 stands for 1)
+    const float *vec3;          // NORM_ADD: a third weight: out2 = rmsnorm(stream) * vec3 beside out
+    const float *in_bias;       // CAUSAL_CONV: [n] added to the input's rows
+    const float *b1;            // GATED_RECURRENCE: [n] bias of the first gate
+    // ACTIVATE: w (null: none) [tokens, k]: times w[token, g_off + c].  GATED_RECURRENCE: decay = [n] log a per unit of the first gate.
+    // EMBED_PAIR: state = int32 [slots, 2, 2].  LINEAR_ATTENTION: vec may be null (no weight).
     // ATTENTION: gated 2: a gate per output element, sigmoid(SLOT_TMP[t, g_off + h dv + e]).  HEAD_LINEAR: gated 2: a gate per head.
     // LATENT_QKV: k_off < 0 makes the heads' queries only, from rows [heads, head_dim + rot_width] at q_off (no cache row, no latent).
     // EXPERTS: score_form 2: softmax over all router outputs, the chosen scores as they are, multiplying the units' outputs;

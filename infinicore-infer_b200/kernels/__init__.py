@@ -676,11 +676,11 @@ def linear_scan(u: torch.Tensor, offsets, heads: int, dk: int, dv: int, qkv_act:
     return out
 
 
-def norm_gate(o: torch.Tensor, u: torch.Tensor, g_off: int, weight: torch.Tensor, eps: float, heads: int, dv: int, per_head,
+def norm_gate(o: torch.Tensor, u: torch.Tensor, g_off: int, weight: Optional[torch.Tensor], eps: float, heads: int, dv: int, per_head,
               gate_act: int, out: torch.Tensor) -> torch.Tensor:
     """out = rmsnorm(o) * weight * act(u[:, g_off : g_off + heads * dv]); the norm over all heads or head by head (``per_head``
-    2: head by head with a weight for every element of every head)."""
-    _need(o, "o", torch.float32); _need(u, "u", torch.float32); _need(weight, "weight", torch.float32); _need(out, "out")
+    2: head by head with a weight for every element of every head; ``weight`` None: none)."""
+    _need(o, "o", torch.float32); _need(u, "u", torch.float32); _need(out, "out")
     lib = _build.load("mixers")
     _check("mixers", lib.jk_norm_gate(_ptr(o), _ptr(u), _c_int(u.shape[1]), _c_int(g_off), _ptr(weight), _c_float(eps), _c_int(heads),
                                       _c_int(dv), _c_int(int(per_head)), _c_int(gate_act), _ptr(out), _c_int(dtype_code(out.dtype)),
@@ -699,13 +699,28 @@ def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, row_req, 
     return out
 
 
-def act_rows(u: torch.Tensor, out: torch.Tensor, act: int) -> torch.Tensor:
-    """out = act(u) in the type of ``out``; ``u`` float32 rows (a view of wider rows is fine)."""
+def act_rows(u: torch.Tensor, out: torch.Tensor, act: int, table: Optional[torch.Tensor] = None, table_off: int = 0,
+             tokens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out = act(u) in the type of ``out``; ``u`` float32 rows (a view of wider rows is fine).  With ``table`` (of ``out``'s type, a
+    row per token id): times table[tokens[t], table_off : table_off + n]."""
     _need(u, "u", torch.float32, contiguous=False); _need(out, "out")
     lib = _build.load("mixers")
     _check("mixers", lib.jk_act_rows(_ptr(u), _c_int(u.stride(0)), _ptr(out), _c_int(dtype_code(out.dtype)), _c_int(out.shape[0]),
-                                     _c_int(out.shape[1]), _c_int(act), _stream()))
+                                     _c_int(out.shape[1]), _c_int(act), _ptr(table), _c_ll(table.shape[1] if table is not None else 0),
+                                     _c_int(table_off), _ptr(tokens), _stream()))
     return out
+
+
+def rotate_rows(u: torch.Tensor, q_off: int, k_off: int, heads: int, dk: int, freq: torch.Tensor, positions: torch.Tensor, half: bool = True,
+                magnitude: float = 1.0) -> torch.Tensor:
+    """Rotate, in place, the first 2 * len(freq) elements of ``heads`` heads of ``dk`` at column ``q_off`` of the float32 rows ``u`` and
+    of as many at ``k_off`` (< 0: none) by positions * freq."""
+    _need(u, "u", torch.float32); _need(freq, "freq", torch.float32)
+    lib = _build.load("mixers")
+    _check("mixers", lib.jk_rotate_rows(_ptr(u), _c_int(u.shape[1]), _c_int(q_off), _c_int(k_off), _c_int(heads), _c_int(dk), _ptr(freq),
+                                        _c_int(2 * freq.numel()), _c_int(1 if half else 0), _c_float(magnitude), _ptr(positions), _c_int(u.shape[0]),
+                                        _stream()))
+    return u
 
 
 # ---- csrc/blocks.cu ---------------------------------------------------------------------------------------------------
@@ -713,13 +728,15 @@ ACT_RELU, ACT_GELU_ERF, ACT_SWISH_CLAMP, ACT_TANH = 4, 5, 6, 7
 
 
 def norm_add(delta: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: float, next_weight: Optional[torch.Tensor] = None,
-             next_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x += rmsnorm(delta) * weight; with ``out``: out = rmsnorm(x) * next_weight (or x itself) in out's type."""
+             next_eps: float = 0.0, out: Optional[torch.Tensor] = None, next_weight2: Optional[torch.Tensor] = None,
+             out2: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += rmsnorm(delta) * weight; with ``out``: out = rmsnorm(x) * next_weight (or x itself) in out's type; with ``out2``: the same
+    with next_weight2."""
     _need(delta, "delta", torch.float32); _need(x, "x", torch.float32); _need(weight, "weight", torch.float32)
     rows, d = x.shape
     lib = _build.load("blocks")
     _check("blocks", lib.jk_norm_add(_ptr(delta), _ptr(x), _ptr(weight), _c_float(eps), _ptr(next_weight), _c_float(next_eps), _ptr(out),
-                                     _c_int(dtype_code(out.dtype) if out is not None else F32), _c_int(rows), _c_int(d), _stream()))
+                                     _ptr(next_weight2), _ptr(out2), _c_int(dtype_code(out.dtype) if out is not None else F32), _c_int(rows), _c_int(d), _stream()))
     return x
 
 
@@ -790,14 +807,15 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, po
 
 
 def causal_conv(u: torch.Tensor, off: int, channels: int, taps: torch.Tensor, bias: Optional[torch.Tensor], act: int,
-                tail: Optional[torch.Tensor], row_req, req_start, slot_ids, y32: Optional[torch.Tensor], yT: Optional[torch.Tensor]) -> None:
-    """y = act(bias + taps over time of u[:, off : off + channels]); the tails ``[slots, taps - 1, channels]`` move forward."""
+                tail: Optional[torch.Tensor], row_req, req_start, slot_ids, y32: Optional[torch.Tensor], yT: Optional[torch.Tensor],
+                in_bias: Optional[torch.Tensor] = None) -> None:
+    """y = act(bias + taps over time of u[:, off : off + channels] (+ in_bias)); the tails ``[slots, taps - 1, channels]`` move forward."""
     _need(u, "u", torch.float32); _need(taps, "taps", torch.float32)
     lib = _build.load("blocks")
     _check("blocks", lib.jk_causal_conv(_ptr(u), _c_int(u.shape[1]), _c_int(off), _c_int(channels), _ptr(taps), _ptr(bias), _c_int(taps.shape[1]),
                                         _c_int(act), _ptr(tail), _ptr(row_req), _ptr(req_start), _ptr(slot_ids), _ptr(y32), _ptr(yT),
                                         _c_int(dtype_code(yT.dtype) if yT is not None else F32), _c_int(u.shape[0]),
-                                        _c_int(req_start.numel() - 1), _stream()))
+                                        _c_int(req_start.numel() - 1), _ptr(in_bias), _stream()))
 
 
 def selective_scan(x: torch.Tensor, low: torch.Tensor, dt_rank: int, states: int, z: torch.Tensor, z_ld: int, w_dt, dt_bias, A, skip,
@@ -820,7 +838,7 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
                    experts: int, top: int, act: int, score_form: int = 0, limit: float = 0.0, router_bias: Optional[torch.Tensor] = None,
                    gate_w: Optional[torch.Tensor] = None, identity: int = 0, groups=(0, 0), correction: Optional[torch.Tensor] = None,
                    x: Optional[torch.Tensor] = None, x_scale: float = 1.0, pending: Optional[torch.Tensor] = None,
-                   pending_scale: float = 1.0) -> torch.Tensor:
+                   pending_scale: float = 1.0, score_scale: float = 1.0) -> torch.Tensor:
     """delta (+)= sum over each row's ``top`` experts of largest sigmoid(router h) of expert(score * h); ``w_gate_up``
     ``[experts * 2 ff, d]`` (an expert's gate rows, then its up rows), ``w_down [experts * d, ff]``.  ``identity``, ``groups``,
     ``correction``: see csrc/blocks.cu (score_form 2).  With ``x`` (float32 ``[T, d]``) the sum goes there instead:
@@ -837,7 +855,7 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
                                            _c_int(dtype_code(h.dtype)), _c_int(T), _c_int(d), _c_int(ff), _c_int(experts), _c_int(top),
                                            _c_int(act), _ptr(route), _ptr(act_buf), _ptr(y), _c_int(score_form), _c_float(limit), _ptr(router_bias), _ptr(gate_w),
                                            _c_int(identity), _c_int(groups[0]), _c_int(groups[1]), _ptr(correction), _ptr(x), _c_float(x_scale),
-                                           _ptr(pending), _c_float(pending_scale), _stream()))
+                                           _ptr(pending), _c_float(pending_scale), _c_float(score_scale), _stream()))
     return delta
 
 
@@ -908,4 +926,49 @@ def delta_rule(c: torch.Tensor, offsets, u: torch.Tensor, b_off: int, a_off: int
                                        _c_int(u.shape[1]), _c_int(b_off), _c_int(a_off), _ptr(a_log), _ptr(dt_bias), _c_int(heads), _c_int(groups),
                                        _c_int(dk), _c_int(dv), _c_float(q_scale), _c_float(unit_eps), _ptr(state), _ptr(req_start),
                                        _ptr(slot_ids), _c_int(req_start.numel() - 1), _ptr(out), _ptr(scratch), _c_int(c.shape[0]), _stream()))
+    return out
+
+
+def embed_pair(tokens, positions, row_req, req_start, req_pos, slot_ids, table: torch.Tensor, pairs: Optional[torch.Tensor], mul_prev: int,
+               mul_cur: int, scale: float, state: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, x: torch.Tensor) -> torch.Tensor:
+    """x = rmsnorm(scale * table[token] + pairs[(previous * mul_prev + token * mul_cur) % buckets]) * weight; ``pairs`` has buckets + 1
+    rows, the last one for position 0; ``state`` [slots, 2, 2] of four bytes each keeps the requests' last tokens."""
+    _need(table, "table"); _need(x, "x", torch.float32)
+    lib = _build.load("blocks")
+    _check("blocks", lib.jk_embed_pair(_ptr(tokens), _ptr(positions), _ptr(row_req), _ptr(req_start), _ptr(req_pos), _ptr(slot_ids), _ptr(table),
+                                       _ptr(pairs), _c_int(dtype_code(table.dtype)), _c_int(pairs.shape[0] - 1 if pairs is not None else 0),
+                                       _c_int(mul_prev), _c_int(mul_cur), _c_float(scale), _ptr(state), _ptr(weight), _c_float(eps), _ptr(x),
+                                       _c_int(x.shape[0]), _c_int(x.shape[1]), _stream()))
+    return x
+
+
+def join_parts(x: torch.Tensor, p1: torch.Tensor, w1: Optional[torch.Tensor], eps1: float, p2: Optional[torch.Tensor] = None,
+               w2: Optional[torch.Tensor] = None, eps2: float = 0.0, p3: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += rmsnorm(p1) * w1 + rmsnorm(p2) * w2 + p3 (a part without a weight as it is); out = x in out's type."""
+    _need(x, "x", torch.float32); _need(p1, "p1", torch.float32)
+    lib = _build.load("blocks")
+    _check("blocks", lib.jk_join_parts(_ptr(x), _ptr(p1), _ptr(w1), _c_float(eps1), _ptr(p2), _ptr(w2), _c_float(eps2), _ptr(p3), _ptr(out),
+                                       _c_int(dtype_code(out.dtype) if out is not None else F32), _c_int(x.shape[0]), _c_int(x.shape[1]), _stream()))
+    return x
+
+
+def gated_recurrence(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, b_r: torch.Tensor, b_i: torch.Tensor, rate: torch.Tensor, y: torch.Tensor,
+                     y_bias: Optional[torch.Tensor], act: int, state: torch.Tensor, req_start, slot_ids, out: torch.Tensor, direct=None,
+                     n_direct: int = 0, pieces=None, n_pieces: int = 0, piece_reqs=None, n_piece_reqs: int = 0) -> torch.Tensor:
+    """The real-gated recurrence of csrc/blocks.cu over each request's rows ``u [T, C]``, from and into ``state [slots, C]``; ``w_r``,
+    ``w_i`` ``[blocks, n, n]`` of ``out``'s type; ``y`` float32 rows (a view of wider ones is fine).  The lists are those of
+    ``linear_scan``."""
+    for t, n in ((u, "u"), (b_r, "b_r"), (b_i, "b_i"), (rate, "rate"), (state, "state")):
+        _need(t, n, torch.float32)
+    _need(w_r, "w_r", out.dtype); _need(w_i, "w_i", out.dtype); _need(y, "y", torch.float32, contiguous=False)
+    T, C = u.shape
+    lib = _build.load("blocks")
+    lib.jk_gated_recurrence_scratch_floats.restype = ctypes.c_longlong
+    floats = int(lib.jk_gated_recurrence_scratch_floats(_c_int(T), _c_int(C), _c_int(n_pieces)))
+    scratch = torch.empty(max(floats, 1), dtype=torch.float32, device=u.device)
+    _check("blocks", lib.jk_gated_recurrence(_ptr(u), _ptr(w_r), _ptr(w_i), _ptr(b_r), _ptr(b_i), _ptr(rate), _ptr(y), _c_int(y.stride(0)), _ptr(y_bias),
+                                             _c_int(act), _ptr(state), _ptr(req_start), _ptr(slot_ids), _c_int(req_start.numel() - 1), _ptr(out),
+                                             _c_int(dtype_code(out.dtype)), _c_int(T), _c_int(C), _c_int(w_r.shape[0]), _ptr(direct), _c_int(n_direct),
+                                             _ptr(pieces), _c_int(n_pieces), _ptr(piece_reqs), _c_int(n_piece_reqs), _ptr(scratch), _c_ll(floats),
+                                             _stream()))
     return out

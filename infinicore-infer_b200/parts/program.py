@@ -24,17 +24,19 @@ from ..kernels import host as _host
 
 _i, _f, _p, _ll = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_longlong
 
-SLOTS = ("x", "delta", "h", "q", "o", "act", "hw", "logits", "tmp", "decode", "mix", "scan", "x0", "route", "shift", "h2")       # RunnerSlot of csrc/runner.h
+SLOTS = ("x", "delta", "h", "q", "o", "act", "hw", "logits", "tmp", "decode", "mix", "scan", "x0", "route", "shift", "h2", "part1", "part2")       # RunnerSlot of csrc/runner.h
 SLOT = {name: i for i, name in enumerate(SLOTS)}
 OP_NAMES = {1: "embed", 2: "norm", 3: "qkv", 4: "attention", 5: "residual", 6: "gate_up", 7: "linear", 8: "cast",
             9: "layernorm", 10: "conv_qkv", 11: "linear_attention", 12: "norm_add", 13: "reinject", 14: "latent_qkv",
             15: "head_linear", 16: "latent_attention", 17: "causal_conv", 18: "selective_scan", 19: "experts", 20: "softcap",
-            21: "token_shift", 22: "activate", 23: "add_rows", 24: "delta_rule", 25: "norm_pair"}
+            21: "token_shift", 22: "activate", 23: "add_rows", 24: "delta_rule", 25: "norm_pair",
+            26: "embed_pair", 27: "join", 28: "rotate", 29: "gated_recurrence"}
 OP = {name: kind for kind, name in OP_NAMES.items()}                                # RunnerOpKind
 ACT = {"none": 0, "silu": 1, "gelu_tanh": 2, "sigmoid": 3, "relu": 4, "gelu_erf": 5, "swish_clamp": 6, "tanh": 7}    # RunnerAct
-_MIXERS_OPS = (OP["cast"], OP["layernorm"], OP["conv_qkv"], OP["linear_attention"], OP["token_shift"], OP["activate"], OP["delta_rule"])
+_MIXERS_OPS = (OP["cast"], OP["layernorm"], OP["conv_qkv"], OP["linear_attention"], OP["token_shift"], OP["activate"], OP["delta_rule"],
+               OP["rotate"])
 _BLOCKS_OPS = tuple(OP[n] for n in ("norm_add", "reinject", "latent_qkv", "head_linear", "latent_attention", "causal_conv",
-                                    "selective_scan", "experts", "softcap", "add_rows", "norm_pair"))
+                                    "selective_scan", "experts", "softcap", "add_rows", "norm_pair", "embed_pair", "join", "gated_recurrence"))
 MAX_GROUPS = 8
 MAX_LISTS = 8
 
@@ -65,7 +67,11 @@ class RunnerOp(ctypes.Structure):
                 + [(n, _p) for n in ("a_log", "dt_bias", "router_bias", "gate_w", "bonus")]
                 # what learned sinks, gates of another shape, identity experts in groups and pairs of norms add
                 + [(n, _i) for n in ("group_count", "group_keep", "identity")]
-                + [(n, _p) for n in ("sink_w", "temp", "correction")])
+                + [(n, _p) for n in ("sink_w", "temp", "correction")]
+                # what pairs of tokens, joined parts, real-gated recurrences and a token's own vectors add
+                + [(n, _i) for n in ("buckets", "mul_prev", "mul_cur", "blocks")]
+                + [("score_scale", _f)]
+                + [(n, _p) for n in ("vec3", "in_bias", "b1")])
 
 
 class Routing(ctypes.Structure):
@@ -99,7 +105,7 @@ class _Fns(ctypes.Structure):
         "norm_gate", "token_shift", "act_rows", "err_mixers", "norm_add", "concat_cast", "add_bias_rows", "latent_qkv", "head_linear", "latent_attention",
         "latent_attention_scratch", "causal_conv", "selective_scan", "routed_experts", "routed_experts_workspace",
         "routed_experts_launches", "softcap", "err_blocks", "linear_small_parts", "linear_small_parts_supports", "add_rows", "delta_rule", "delta_rule_scratch",
-        "norm_pair")]
+        "norm_pair", "embed_pair", "join_parts", "gated_recurrence", "gated_recurrence_scratch", "gated_recurrence_launches", "rotate_rows")]
 
 
 def _addr(lib, name: str) -> int:
@@ -160,7 +166,9 @@ def runner_lib(gemm_tcgen05: bool = False, attention_tcgen05: bool = False, mixe
         linear_small_parts=get("linear_small", "jk_linear_small_parts"),
         linear_small_parts_supports=get("linear_small", "jk_linear_small_parts_supports"),
         add_rows=get("blocks", "jk_add_rows"), delta_rule=get("mixers", "jk_delta_rule"), delta_rule_scratch=get("mixers", "jk_delta_rule_scratch_floats"),
-        norm_pair=get("blocks", "jk_norm_pair"))
+        norm_pair=get("blocks", "jk_norm_pair"), embed_pair=get("blocks", "jk_embed_pair"), join_parts=get("blocks", "jk_join_parts"),
+        gated_recurrence=get("blocks", "jk_gated_recurrence"), gated_recurrence_scratch=get("blocks", "jk_gated_recurrence_scratch_floats"),
+        gated_recurrence_launches=get("blocks", "jk_gated_recurrence_launches"), rotate_rows=get("mixers", "jk_rotate_rows"))
     if lib.jk_runner_bind(ctypes.byref(fns)):
         from ..kernels import KernelError
         raise KernelError(lib.jk_runner_last_error().decode(errors="replace"))
@@ -210,7 +218,7 @@ class HostIO:
         """``[rows, width]`` of a slot (the activations' type unless said otherwise; ``x`` and ``delta`` are float32)."""
         rows = self.rows if rows is None else rows
         if dtype is None:
-            dtype = torch.float32 if slot in ("x", "delta", "logits", "tmp", "decode", "mix", "scan", "x0", "route") else self._runner.runtime.dtype
+            dtype = torch.float32 if slot in ("x", "delta", "logits", "tmp", "decode", "mix", "scan", "x0", "route", "part1", "part2") else self._runner.runtime.dtype
         raw = self._runner.slot_tensor(slot)
         need = rows * width * torch.empty((), dtype=dtype).element_size()
         if need > raw.numel():
