@@ -1,6 +1,6 @@
 """Configuration: typed specifications, the MiniCPM/FM9G config, the architecture registry."""
 from .specs import (AttentionSpec, BlockSpec, ConfigError, ConvAttentionSpec, FrequencyBandSpec, FrequencyRampSpec, GLUSpec,
-                    LatentAttentionSpec, ParallelBlockSpec,
+                    GatedRecurrenceSpec, LatentAttentionSpec, PairEmbeddingSpec, ParallelBlockSpec, TokenSideSpec,
                     DeltaRuleSpec, StepVectorSpec, LayerNormSpec, LinearAttentionSpec, MLPSpec, ModelSpec, PairRotarySpec, ParallelMixerSpec, PostNormBlockSpec, ReinjectSpec, RMSNormSpec,
                     RopeSpec, RoutedExpertsSpec, RunEntry, SandwichBlockSpec, SelectiveScanSpec, SwiGLUSpec, default_order)
 from .minicpm import MiniCPMConfig
@@ -9,6 +9,7 @@ from .vunelix import VunelixConfig
 from .vipovik import VipovikConfig
 from .fapenex import FapenexConfig
 from .fupapel import FupapelConfig
+from .piratar import PiratarConfig
 from .presets import PRESETS, Preset
 from .registry import (architecture_names, config_class_for, read_config,
                        register_architecture)
@@ -22,10 +23,12 @@ register_architecture("vunelix", VunelixConfig)
 register_architecture("vipovik", VipovikConfig)
 register_architecture("fapenex", FapenexConfig)
 register_architecture("fupapel", FupapelConfig)
+register_architecture("piratar", PiratarConfig)
 
 __all__ = [
     "DeltaRuleSpec", "StepVectorSpec", "FapenexConfig",
     "FrequencyBandSpec", "FupapelConfig", "ParallelBlockSpec",
+    "GatedRecurrenceSpec", "PairEmbeddingSpec", "TokenSideSpec", "PiratarConfig",
     "MLPSpec", "ParallelMixerSpec", "VipovikConfig",
     "FrequencyRampSpec", "LatentAttentionSpec", "ReinjectSpec", "RoutedExpertsSpec", "SandwichBlockSpec", "SelectiveScanSpec", "VunelixConfig",
     "ConvAttentionSpec", "GLUSpec", "LayerNormSpec", "LinearAttentionSpec", "PairRotarySpec", "PostNormBlockSpec", "SitelornConfig",

@@ -221,7 +221,9 @@ class LinearAttentionSpec:
     state; ``bonus_name``: a tensor u [heads, head_dim], and a row reads the state BEFORE its own decay with a bonus for its
     own key, o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t; ``decay_form`` "exp_neg_exp": a_t = exp(-exp(z)) instead of
     sigmoid(z) ** (1 / tau); ``decay_act``: an activation on W1's output; ``decay_bias_name`` names the bias of W2;
-    ``norm_per_head`` "unit": the mean per head, a weight of heads * v_head_dim."""
+    ``norm_per_head`` "unit": the mean per head, a weight of heads * v_head_dim; ``norm_name`` None: the norm has no weight.
+    ``position``: a rotation of q and k ahead of the recurrence.  (A factor on k is a factor on what S^T q gives, so it may ride
+    on ``q_scale``.)"""
     hidden_size: int
     num_heads: int
     head_dim: int
@@ -239,7 +241,7 @@ class LinearAttentionSpec:
     v_name: str = "v"
     gate_name: str = "g"
     o_name: str = "o"
-    norm_name: str = "norm"
+    norm_name: Optional[str] = "norm"
     decay_down_name: str = "a1"
     decay_up_name: str = "a2"
     bias_suffix: str = ".b"
@@ -250,6 +252,7 @@ class LinearAttentionSpec:
     decay_form: str = "sigmoid_pow"
     decay_act: str = "none"
     decay_bias_name: Optional[str] = None
+    position: Optional[PairRotarySpec] = None
     kind: str = "linear_attention"
 
 
@@ -332,7 +335,7 @@ class RoutedExpertsSpec:
     ``groups`` (count, keep): the outputs form ``count`` groups of neighbours, and only those of the ``keep`` groups whose best
     choice score is largest can be chosen.
     ``shared_gate_name``: the shared unit's output is multiplied by sigmoid(w . h), one number per row, w that tensor
-    ([1, hidden], below ``shared_prefix``)."""
+    ([1, hidden], below ``shared_prefix``).  ``score_scale``: a factor on the renormalised scores ("softmax_renorm" only)."""
     hidden_size: int
     num_experts: int
     top: int
@@ -349,6 +352,7 @@ class RoutedExpertsSpec:
     num_identity: int = 0
     correction_name: Optional[str] = None
     groups: Optional[Tuple[int, int]] = None
+    score_scale: float = 1.0
     expert_prefix: str = "e{}."
     shared_prefix: str = "shared."
     gate_name: str = "gate"
@@ -420,6 +424,66 @@ class DeltaRuleSpec:
 
 
 @dataclass(frozen=True)
+class GatedRecurrenceSpec:
+    """A linear recurrence per channel with real gates, behind a short convolution and beside a gated branch:
+
+        y = act(``y_name`` h + b),   u = conv(``x_name`` h + b)                    ``inner`` channels each
+        r = sigmoid(R u + b), i = sigmoid(I u + b),   log a = -``rate`` r softplus(``lam_name``)
+        S <- a S + sqrt(1 - a^2) i u;   output ``o_name`` (S y)
+
+    R (``r_name``) and I (``i_name``) are block-diagonal, [``blocks``, n, n] with n = inner / blocks, their biases [blocks, n].  The
+    convolution has ``conv_taps`` taps per channel ([inner, taps], the last column the current row's), a bias and no activation; the
+    projection's bias comes before it, so what precedes the sequence is zero.  S [inner] and the convolution's last taps - 1 inputs
+    are kept per request, in float32."""
+    hidden_size: int
+    inner: int
+    blocks: int
+    conv_taps: int
+    rate: float = 8.0
+    act: str = "gelu_tanh"
+    y_name: str = "y"
+    x_name: str = "x"
+    conv_name: str = "conv"
+    r_name: str = "ra"
+    i_name: str = "ri"
+    lam_name: str = "lam"
+    o_name: str = "o"
+    bias_suffix: str = ".b"
+    kind: str = "gated_recurrence"
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """A step after a layer that brings in a vector of the row's own token: with e the ``dim`` elements from ``offset`` on of the
+    token's row of ``table_name`` [vocab, ``table_width``],
+
+        y = ``proj_name`` (act(``gate_name`` x) * e);   x <- x + y / sqrt(mean(y^2) + eps) * w  (``norm``)
+
+    ``gate_name`` [dim, hidden], ``proj_name`` [hidden, dim]."""
+    hidden_size: int
+    vocab_size: int
+    dim: int
+    table_width: int
+    offset: int
+    norm: RMSNormSpec
+    gate_name: str
+    proj_name: str
+    act: str = "gelu_tanh"
+    table_name: str = "side.embed"
+    kind: str = "token_side"
+
+
+@dataclass(frozen=True)
+class PairEmbeddingSpec:
+    """A table with a vector per pair of neighbouring tokens, by a hash: row (previous * ``mul_prev`` + token * ``mul_cur``) mod
+    ``buckets`` of ``table_name`` [buckets + 1, hidden], its last row for a sequence's first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    table_name: str = "bigram"
+
+
+@dataclass(frozen=True)
 class SandwichBlockSpec:
     """One layer with a norm before and after each sublayer: x += norm_b(mixer(norm_a(x))); x += norm_d(ff(norm_c(x))).
     ``feed_forward`` None: the layer has a mixer only."""
@@ -467,13 +531,16 @@ class MLPSpec:
 @dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input: ``left_scale`` * left(h) + ``right_scale`` * right(h).  Each is any
-    mixer's specification; at most one of them keeps pages."""
+    mixer's specification; at most one of them keeps pages.  ``left_norm``, ``right_norm``: an RMS norm that the side's output passes
+    before its factor; its weight's name follows the side's prefix."""
     left: object
     right: object
     left_scale: float = 1.0
     right_scale: float = 1.0
     left_prefix: str = "left."
     right_prefix: str = "right."
+    left_norm: Optional[RMSNormSpec] = None
+    right_norm: Optional[RMSNormSpec] = None
     kind: str = "parallel"
 
 
@@ -497,13 +564,15 @@ class ParallelBlockSpec:
     """One layer whose two sublayers stand side by side, each behind a norm of its own of the same stream:
     x += s * (mixer(shift(norm_a(x))) + feed_forward(norm_b(x))).  ``feed_forward`` None: the layer has a mixer only.
     ``shift_name``: a tensor [hidden] below the layer's prefix; what the mixer reads is h_t + (h_(t-1) - h_t) * that tensor,
-    h the norm's output (h_(-1) = 0); None: h itself."""
+    h the norm's output (h_(-1) = 0); None: h itself.  ``joined``: neither side adds into the stream by itself; their outputs wait and
+    one kernel adds them all (``residual_scale`` 1 only)."""
     mixer: object
     feed_forward: Optional[object]
     mixer_norm: object
     ffn_norm: Optional[object]
     residual_scale: float = 1.0
     shift_name: Optional[str] = None
+    joined: bool = False
     mixer_prefix: str = "mix."
     ffn_prefix: str = "mlp."
     mixer_norm_prefix: str = "norm1"
@@ -543,6 +612,7 @@ class RunEntry:
     cache: int
     writes_cache: bool = True
     before: Optional[object] = None     # a step on the stream that runs before the layer (``ReinjectSpec``), or None
+    after: Optional[object] = None      # one that runs after it (``TokenSideSpec``), or None
 
 
 @dataclass(frozen=True)
@@ -559,6 +629,9 @@ class ModelSpec:
     logit_softcap: float = 0.0         # c > 0: logits <- c tanh(logits / c)
     position_table_name: Optional[str] = None      # a learned vector per position [position_rows, hidden], added to the embedding
     position_rows: int = 0
+    pairs: Optional[PairEmbeddingSpec] = None      # a vector per pair of neighbouring tokens, added to the embedding
+    embed_norm: Optional[RMSNormSpec] = None       # a norm of the embedding (and what was added to it)
+    embed_norm_prefix: str = ""
     tie_embeddings: bool = False
     embed_name: str = "model.embed_tokens.weight"
     lm_head_name: str = "lm_head.weight"

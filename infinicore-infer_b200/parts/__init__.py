@@ -22,10 +22,13 @@ from .parallel_mixer import ParallelMixer
 from .step_vector import StepVector
 from .delta_rule import DeltaRule
 from .parallel_block import ParallelBlock
+from .gated_recurrence import GatedRecurrence
+from .token_side import TokenSide
 from .model import Model, cache_needs, model_manifest, state_needs
 
 __all__ = ["BLOCKS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITIONS", "ResidualStream", "Runtime", "StepContext", "Program",
            "ProgramRunner", "HostIO", "part_class", "register", "RMSNorm", "RotaryTables", "Attention", "SwiGLU",
            "PreNormBlock", "LayerNorm", "GLU", "LinearAttention", "ConvAttention", "PostNormBlock", "LatentAttention",
-           "SelectiveScan", "RoutedExperts", "SandwichBlock", "Reinject", "MLP", "ParallelMixer", "StepVector", "DeltaRule", "ParallelBlock", "Model", "cache_needs", "model_manifest",
+           "SelectiveScan", "RoutedExperts", "SandwichBlock", "Reinject", "MLP", "ParallelMixer", "StepVector", "DeltaRule", "ParallelBlock",
+           "GatedRecurrence", "TokenSide", "Model", "cache_needs", "model_manifest",
            "state_needs"]

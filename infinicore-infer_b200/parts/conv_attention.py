@@ -123,9 +123,10 @@ class ConvAttention:
         itself."""
         self.plan_delta(program, view, writes_cache, state_view=state_view, into_stream=residual_scale)
 
-    def plan_delta(self, program, view, writes_cache: bool = True, state_view=None, into_stream=None) -> None:
+    def plan_delta(self, program, view, writes_cache: bool = True, state_view=None, into_stream=None,
+                   out_slot: str = "delta") -> None:
         """Four records: the fused product (h -> float32 rows), convolution / norm / rotation / cache write (-> q), the
-        attention (-> o), the output product into the delta slot (``into_stream`` s: added into the stream times s)."""
+        attention (-> o), the output product into the delta slot or another (``into_stream`` s: added into the stream times s)."""
         s = self.spec
         if writes_cache == s.shares_kv:
             raise ValueError("a layer that borrows its keys writes no cache, and one that has keys writes its own")
@@ -153,7 +154,7 @@ class ConvAttention:
                    list_tiles=tiles, max_positions=program.max_blocks * program.page_size, k_pages=view.k_pages,
                    v_pages=view.v_pages, num_pages=view.k_pages.shape[0], sink=s.sink, sink_w=self.sink_w, gated=2 if s.element_gate else int(s.head_gate), ld=ld, g_off=g_off,
                    cap=float(s.score_cap or 0.0), keep_first=s.keep_first if s.window else 0),
-            record("linear", "o", "delta", n=s.hidden_size, k=s.num_heads * s.v_head_dim, w=self.w_o) if into_stream is None else
+            record("linear", "o", out_slot, n=s.hidden_size, k=s.num_heads * s.v_head_dim, w=self.w_o) if into_stream is None else
             record("residual", "o", "x", n=s.hidden_size, k=s.num_heads * s.v_head_dim, w=self.w_o, scale=float(into_stream)),
         ], keep=(self.w_in, self.w_o, self.conv, self.norms, self.freq, state, view.k_pages, view.v_pages, self.bias, self.temp, self.sink_w))
 

@@ -37,8 +37,9 @@ class LinearAttention:
         nk, nv = LinearAttention._widths(spec)
         shared_norm = spec.norm_per_head and spec.norm_per_head != "unit"
         decls = {spec.q_name: TensorDecl((nk, d)), spec.k_name: TensorDecl((nk, d)), spec.v_name: TensorDecl((nv, d)),
-                 spec.gate_name: TensorDecl((nv, d)), spec.o_name: TensorDecl((d, nv)),
-                 spec.norm_name: TensorDecl((spec.v_head_dim if shared_norm else nv,), VECTOR, init="ones")}
+                 spec.gate_name: TensorDecl((nv, d)), spec.o_name: TensorDecl((d, nv))}
+        if spec.norm_name:
+            decls[spec.norm_name] = TensorDecl((spec.v_head_dim if shared_norm else nv,), VECTOR, init="ones")
         if spec.decay is None:
             decls[spec.decay_down_name] = TensorDecl((spec.decay_rank, d))
             decls[spec.decay_up_name] = TensorDecl((nk, spec.decay_rank))
@@ -83,7 +84,15 @@ class LinearAttention:
         names = [spec.q_name, spec.k_name, spec.v_name, spec.gate_name] + ([spec.decay_down_name] if spec.decay is None else [])
         self.w_in = weights.get_rows([prefix + n for n in names], MATRIX)
         self.w_o = weights.get(prefix + spec.o_name, MATRIX)
-        self.norm = weights.get(prefix + spec.norm_name, VECTOR)
+        self.norm = weights.get(prefix + spec.norm_name, VECTOR) if spec.norm_name else None
+        self.freq, self.rot_mag = None, 1.0
+        if spec.position is not None and spec.position.dims:
+            if spec.position.layout not in ("pairs", "halves"):
+                raise ValueError(f"a rotation pairs neighbours (\"pairs\") or halves (\"halves\"), not {spec.position.layout!r}")
+            if spec.qkv_act != "none":
+                raise ValueError("a rotation of activated queries and keys is not built")
+            freq, self.rot_mag = spec.position.frequencies()          # float64, rounded once
+            self.freq = torch.tensor(freq, dtype=torch.float64).to(torch.float32).to(runtime.device)
         self.decay = self.w2 = self.b2 = self.mu = self.bonus = None
         if spec.token_shift:        # the mixing vectors, one row per projection in the order of their columns
             self.mu = torch.stack([weights.get(prefix + spec.shift_prefix + mu, VECTOR) for mu, _ in self._shifted(spec)]).contiguous()
@@ -137,10 +146,10 @@ class LinearAttention:
         """The mixer in a block that adds its output to the stream itself."""
         self.plan_delta(program, view, writes_cache, state_view=state_view, into_stream=residual_scale)
 
-    def plan_delta(self, program, view, writes_cache: bool = True, state_view=None, into_stream=None) -> None:
+    def plan_delta(self, program, view, writes_cache: bool = True, state_view=None, into_stream=None, out_slot: str = "delta") -> None:
         """Three records: the fused product (h -> float32 rows), the recurrence with norm and gate (-> o), the output product
-        into the delta slot (``into_stream`` s: added into the stream times s).  With a token shift the first is the shift
-        and one product per projection."""
+        into the delta slot or another (``into_stream`` s: added into the stream times s).  With a token shift the first is the
+        shift and one product per projection; a rotation is a record behind it."""
         s = self.spec
         nk, nv = self._widths(s)
         ld = self.w_in.shape[0]
@@ -158,6 +167,9 @@ class LinearAttention:
                 row += width
         else:
             records = [record("linear", "h", "tmp", n=ld, k=s.hidden_size, w=self.w_in)]
+        if self.freq is not None:
+            records.append(record("rotate", "tmp", "tmp", heads=s.num_heads, head_dim=s.head_dim, ld=ld, q_off=0, k_off=nk, freq=self.freq,
+                                  rot_dims=s.position.dims, rot_half=s.position.layout == "halves", rot_mag=self.rot_mag))
         per_head = 2 if s.norm_per_head == "unit" else (1 if s.norm_per_head else 0)
         records += [
             record("linear_attention", "tmp", "o", list_short=direct, list_tiles=pieces, list_aux=piece_reqs, heads=s.num_heads, head_dim=s.head_dim, v_head_dim=s.v_head_dim, ld=ld,
@@ -165,10 +177,10 @@ class LinearAttention:
                    gate_act=ACT[s.gate_act], per_head_norm=per_head, eps=s.norm_eps, vec=self.norm, decay=self.decay,
                    w2=self.w2, b2=self.b2, rank=s.decay_rank if s.decay is None else 0, tau=s.decay_tau, state=view.state,
                    bonus=self.bonus, decay_form=1 if s.decay_form == "exp_neg_exp" else 0, rank_act=ACT[s.decay_act]),
-            record("linear", "o", "delta", n=s.hidden_size, k=nv, w=self.w_o) if into_stream is None else
+            record("linear", "o", out_slot, n=s.hidden_size, k=nv, w=self.w_o) if into_stream is None else
             record("residual", "o", "x", n=s.hidden_size, k=nv, w=self.w_o, scale=float(into_stream)),
         ]
-        program.emit_records(records, keep=(self.w_in, self.w_o, self.norm, self.decay, self.w2, self.b2, view.state, self.mu, self.bonus,
+        program.emit_records(records, keep=(self.w_in, self.w_o, self.norm, self.decay, self.w2, self.b2, view.state, self.mu, self.bonus, self.freq,
                                             state_view.state if state_view is not None else None))
 
     def forward(self, h: torch.Tensor, ctx, view, writes_cache: bool = True, state_view=None) -> torch.Tensor:

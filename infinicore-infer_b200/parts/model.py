@@ -11,6 +11,7 @@ from typing import Dict, List
 
 import torch
 
+from ..cache import StateSlot
 from ..weights import MATRIX, TensorDecl
 from .base import ResidualStream, Runtime, StepContext, part_class
 from .program import Program
@@ -23,6 +24,11 @@ def model_manifest(spec) -> Dict[str, TensorDecl]:
            spec.lm_head_name: TensorDecl((spec.vocab_size, spec.hidden_size), optional=True)}
     if spec.position_table_name:
         out[spec.position_table_name] = TensorDecl((spec.position_rows, spec.hidden_size))
+    if spec.pairs is not None:
+        out[spec.pairs.table_name] = TensorDecl((spec.pairs.buckets + 1, spec.hidden_size))
+    if spec.embed_norm is not None:
+        for name, decl in part_class("norm", spec.embed_norm).tensor_decls(spec.embed_norm).items():
+            out[spec.embed_norm_prefix + name] = decl
     for name, decl in part_class("norm", spec.final_norm).tensor_decls(spec.final_norm).items():
         out[spec.final_norm_prefix + name] = decl
     for i, layer in enumerate(spec.layers):
@@ -30,8 +36,9 @@ def model_manifest(spec) -> Dict[str, TensorDecl]:
         for name, decl in part_class("block", layer).tensor_decls(layer).items():
             out[prefix + name] = decl
     for e in spec.order:          # steps between layers name their tensors without a layer's prefix
-        if e.before is not None:
-            out.update(part_class("stream", e.before).tensor_decls(e.before))
+        for step in (e.before, e.after):
+            if step is not None:
+                out.update(part_class("stream", step).tensor_decls(step))
     return out
 
 
@@ -58,12 +65,15 @@ def cache_needs(spec) -> List[object]:
 
 def state_needs(spec) -> List[object]:
     """What each entry of the run order keeps for itself beside its cache (``StateSlot`` or None), asked of the block
-    class's ``state_need(spec, writes_cache)`` where it has one."""
+    class's ``state_need(spec, writes_cache)`` where it has one; behind those, what the embedding keeps (the last token, where pairs of
+    tokens have vectors)."""
     out: List[object] = []
     for e in spec.order:
         layer = spec.layers[e.layer]
         ask = getattr(part_class("block", layer), "state_need", None)
         out.append(ask(layer, e.writes_cache) if ask is not None else None)
+    if spec.pairs is not None:
+        out.append(StateSlot((2, 2), "float32"))    # two marked tokens that take turns, as integers (csrc/blocks.cu: embed_pair)
     return out
 
 
@@ -80,6 +90,10 @@ class Model:
             self.position_table = weights.get(spec.position_table_name, MATRIX)
             if spec.max_positions > self.position_table.shape[0]:
                 raise ValueError(f"sequences of up to {spec.max_positions} positions, but {spec.position_table_name} holds {self.position_table.shape[0]}")
+        self.pair_table = weights.get(spec.pairs.table_name, MATRIX) if spec.pairs is not None else None
+        self.embed_norm = None
+        if spec.embed_norm is not None:
+            self.embed_norm = part_class("norm", spec.embed_norm)(spec.embed_norm, weights, spec.embed_norm_prefix, runtime)
         self.final_norm = part_class("norm", spec.final_norm)(spec.final_norm, weights,
                                                               spec.final_norm_prefix, runtime)
         self.layers = [part_class("block", layer)(layer, weights, spec.layer_prefix.format(i), runtime)
@@ -87,6 +101,10 @@ class Model:
         shared: dict = {}          # tensors that several steps between layers use are loaded once
         self.before = [None if e.before is None else part_class("stream", e.before)(e.before, weights, "", runtime, shared=shared)
                        for e in spec.order]
+        self.after = [None if e.after is None else part_class("stream", e.after)(e.after, weights, "", runtime, shared=shared)
+                      for e in spec.order]
+        if (self.pair_table is not None or self.embed_norm is not None) and any(getattr(b, "needs_embedding_output", False) for b in self.before):
+            raise ValueError("an embedding with pairs or a norm that is fed in again later is not built")
 
     @property
     def graph_safe(self) -> bool:
@@ -99,7 +117,7 @@ class Model:
             total += self.spec.hidden_size * self.position_table.element_size()
         for e in self.spec.order:
             total += getattr(self.layers[e.layer], "weight_bytes", lambda: 0)()
-        total += sum(b.weight_bytes() for b in self.before if b is not None and hasattr(b, "weight_bytes"))
+        total += sum(b.weight_bytes() for b in self.before + self.after if b is not None and hasattr(b, "weight_bytes"))
         return total
 
     def plan(self, views, page_size: int, max_blocks: int, state_views=None) -> Program:
@@ -109,8 +127,11 @@ class Model:
         from .. import kernels
         spec = self.spec
         program = Program(self.runtime, spec.hidden_size, page_size, max_blocks, capacity=8 * len(spec.order) + 8)
-        program.emit("jk_emit_embedding", ctypes.c_void_p(self.embedding.data_ptr()), ctypes.c_int(kernels.dtype_code(self.embedding.dtype)),
-                     ctypes.c_int(spec.hidden_size), ctypes.c_float(spec.embed_scale), keep=(self.embedding,))
+        if self.pair_table is not None or self.embed_norm is not None:
+            self._plan_pair_embedding(program, state_views)
+        else:
+            program.emit("jk_emit_embedding", ctypes.c_void_p(self.embedding.data_ptr()), ctypes.c_int(kernels.dtype_code(self.embedding.dtype)),
+                         ctypes.c_int(spec.hidden_size), ctypes.c_float(spec.embed_scale), keep=(self.embedding,))
         hidden = spec.hidden_size
         if self.position_table is not None:
             from .program import record
@@ -132,6 +153,8 @@ class Model:
                     layer.plan(program, view, e.writes_cache)
             else:
                 program.host(_host_block(layer, view, e.writes_cache, hidden))
+            if self.after[index] is not None:
+                self.after[index].plan(program)
         if hasattr(self.final_norm, "plan"):
             self.final_norm.plan(program, out_scale=spec.logit_scale, wanted_rows=True)
         else:
@@ -142,6 +165,21 @@ class Model:
             from .program import record
             program.emit_records([record("softcap", "logits", None, n=spec.vocab_size, cap=float(spec.logit_softcap), wanted_rows=True)])
         return program
+
+    def _plan_pair_embedding(self, program, state_views) -> None:
+        """The embedding, the vectors of pairs of tokens and the norm as one record."""
+        from .. import kernels
+        from .program import record
+        spec, pairs, norm = self.spec, self.spec.pairs, self.embed_norm
+        kept = state_views[len(spec.order)].state if pairs is not None and state_views else None
+        if pairs is not None and kept is None:
+            raise ValueError("vectors of pairs of tokens need the state that keeps a request's last token")
+        fields = dict(w3=self.pair_table, buckets=pairs.buckets, mul_prev=pairs.mul_prev, mul_cur=pairs.mul_cur, state=kept) if pairs is not None else {}
+        if norm is not None:
+            fields.update(vec=norm.weight, eps=norm.spec.eps)
+        program.emit_records([record("embed_pair", None, "x", n=spec.hidden_size, w=self.embedding, w_dtype=kernels.dtype_code(self.embedding.dtype),
+                                     scale=spec.embed_scale, **fields)],
+                             keep=(self.embedding, self.pair_table, kept, norm.weight if norm is not None else None))
 
 
 def _host_block(layer, view, writes_cache: bool, hidden: int):

@@ -50,6 +50,19 @@ class RMSNorm:
         else:
             program.keep.append(self.weight)
 
+    def plan_pair_after_add(self, program, other) -> bool:
+        """This norm and ``other`` (None: this one alone) over every row into the slots ``h`` and ``h2``, right after a ``plan_add``, by
+        joining that record; whether it did."""
+        fields = dict(out_slot="h", vec2=self.weight, eps2=self.spec.eps)
+        if other is not None:
+            if other.spec.eps != self.spec.eps:
+                return False
+            fields.update(out2_slot="h2", vec3=other.weight)
+        if not program.amend_last("norm_add", **fields):
+            return False
+        program.keep.extend([self.weight] + ([other.weight] if other is not None else []))
+        return True
+
     def forward(self, residual: ResidualStream, ctx, out_scale: float = 1.0,
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Normalise every row, or only ``rows`` (int32 indices) of the residual stream."""

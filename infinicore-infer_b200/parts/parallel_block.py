@@ -5,6 +5,9 @@ once), the first mixed with the row before it where the block has a token shift;
 feed-forward a second one.  The mixer's output product then adds into the stream (or waits for it), and the feed-forward
 adds after it.  The row that the shift needs from the step before is kept per request in float32 (as two rows that take
 turns: a step reads one and leaves the other), beside whatever the mixer keeps.
+
+``joined``: the mixer's output (or those of its sides, each with a norm) and the feed-forward's wait in slots of their own, and one
+``join`` record adds them all.  Without a shift both norms join the record before, where that is a norm that adds to the stream.
 """
 from __future__ import annotations
 
@@ -63,6 +66,8 @@ class ParallelBlock:
                 raise TypeError(f"{type(self.feed_forward).__name__} cannot read a slot of its own beside the mixer's (no plan with in_slot)")
         if not hasattr(self.mixer, "plan"):
             raise TypeError(f"{type(self.mixer).__name__} cannot add its output into the stream (no plan)")
+        if spec.joined and spec.residual_scale != 1.0:
+            raise ValueError("joined sublayers with a residual factor are not built")
         for norm in (self.mixer_norm, self.ffn_norm):
             if norm is not None and getattr(norm.spec, "kind", None) != "rmsnorm":
                 raise TypeError(f"a pair of norms is built of RMS norms, not of {type(norm).__name__}")
@@ -84,17 +89,36 @@ class ParallelBlock:
                 mixer_state = state_view.rest(1) if isinstance(mine, StateSlots) else state_view[1]
         else:
             mixer_state = state_view
-        program.emit_records([
-            record("norm_pair", "x", "h", out2_slot="h2" if second is not None else None, n=first.spec.size, vec=first.weight, eps=first.spec.eps,
-                   vec2=second.weight if second is not None else None, eps2=second.spec.eps if second is not None else 0.0,
-                   bias=self.shift, state=kept),
-        ], keep=(first.weight, second.weight if second is not None else None, self.shift, kept))
+        if s.shift_name or not first.plan_pair_after_add(program, second):
+            self._plan_norms(program, first, second, kept)
+        if s.joined:
+            self._plan_joined(program, view, writes_cache, mixer_state)
+            return
         if mixer_state is not None or hasattr(type(self.mixer), "state_need"):
             self.mixer.plan(program, view, writes_cache, s.residual_scale, state_view=mixer_state)
         else:
             self.mixer.plan(program, view, writes_cache, s.residual_scale)
         if self.feed_forward is not None:
             self.feed_forward.plan(program, s.residual_scale, in_slot="h2")
+
+    def _plan_norms(self, program, first, second, kept) -> None:
+        program.emit_records([
+            record("norm_pair", "x", "h", out2_slot="h2" if second is not None else None, n=first.spec.size, vec=first.weight, eps=first.spec.eps,
+                   vec2=second.weight if second is not None else None, eps2=second.spec.eps if second is not None else 0.0,
+                   bias=self.shift, state=kept),
+        ], keep=(first.weight, second.weight if second is not None else None, self.shift, kept))
+
+    def _plan_joined(self, program, view, writes_cache: bool, mixer_state) -> None:
+        extra = {"state_view": mixer_state} if mixer_state is not None or hasattr(type(self.mixer), "state_need") else {}
+        parts = self.mixer.plan_parts(program, view, writes_cache, **extra) if hasattr(self.mixer, "plan_parts") else None
+        if parts is None:
+            self.mixer.plan_delta(program, view, writes_cache, out_slot="part1", **extra)
+            parts = [("part1", None, 0.0)]
+        if self.feed_forward is not None:
+            self.feed_forward.plan_delta(program, in_slot="h2")
+        (a, wa, ea), (b, wb, eb) = (parts + [(None, None, 0.0)])[:2]
+        program.emit_records([record("join", a, None, in2_slot=b, n=self.mixer_norm.spec.size, vec=wa, eps=ea, vec2=wb, eps2=eb,
+                                     add=self.feed_forward is not None)], keep=(wa, wb))
 
 
 def _children(spec):

@@ -59,6 +59,8 @@ class RoutedExperts:
             raise ValueError("built are sigmoid scores on a unit's input and softmax scores on its output")
         if spec.score_form != "softmax" and (spec.num_identity or spec.correction_name or spec.groups):
             raise ValueError("identity units, a corrected choice and groups are built for plain softmax scores")
+        if spec.score_scale != 1.0 and (spec.score_form != "softmax_renorm" or not spec.score_scale > 0):
+            raise ValueError("a factor of the scores is built for renormalised softmax scores, and positive")
         if spec.act == "swish_clamp" and not spec.limit > 0:
             raise ValueError("a clamped unit needs a positive limit")
         outputs = spec.num_experts + spec.num_identity
@@ -104,7 +106,7 @@ class RoutedExperts:
                    w=self.w_gate_up, w3=self.w_down, add=self.shared is not None, act=ACT[s.act], limit=float(s.limit),
                    score_form=SCORE_FORMS.index(s.score_form), into_stream=into_stream, router_bias=self.router_bias,
                    gate_w=self.shared_gate, identity=s.num_identity, group_count=count, group_keep=keep, correction=self.correction,
-                   scale=float(scale)),
+                   scale=float(scale), score_scale=float(s.score_scale)),
         ], keep=(self.correction, self.router, self.w_gate_up, self.w_down, self.router_bias, self.shared_gate))
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
