@@ -114,4 +114,18 @@ PRESETS: Dict[str, Preset] = {
                                               "kv_from": 0},
              "mlp": {"kind": "moe", "router": {"experts": 3, "identity": 3, "top": 2, "groups": {"count": 3, "keep": 2}}, "expert": {"ff": 32}}},
         ]), 0.1, 0.05, 16),
+    # a small Piratar: attention beside retention, a real-gated recurrence, a dense, a routed and no feed-forward, pairs of tokens and
+    # token vectors in every layer
+    "piratar-tiny": Preset(dict(
+        architecture="Piratar", vocab=320, width=96, norm={"eps": 1e-5}, embedding={"scale": 8.0, "bigram": {"buckets": 211, "mul_prev": 31, "mul_cur": 7}},
+        token_side={"dim": 16}, layers=[
+            {"type": "parallel", "mixer": {
+                "left": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.25, "conv": 4, "rot": {"base": 1e4, "dims": 16}},
+                "right": {"heads": 3, "dim": 16, "vdim": 24, "decay": [0.75, 0.96875, 0.998], "rot": {"base": 1e5, "dims": 16}}},
+             "mlp": {"kind": "moe", "router": {"experts": 6, "top": 2, "scale": 1.5}, "expert": {"ff": 48}, "shared": {"ff": 64}}},
+            {"type": "rglru", "mixer": {"width": 128, "blocks": 4, "conv": 3}, "mlp": {"kind": "dense", "ff": 160}},
+            {"type": "parallel", "mixer": {
+                "left": {"heads": 2, "kv_heads": 1, "dim": 32, "vdim": 16, "scale": 0.2, "conv": 2, "rot": {"base": 5e4, "dims": 32}},
+                "right": {"heads": 2, "dim": 24, "vdim": 16, "decay": [0.9, 0.99], "rot": {"base": 1e4, "dims": 8}}}, "mlp": None},
+        ]), 0.1, 0.05, 16),
 }
