@@ -325,6 +325,25 @@ def fupapel_shape(width, ff, heads, kv_heads, dim, vocab, window):
             "layers": [att, conv, lat, lat, att, borrows, lat, att]}
 
 
+def piratar_shape(width, ff, heads, kv_heads, dim, vocab):
+    """Eight layers P P R U P R U P, mixers and feed-forwards side by side: P attention with grouped heads of ``dim`` behind
+    convolutions of four taps, rotated whole, a gate per output element, beside retention with heads of ``dim`` x ``dim``; U the same
+    with attention keys of dim / 2 and values of ``dim`` and retention heads of dim / 2 x dim; R a real-gated recurrence over the width
+    with gates' maps of 256.  A dense feed-forward in the first layer, then eight experts of ff / 4 of which a row takes two, and a
+    shared one with a gate per row; pairs of tokens, and token vectors of 256 in every layer."""
+    decay = lambda n: [1.0 - 2.0 ** (-5 - 6 * h / max(1, n - 1)) for h in range(n)]
+    def both(dk):
+        return {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dk, "vdim": dim, "scale": dk ** -0.5, "conv": 4, "rot": {"base": 5e5, "dims": dk}},
+                "right": {"heads": heads, "dim": dk, "vdim": dim, "decay": decay(heads), "rot": {"base": 1e4, "dims": dk}}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2, "scale": 2.0}, "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4}}
+    P, U = ({"type": "parallel", "mixer": both(dk), "mlp": moe} for dk in (dim, dim // 2))
+    R = {"type": "rglru", "mixer": {"width": width, "blocks": width // 256, "conv": 4}, "mlp": moe}
+    return {"architecture": "Piratar", "norm": {"eps": 1e-5}, "vocab": vocab, "width": width,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}, "token_side": {"dim": 256},
+            "layers": [dict(P, mlp=dense), P, R, U, P, R, U, P]}
+
+
 def decoder_shape(width, ff, heads, kv_heads, dim, vocab, layers=8):
     return dict(model_type="llama", num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv_heads,
                 head_dim=dim, intermediate_size=ff, vocab_size=vocab, max_position_embeddings=4096, rms_norm_eps=1e-5,
@@ -355,13 +374,22 @@ def record_cost(op, T, B, context, decode, page_bytes):
     if kind == "token_shift":
         return T * op.n * 2 * (1 + op.heads) + B * op.n * 8, 2.0 * T * op.n * op.heads
     if kind == "activate":
-        return T * op.n * (4 + 2), 0.0
+        return T * op.n * (4 + 2 + (2 if op.w else 0)), 0.0
+    if kind == "rotate":
+        return T * op.heads * op.rot_dims * 2 * (4 + 4), 0.0
+    if kind == "embed_pair":
+        return T * op.n * (2 + (2 if op.w3 else 0) + 4), 0.0
+    if kind == "join":
+        return T * op.n * (4 + 4 + 4 + (4 if op.in2_slot >= 0 else 0) + (4 if op.add else 0) + (2 if op.out_slot >= 0 else 0)), 0.0
+    if kind == "gated_recurrence":
+        size = op.n // op.blocks
+        return 2 * 2 * op.n * size + T * op.n * (4 + 4 + 2) + B * op.n * 8, 4.0 * T * op.n * size
     if kind in ("layernorm", "norm"):
         return T * op.n * (4 + 4 + 4 + 2), 0.0
     if kind == "cast":
         return T * op.n * 6, 0.0
     if kind == "norm_add":
-        return T * op.n * (4 + 4 + 4 + 2), 0.0
+        return T * op.n * (4 + 4 + 4 + 2 + (2 if op.out2_slot >= 0 else 0)), 0.0
     if kind == "norm_pair":
         return T * op.n * (4 + 2 + (2 if op.out2_slot >= 0 else 0)) + B * op.n * 8, 0.0
     if kind == "reinject":
@@ -396,13 +424,13 @@ def record_cost(op, T, B, context, decode, page_bytes):
 
 
 def run_design(args):
-    """Prefill and decode of another design (Sitelorn, Vunelix, Vipovik, Fapenex, Fupapel) at layer sizes of real models beside the decoder (llama graph) of
+    """Prefill and decode of another design (Sitelorn, Vunelix, Vipovik, Fapenex, Fupapel, Piratar) at layer sizes of real models beside the decoder (llama graph) of
     the same width, feed-forward, heads and layer count (Vipovik: also beside Sitelorn, Fapenex: also beside Vunelix, Fupapel: also
-    beside Fapenex, the designs closest to them), and every kind
+    beside Fapenex, Piratar: also beside Vipovik and Fupapel, the designs closest to them), and every kind
     of launch record of each timed alone against its roofline.  Prints one JSON line of its own kind; the default benchmark is
     untouched."""
     import torch
-    from infinicore_infer_b200.config import FapenexConfig, FupapelConfig, MiniCPMConfig, SitelornConfig, VipovikConfig, VunelixConfig
+    from infinicore_infer_b200.config import FapenexConfig, FupapelConfig, MiniCPMConfig, PiratarConfig, SitelornConfig, VipovikConfig, VunelixConfig
     from infinicore_infer_b200.engine import Engine, StepEntry
     from infinicore_infer_b200.parts import model_manifest
     from infinicore_infer_b200.parts.program import OP_NAMES
@@ -420,9 +448,11 @@ def run_design(args):
         for size in args.design_sizes.split(","):
             width, ff, heads, kv_heads, dim, vocab = DESIGN_SIZES[size]
             block = out["sizes"][size] = {"width": width, "ff": ff, "heads": heads, "kv_heads": kv_heads, "head_dim": dim, "layers": 8}
-            beside = {"vipovik": ("sitelorn",), "fapenex": ("vunelix",), "fupapel": ("fapenex",)}.get(args.design, ())
+            beside = {"vipovik": ("sitelorn",), "fapenex": ("vunelix",), "fupapel": ("fapenex",), "piratar": ("vipovik", "fupapel")}.get(args.design, ())
             for which in (args.design,) + beside + ("decoder",):
-                if which == "fupapel":
+                if which == "piratar":
+                    cfg = PiratarConfig.from_dict(piratar_shape(width, ff, heads, kv_heads, dim, vocab), max_tokens=max(4096, context + page))
+                elif which == "fupapel":
                     cfg = FupapelConfig.from_dict(fupapel_shape(width, ff, heads, kv_heads, dim, vocab, args.design_window),
                                                   max_tokens=max(4096, context + page))
                 elif which == "fapenex":
@@ -551,7 +581,7 @@ def main():
                     help="run a few steps between cudaProfilerStart/Stop (for ncu --profile-from-start off) and exit")
     ap.add_argument("--shape", default="2b", choices=["2b", "1b", "8b"],
                     help="layer sizes: 2b is the headline configuration; the others are for profiles and side measurements")
-    ap.add_argument("--design", default=None, choices=["sitelorn", "vunelix", "vipovik", "fapenex", "fupapel"],
+    ap.add_argument("--design", default=None, choices=["sitelorn", "vunelix", "vipovik", "fapenex", "fupapel", "piratar"],
                     help="instead of the benchmark: prefill and decode of this design at real layer sizes beside the decoder of equal size")
     ap.add_argument("--design-sizes", default="2k,4k", help="comma-separated names of " + ", ".join(sorted(DESIGN_SIZES)))
     ap.add_argument("--design-prompt", type=int, default=2048)

@@ -230,7 +230,8 @@ struct DecodeArgs {
     float cap_log2;                // a cap on the scores times log2(e): s <- cap tanh(s / cap) (0: none)
     int keep_first;                // with a window: keys at positions below this stay visible when the window has passed them
     const float *sink_w;
-    int gate_elem;                 // 1: the gate has one column per output element, gate[t, h dh + e]
+    int gate_elem;                 // 1: the gate has one column per output element, gate[t, h dv + e]
+    int dv;                        // size of a value head: v_pages [pages, nkvh, page_size, dv], out [T, nh, dv], part_acc [.., dv]
 };
 
 // cap tanh(s / cap) through one exponential and one quotient (both to about 1e-7 of their result: the sum of a capped
@@ -256,7 +257,7 @@ struct KeyRange {
 __device__ __forceinline__ float decode_finish(const DecodeArgs &a, float M, float L, int t, int h, int e) {
     if (a.sink) L += exp2f(jk_sink_log2(a.sink_w, h) - M);
     float f = 1.f / L;
-    if (a.gate != nullptr) f *= jk_sigmoid(a.gate[(size_t)t * a.gate_ld + (a.gate_elem ? (size_t)h * a.dh + e : (size_t)h)]);
+    if (a.gate != nullptr) f *= jk_sigmoid(a.gate[(size_t)t * a.gate_ld + (a.gate_elem ? (size_t)h * a.dv + e : (size_t)h)]);
     return f;
 }
 
@@ -477,13 +478,13 @@ __global__ void attention_combine_kernel(DecodeArgs a) {
         const float ms = a.part_ml[(base + s) * 2];
         if (ms > -INFINITY) L += exp2f(ms - M) * a.part_ml[(base + s) * 2 + 1];
     }
-    for (int e = threadIdx.x; e < a.dh; e += blockDim.x) {
+    for (int e = threadIdx.x; e < a.dv; e += blockDim.x) {
         float A = 0.f;
         for (int s = 0; s < a.splits; ++s) {
             const float ms = a.part_ml[(base + s) * 2];
-            if (ms > -INFINITY) A += exp2f(ms - M) * a.part_acc[(base + s) * a.dh + e];
+            if (ms > -INFINITY) A += exp2f(ms - M) * a.part_acc[(base + s) * a.dv + e];
         }
-        a.out[((size_t)t * a.nh + h) * a.dh + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h, e));
+        a.out[((size_t)t * a.nh + h) * a.dv + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h, e));
     }
 }
 
@@ -512,7 +513,7 @@ static int launch_decode(const DecodeArgs &a, cudaStream_t stream) {
 
 static int decode_gqa(const DecodeArgs &a, cudaStream_t stream, bool *taken);      // further down, beside its helpers
 
-// Scratch floats that `jk_attention_decode` needs for (nrows, nh, dh, splits).
+// Scratch floats that `jk_attention_decode` needs for (nrows, nh, size of a value head, splits).
 JK_EXPORT long long jk_attention_decode_scratch_floats(int nrows, int nh, int dh, int splits) {
     if (splits <= 1) return 0;
     return (long long)nrows * nh * splits * (dh + 2);
@@ -523,12 +524,15 @@ JK_EXPORT int jk_attention_decode(const void *q, const void *k_pages, const void
                                   const int *row_req, const int *block_table, int max_blocks,
                                   int page_size, int nh, int nkvh, int dh, float scale, int window,
                                   int splits, int sink, const float *gate, int gate_ld, float cap, int keep_first,
-                                  const float *sink_w, int gate_elem, cudaStream_t stream) {
+                                  const float *sink_w, int gate_elem, int dv, cudaStream_t stream) {
     if (nrows == 0) return JK_OK;
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dh : 1), "attention_decode: a gate row of %d holds no %d heads", gate_ld, nh);
+    if (dv <= 0) dv = dh;
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dv : 1), "attention_decode: a gate row of %d holds no %d heads", gate_ld, nh);
     JK_REQUIRE(cap >= 0.f && keep_first >= 0, "attention_decode: cap %g, %d kept keys", cap, keep_first);
     JK_REQUIRE(nrows > 0 && nh > 0 && nkvh > 0 && nh % nkvh == 0, "attention_decode: rows %d heads %d/%d", nrows, nh, nkvh);
     JK_REQUIRE(dh % 8 == 0 && dh >= 8 && dh <= 256, "attention_decode: head size %d (takes multiples of 8 up to 256)", dh);
+    JK_REQUIRE(dv == dh || (dh <= 128 && dv % 8 == 0 && dv >= 8 && dv <= 128),
+               "attention_decode: keys of %d and values of %d (unlike sizes are multiples of 8 up to 128)", dh, dv);
     JK_REQUIRE(page_size > 0 && max_blocks > 0, "attention_decode: page size %d, blocks %d, window %d",
                page_size, max_blocks, window);
     JK_REQUIRE(splits >= 1 && splits <= 256, "attention_decode: %d splits", splits);
@@ -536,11 +540,11 @@ JK_EXPORT int jk_attention_decode(const void *q, const void *k_pages, const void
     JK_REQUIRE(nrows <= 65535, "attention_decode: %d rows exceed one launch", nrows);
     DecodeArgs a{(const __nv_bfloat16 *)q, (const __nv_bfloat16 *)k_pages, (const __nv_bfloat16 *)v_pages,
                  (__nv_bfloat16 *)out, scratch,
-                 scratch ? scratch + (size_t)nrows * nh * splits * dh : nullptr,
+                 scratch ? scratch + (size_t)nrows * nh * splits * dv : nullptr,
                  rows, positions, row_req, block_table,
                  nrows, nh, nkvh, dh, page_size, max_blocks, window, splits, 0,
                  scale * 1.4426950408889634f, 0, sink, gate, gate_ld, cap * 1.4426950408889634f, window > 0 ? keep_first : 0,
-                 sink_w, gate_elem};
+                 sink_w, gate_elem, dv};
     const bool pow2 = (page_size & (page_size - 1)) == 0;
     while ((1 << a.page_shift) < page_size) ++a.page_shift;
     const int g = nh / nkvh;
@@ -859,13 +863,15 @@ __device__ __forceinline__ void cluster_sync_all() {      // every thread of eve
 // NW warps take 16 keys each of a tile of NW * 16 keys: four as a rule; eight (tiles of 128 keys, one block an SM with
 // heads of 128) for launches of so few blocks that every SM has at most one: a block's pace is set by the chain of a
 // tile's instructions in each warp, and twice the warps pass twice the keys in the same time.
-template <int DH, int NW>
+// Keys and values may differ in size: DK and DV are their sizes rounded up to 64 or 128, and the chunks of a row beyond a.dh and
+// a.dv are zeros in shared memory.
+template <int DK, int DV, int NW>
 __global__ void __launch_bounds__(NW * 32)
 attention_decode_gqa_kernel(DecodeArgs a) {
     constexpr int KEYS = NW * 16, NT = NW * 32;
-    static_assert(DH == 64 || DH == 128, "the swizzle chunk ^ (key & 7) needs rows of 8 or 16 chunks");
-    constexpr int CH = DH / 8;                     // 16-byte chunks of a key row
-    constexpr int TILE = KEYS * CH;             // uint4 per tile of keys (or values)
+    static_assert((DK == 64 || DK == 128) && (DV == 64 || DV == 128), "the swizzle chunk ^ (key & 7) needs rows of 8 or 16 chunks");
+    constexpr int CK = DK / 8, CV = DV / 8;        // 16-byte chunks of a key and of a value row
+    constexpr int TILE_K = KEYS * CK, STAGE = KEYS * (CK + CV);      // uint4 per tile of keys; per tile of keys and values
     extern __shared__ uint4 gq_smem[];
     pdl_trigger();
     const int split = blockIdx.x, kh = blockIdx.y % a.nkvh, ht = blockIdx.y / a.nkvh, ri = blockIdx.z;
@@ -900,9 +906,9 @@ attention_decode_gqa_kernel(DecodeArgs a) {
     const int ntiles = (k1 - k0 + KEYS - 1) / KEYS;
     const int *bt = a.block_table + (size_t)req * a.max_blocks;
 
-    // Where a tile's 64 keys lie (element offset of the key's row in the pages, -1 beyond the range) is worked out
+    // Where a tile's 64 keys lie (the key's row among the rows of the pages, -1 beyond the range) is worked out
     // once per tile by 64 threads into a table of two turns; the copies then cost a table read each.
-    long long *tab = reinterpret_cast<long long *>(gq_smem + (size_t)GQ_STAGES * 2 * TILE);       // [2][KEYS]
+    long long *tab = reinterpret_cast<long long *>(gq_smem + (size_t)GQ_STAGES * STAGE);       // [2][KEYS]
     // in two halves: the read of the block table is issued at the start of an iteration and used at its end, so
     // that the warp does not sit on it
     auto locate_begin = [&](int i) -> int {
@@ -913,25 +919,40 @@ attention_decode_gqa_kernel(DecodeArgs a) {
         if (threadIdx.x < KEYS) {
             const int kj = range.position(k0 + i * KEYS + threadIdx.x);
             tab[(i & 1) * KEYS + threadIdx.x] =
-                page < 0 ? -1 : (((long long)page * a.nkvh + kh) * a.page_size + kj % a.page_size) * DH;
+                page < 0 ? -1 : ((long long)page * a.nkvh + kh) * a.page_size + kj % a.page_size;
         }
     };
     auto locate_tile = [&](int i) { locate_end(i, locate_begin(i)); };
     // 16 bytes of key `key` of a tile lie at chunk ^ (key & 7): ldmatrix reads eight rows without conflicts.  A
-    // thread copies the same chunk of every (128 / CH)-th key, so its swizzled chunk never changes.
-    constexpr int KEYS_PER_PASS = NT / CH;
-    const int my_key = threadIdx.x / CH, my_ch = threadIdx.x % CH;
-    const int my_slot = my_key * CH + (my_ch ^ (my_key & 7));
+    // thread copies the same chunk of every (NT / chunks)-th key, so its swizzled chunk never changes.
+    constexpr int PASS_K = NT / CK, PASS_V = NT / CV;
+    const int key_k = threadIdx.x / CK, ch_k = threadIdx.x % CK, key_v = threadIdx.x / CV, ch_v = threadIdx.x % CV;
+    const int slot_k = key_k * CK + (ch_k ^ (key_k & 7)), slot_v = TILE_K + key_v * CV + (ch_v ^ (key_v & 7));
+    const bool has_k = ch_k * 8 < a.dh, has_v = ch_v * 8 < a.dv;
     auto load_tile = [&](int i) {
-        uint4 *kd = gq_smem + (size_t)(i % GQ_STAGES) * 2 * TILE + my_slot, *vd = kd + TILE;
-        const long long *where = tab + (i & 1) * KEYS + my_key;
+        uint4 *stage = gq_smem + (size_t)(i % GQ_STAGES) * STAGE;
+        const long long *where = tab + (i & 1) * KEYS;
+        if constexpr (DK == DV) {           // one look at a key's place for both rows
 #pragma unroll
-        for (int c = 0; c < KEYS / KEYS_PER_PASS; ++c) {
-            const long long off = where[c * KEYS_PER_PASS];
-            const bool valid = off >= 0;
-            const size_t src = valid ? (size_t)off + my_ch * 8 : 0;
-            cp_async16_or_zero(kd + c * KEYS_PER_PASS * CH, a.k_pages + src, valid);
-            cp_async16_or_zero(vd + c * KEYS_PER_PASS * CH, a.v_pages + src, valid);
+            for (int c = 0; c < KEYS / PASS_K; ++c) {
+                const long long row = where[c * PASS_K + key_k];
+                const bool vk = row >= 0 && has_k, vv = row >= 0 && has_v;
+                cp_async16_or_zero(stage + slot_k + c * PASS_K * CK, a.k_pages + (vk ? (size_t)row * a.dh + ch_k * 8 : 0), vk);
+                cp_async16_or_zero(stage + slot_v + c * PASS_K * CK, a.v_pages + (vv ? (size_t)row * a.dv + ch_k * 8 : 0), vv);
+            }
+        } else {
+#pragma unroll
+            for (int c = 0; c < KEYS / PASS_K; ++c) {
+                const long long row = where[c * PASS_K + key_k];
+                const bool valid = row >= 0 && has_k;
+                cp_async16_or_zero(stage + slot_k + c * PASS_K * CK, a.k_pages + (valid ? (size_t)row * a.dh + ch_k * 8 : 0), valid);
+            }
+#pragma unroll
+            for (int c = 0; c < KEYS / PASS_V; ++c) {
+                const long long row = where[c * PASS_V + key_v];
+                const bool valid = row >= 0 && has_v;
+                cp_async16_or_zero(stage + slot_v + c * PASS_V * CV, a.v_pages + (valid ? (size_t)row * a.dv + ch_v * 8 : 0), valid);
+            }
         }
     };
     locate_tile(0);
@@ -948,11 +969,12 @@ attention_decode_gqa_kernel(DecodeArgs a) {
     pdl_wait();
     {
         // the queries of the group's heads are one contiguous piece of q; heads beyond the group read as zeros
-        uint4 *qs = gq_smem + (size_t)GQ_STAGES * 2 * TILE + 2 * KEYS * sizeof(long long) / sizeof(uint4);
-        const uint4 *qg = reinterpret_cast<const uint4 *>(a.q + ((size_t)t * a.nh + h0) * DH);
-        for (int idx = threadIdx.x; idx < GQ_HEADS * CH; idx += NT) {
-            const int head = idx / CH, ch = idx % CH;
-            qs[head * CH + (ch ^ (head & 7))] = head < heads ? qg[idx] : make_uint4(0u, 0u, 0u, 0u);
+        uint4 *qs = gq_smem + (size_t)GQ_STAGES * STAGE + 2 * KEYS * sizeof(long long) / sizeof(uint4);
+        const uint4 *qg = reinterpret_cast<const uint4 *>(a.q + ((size_t)t * a.nh + h0) * a.dh);
+        const int chunks = a.dh / 8;
+        for (int idx = threadIdx.x; idx < GQ_HEADS * CK; idx += NT) {
+            const int head = idx / CK, ch = idx % CK;
+            qs[head * CK + (ch ^ (head & 7))] = head < heads && ch < chunks ? qg[head * chunks + ch] : make_uint4(0u, 0u, 0u, 0u);
         }
     }
     for (int i = first; i < GQ_STAGES - 1; ++i) {
@@ -962,23 +984,23 @@ attention_decode_gqa_kernel(DecodeArgs a) {
     __syncthreads();                               // the first tables have been read (and the queries are written)
     locate_tile(2);
     // the group's queries as A fragments: rows are heads (zero beyond the group), 16 dims per step; they came
-    // with the first tile's group of copies into their own 16 x DH corner of shared memory
-    unsigned qf[DH / 16][4];
+    // with the first tile's group of copies into their own 16 x DK corner of shared memory
+    unsigned qf[DK / 16][4];
     {
         cp_async_wait<GQ_STAGES - 2>();
         __syncthreads();
-        const uint4 *qs = gq_smem + (size_t)GQ_STAGES * 2 * TILE + 2 * KEYS * sizeof(long long) / sizeof(uint4);
+        const uint4 *qs = gq_smem + (size_t)GQ_STAGES * STAGE + 2 * KEYS * sizeof(long long) / sizeof(uint4);
         // matrices: (heads 0-7, dims 0-7), (heads 8-15, dims 0-7), (heads 0-7, dims 8-15), (heads 8-15, dims 8-15)
         const int head = (((lane >> 3) & 1) << 3) + (lane & 7);
 #pragma unroll
-        for (int kk = 0; kk < DH / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
             const int ch = kk * 2 + (lane >> 4);
-            ldmatrix_x4(qf[kk], qs + head * CH + (ch ^ (head & 7)));
+            ldmatrix_x4(qf[kk], qs + head * CK + (ch ^ (head & 7)));
         }
     }
-    float o[DH / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int n = 0; n < DH / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;      // heads lane / 4 and lane / 4 + 8
 
     for (int i = 0; i < ntiles; ++i) {
@@ -987,7 +1009,7 @@ attention_decode_gqa_kernel(DecodeArgs a) {
         const int page_ahead = locate_begin(i + GQ_STAGES);
         if (i + GQ_STAGES - 1 < ntiles) load_tile(i + GQ_STAGES - 1);
         cp_async_commit();
-        const uint4 *kt = gq_smem + (size_t)(i % GQ_STAGES) * 2 * TILE, *vt = kt + TILE;
+        const uint4 *kt = gq_smem + (size_t)(i % GQ_STAGES) * STAGE, *vt = kt + TILE_K;
         const int kw = k0 + i * KEYS + warp * 16;          // this warp's first key of the tile
         if (kw >= k1) {                                        // warp-uniform: no key of the tile is this warp's
             locate_end(i + GQ_STAGES, page_ahead);
@@ -997,9 +1019,9 @@ attention_decode_gqa_kernel(DecodeArgs a) {
         {
             float sd[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};      // odd steps: two chains of half the length
             const int key = warp * 16 + ((lane >> 4) << 3) + (lane & 7);
-            const uint4 *krow = kt + key * CH;
+            const uint4 *krow = kt + key * CK;
 #pragma unroll
-            for (int kk = 0; kk < DH / 16; ++kk) {
+            for (int kk = 0; kk < DK / 16; ++kk) {
                 // matrices: (keys 0-7, dims 0-7), (keys 0-7, dims 8-15), (keys 8-15, dims 0-7), (keys 8-15, dims 8-15)
                 const int ch = kk * 2 + ((lane >> 3) & 1);
                 unsigned b[4];
@@ -1048,14 +1070,14 @@ attention_decode_gqa_kernel(DecodeArgs a) {
         pa[2] = pack_bf16(p[1][0], p[1][1]); pa[3] = pack_bf16(p[1][2], p[1][3]);
         if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {           // a maximum moved: seldom after the first tiles
 #pragma unroll
-            for (int n = 0; n < DH / 8; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
+            for (int n = 0; n < DV / 8; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
         }
 #pragma unroll
-        for (int d2 = 0; d2 < DH / 16; ++d2) {
+        for (int d2 = 0; d2 < DV / 16; ++d2) {
             // transposed: (keys 0-7, dims 16 d2 ..+7), (keys 8-15, same dims), (keys 0-7, dims +8..+15), (keys 8-15, ...)
             const int key = warp * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), ch = d2 * 2 + (lane >> 4);
             unsigned b[4];
-            ldmatrix_x4_trans(b, vt + key * CH + (ch ^ (key & 7)));
+            ldmatrix_x4_trans(b, vt + key * CV + (ch ^ (key & 7)));
             mma_bf16(o[2 * d2], pa, b[0], b[1]);
             mma_bf16(o[2 * d2 + 1], pa, b[2], b[3]);
         }
@@ -1065,46 +1087,47 @@ attention_decode_gqa_kernel(DecodeArgs a) {
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     __syncthreads();                               // the ring is free: it carries the warps' results
-    // [warp][head][DH + 8]: the accumulator, then maximum and sum; with this stride the 8-byte stores of a half warp
+    // [warp][head][DV + 8]: the accumulator, then maximum and sum; with this stride the 8-byte stores of a half warp
     // (four heads, dims 0..7) fall into 32 different banks
-    constexpr int RS = DH + 8;
+    constexpr int RS = DV + 8;
     float *red = reinterpret_cast<float *>(gq_smem);
-    float *fin = red + NW * GQ_HEADS * RS, *fin_ml = fin + GQ_HEADS * DH;      // this block's result, for its cluster
+    float *fin = red + NW * GQ_HEADS * RS, *fin_ml = fin + GQ_HEADS * DV;      // this block's result, for its cluster
     {
         float *mine = red + (size_t)warp * GQ_HEADS * RS;
         const int r0 = lane >> 2, c0 = (lane & 3) * 2;
 #pragma unroll
-        for (int n = 0; n < DH / 8; ++n) {
+        for (int n = 0; n < DV / 8; ++n) {
             *reinterpret_cast<float2 *>(mine + r0 * RS + n * 8 + c0) = make_float2(o[n][0], o[n][1]);
             *reinterpret_cast<float2 *>(mine + (r0 + 8) * RS + n * 8 + c0) = make_float2(o[n][2], o[n][3]);
         }
         if ((lane & 3) == 0) {
-            *reinterpret_cast<float2 *>(mine + r0 * RS + DH) = make_float2(m0, l0);
-            *reinterpret_cast<float2 *>(mine + (r0 + 8) * RS + DH) = make_float2(m1, l1);
+            *reinterpret_cast<float2 *>(mine + r0 * RS + DV) = make_float2(m0, l0);
+            *reinterpret_cast<float2 *>(mine + (r0 + 8) * RS + DV) = make_float2(m1, l1);
         }
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < heads * DH; idx += NT) {
-        const int r = idx / DH, e = idx % DH;
+    for (int idx = threadIdx.x; idx < heads * DV; idx += NT) {
+        const int r = idx / DV, e = idx % DV;
+        if (e >= a.dv) continue;
         float M = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < NW; ++w) M = fmaxf(M, red[((size_t)w * GQ_HEADS + r) * RS + DH]);
+        for (int w = 0; w < NW; ++w) M = fmaxf(M, red[((size_t)w * GQ_HEADS + r) * RS + DV]);
         float L = 0.f, A = 0.f;
 #pragma unroll
         for (int w = 0; w < NW; ++w) {
             const float *src = red + ((size_t)w * GQ_HEADS + r) * RS;
-            const float f = M == -INFINITY ? 0.f : fast_exp2(src[DH] - M);      // a warp without keys: 2^-inf = 0
-            L += f * src[DH + 1];
+            const float f = M == -INFINITY ? 0.f : fast_exp2(src[DV] - M);      // a warp without keys: 2^-inf = 0
+            L += f * src[DV + 1];
             A += f * src[e];
         }
         if (a.cluster) {
-            fin[r * DH + e] = A;
+            fin[r * DV + e] = A;
             if (e == 0) { fin_ml[2 * r] = M; fin_ml[2 * r + 1] = L; }
         } else if (a.splits == 1) {
-            a.out[((size_t)t * a.nh + h0 + r) * DH + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, e));
+            a.out[((size_t)t * a.nh + h0 + r) * a.dv + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, e));
         } else {
             const size_t slot = pbase + (size_t)r * a.splits;
-            a.part_acc[slot * DH + e] = A;
+            a.part_acc[slot * a.dv + e] = A;
             if (e == 0) { a.part_ml[slot * 2] = M; a.part_ml[slot * 2 + 1] = L; }
         }
     }
@@ -1113,8 +1136,9 @@ attention_decode_gqa_kernel(DecodeArgs a) {
         // out of their shared memory and writes the row (the same sums, in the same order, as the merge kernel)
         cluster_sync_all();
         if (split == 0) {
-            for (int idx = threadIdx.x; idx < heads * DH; idx += NT) {
-                const int r = idx / DH;
+            for (int idx = threadIdx.x; idx < heads * DV; idx += NT) {
+                const int r = idx / DV, e = idx % DV;
+                if (e >= a.dv) continue;
                 float M = -INFINITY;
                 for (int p = 0; p < a.splits; ++p) M = fmaxf(M, ld_cluster_f32(fin_ml + 2 * r, p));
                 float L = 0.f, A = 0.f;
@@ -1126,22 +1150,22 @@ attention_decode_gqa_kernel(DecodeArgs a) {
                         A += f * ld_cluster_f32(fin + idx, p);
                     }
                 }
-                a.out[((size_t)t * a.nh + h0 + r) * DH + (idx % DH)] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, idx % DH));
+                a.out[((size_t)t * a.nh + h0 + r) * a.dv + e] = __float2bfloat16_rn(A * decode_finish(a, M, L, t, h0 + r, e));
             }
         }
         cluster_sync_all();                        // nobody leaves while its shared memory may still be read
     }
 }
 
-template <int DH, int NW>
+template <int DK, int DV, int NW>
 static int launch_decode_gqa_warps(const DecodeArgs &a, int sms, cudaStream_t stream) {
     constexpr int KEYS = NW * 16;
     const int g = a.nh / a.nkvh;
-    const size_t ring = (size_t)GQ_STAGES * 2 * KEYS * DH * sizeof(__nv_bfloat16) + 2 * KEYS * sizeof(long long)
-                        + (size_t)GQ_HEADS * DH * sizeof(__nv_bfloat16);       // tiles, the two tables, the queries
-    const size_t merge = (size_t)NW * GQ_HEADS * (DH + 8) * sizeof(float) + (size_t)GQ_HEADS * (DH + 2) * sizeof(float);
+    const size_t ring = (size_t)GQ_STAGES * KEYS * (DK + DV) * sizeof(__nv_bfloat16) + 2 * KEYS * sizeof(long long)
+                        + (size_t)GQ_HEADS * DK * sizeof(__nv_bfloat16);       // tiles, the two tables, the queries
+    const size_t merge = (size_t)NW * GQ_HEADS * (DV + 8) * sizeof(float) + (size_t)GQ_HEADS * (DV + 2) * sizeof(float);
     const size_t smem = ring > merge ? ring : merge;
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_gqa_kernel<DH, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_gqa_kernel<DK, DV, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "attention_decode: %s", cudaGetErrorString(e));
     dim3 grid(a.splits, a.nkvh * ((g + GQ_HEADS - 1) / GQ_HEADS), a.nrows);
     // Measured: with heads of 64 (52 KB of shared memory a block) clusters of two are faster than the merge kernel
@@ -1150,15 +1174,15 @@ static int launch_decode_gqa_warps(const DecodeArgs &a, int sms, cudaStream_t st
     // heads of 128, wait for whole groups of free SMs and lose more than the merge kernel costs (37.6 against 30.9 us;
     // the blocks of eight warps, 203 KB each, in clusters of eight: 36.1 against 15.0 us at 8 rows x 4,096 keys).
     const long long blocks = (long long)grid.x * grid.y * grid.z;
-    if (DH == 64 && NW == 4 && a.splits >= 2 && a.splits <= 8 && (a.splits == 2 || blocks <= 2LL * sms)) {
+    if (DK == 64 && DV == 64 && NW == 4 && a.splits >= 2 && a.splits <= 8 && (a.splits == 2 || blocks <= 2LL * sms)) {
         // the splits are one cluster and merge through distributed shared memory: no merge kernel, no scratch
         DecodeArgs c = a;
         c.cluster = 1;
-        const cudaError_t err = jk_launch_clusters(attention_decode_gqa_kernel<DH, NW>, a.splits, grid, dim3(NW * 32), smem, stream, c);
+        const cudaError_t err = jk_launch_clusters(attention_decode_gqa_kernel<DK, DV, NW>, a.splits, grid, dim3(NW * 32), smem, stream, c);
         if (err != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "attention_decode_gqa (clusters of %d): %s", a.splits, cudaGetErrorString(err));
         return JK_OK;
     }
-    jk_launch(attention_decode_gqa_kernel<DH, NW>, grid, dim3(NW * 32), smem, stream, a);
+    jk_launch(attention_decode_gqa_kernel<DK, DV, NW>, grid, dim3(NW * 32), smem, stream, a);
     JK_CHECK_LAUNCH("attention_decode_gqa");
     if (a.splits > 1) {
         jk_launch(attention_combine_kernel, dim3(a.nh, a.nrows), dim3(64), 0, stream, a);
@@ -1167,7 +1191,7 @@ static int launch_decode_gqa_warps(const DecodeArgs &a, int sms, cudaStream_t st
     return JK_OK;
 }
 
-template <int DH>
+template <int DK, int DV>
 static int launch_decode_gqa(const DecodeArgs &a, cudaStream_t stream) {
     static int sms = 0;
     if (sms == 0) {
@@ -1180,20 +1204,25 @@ static int launch_decode_gqa(const DecodeArgs &a, cudaStream_t stream) {
     // (Heads of 64 gain less and not everywhere: 8 key/value heads, one row, 4,096 keys at 8 cuts 10.7 -> 8.2 us, but a
     // step of that shape at 512 keys loses 3 %, and where the cuts would have to be halved for it, 36 heads and two
     // rows, 20.4 -> 22.2 us: they keep blocks of four warps, whose cuts merge inside clusters.)
-    if (DH == 128 && blocks <= sms && !wide_off) return launch_decode_gqa_warps<DH, 8>(a, sms, stream);
-    return launch_decode_gqa_warps<DH, 4>(a, sms, stream);
+    if ((DK == 128 || DV == 128) && blocks <= sms && !wide_off) return launch_decode_gqa_warps<DK, DV, 8>(a, sms, stream);
+    return launch_decode_gqa_warps<DK, DV, 4>(a, sms, stream);
 }
 
 // Head sizes 64 and 128 go to the tensor-core decode kernel, which reads keys and values once per group of query
 // heads: measured against the kernel of the CUDA cores it is 1.1 times as fast without groups, 1.4 to 2 times at groups
-// of 2 to 4 and five times at 16 (JK_GQA_MIN_GROUP=n keeps groups below n on the old kernel).  Other head sizes stay there.
+// of 2 to 4 and five times at 16 (JK_GQA_MIN_GROUP=n keeps groups below n on the old kernel).  Other head sizes stay there, unless
+// keys and values differ in size: those always come here, padded to 64 or 128.
 static int decode_gqa(const DecodeArgs &a, cudaStream_t stream, bool *taken) {
     *taken = true;
     static const int min_group = [] { const char *v = getenv("JK_GQA_MIN_GROUP"); return v ? atoi(v) : 1; }();
+    if (a.dv != a.dh) {
+        if (a.dh <= 64) return a.dv <= 64 ? launch_decode_gqa<64, 64>(a, stream) : launch_decode_gqa<64, 128>(a, stream);
+        return a.dv <= 64 ? launch_decode_gqa<128, 64>(a, stream) : launch_decode_gqa<128, 128>(a, stream);
+    }
     if (a.nh / a.nkvh >= min_group) {
         switch (a.dh) {
-            case 64: return launch_decode_gqa<64>(a, stream);       // rows of 8 or 16 chunks: what the swizzle takes
-            case 128: return launch_decode_gqa<128>(a, stream);
+            case 64: return launch_decode_gqa<64, 64>(a, stream);       // rows of 8 or 16 chunks: what the swizzle takes
+            case 128: return launch_decode_gqa<128, 128>(a, stream);
         }
     }
     *taken = false;
@@ -1287,5 +1316,5 @@ JK_EXPORT int jk_attention_decode_static(const void *q, const void *k_pages, con
     // every partial slot that the merge kernel reads is written by the split kernel of this same call,
     // so what an earlier call left in the array needs no clearing
     return jk_attention_decode(q, k_pages, v_pages, out, need ? scratch : nullptr, rows, nrows, positions, row_req,
-                               block_table, max_blocks, page_size, nh, nkvh, dh, scale, window, splits, 0, nullptr, 0, 0.f, 0, nullptr, 0, stream);
+                               block_table, max_blocks, page_size, nh, nkvh, dh, scale, window, splits, 0, nullptr, 0, 0.f, 0, nullptr, 0, dh, stream);
 }

@@ -34,6 +34,7 @@
 // (reference: the per-request loop of two batched products and a causal softmax over a materialised
 // score buffer, src/models/jiuge/jiuge.cpp:206-233.)
 #include "common.cuh"
+#include "host_rules.h"
 
 #include <cuda.h>
 #include <map>
@@ -51,7 +52,7 @@ constexpr float AT_RESCALE_THRESHOLD = 8.f;      // in log2 units
 constexpr int AT_POLY_OF_8 = 2;
 
 struct AtArgs {
-    __nv_bfloat16 *out;       // [T, nh, dh]
+    __nv_bfloat16 *out;       // [T, nh, dv]
     const int *tiles;         // [ntiles][2]: batch entry, first row of the tile (row index in the step); most keys first
     const int *req_start;     // [nreq + 1]
     const int *req_pos;       // [nreq]
@@ -65,6 +66,7 @@ struct AtArgs {
     float cap_raw;            // a cap on the scores divided by the softmax scale: raw s <- cap tanh(s / cap) (0: none)
     int keep_first;           // with a window: keys at positions below this stay visible when the window has passed them
     const float *sink_w;
+    int dk, dv;               // sizes of a key and of a value head (DK and DV are these rounded up to 64 or 128)
 };
 
 // ---- PTX wrappers (see gemm_tcgen05.cu for the same set) -----------------------------------------
@@ -218,11 +220,11 @@ __host__ __device__ constexpr unsigned instr_desc(int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn ? 1u : 0u) << 16) | ((unsigned)(n >> 3) << 17) | ((unsigned)(AT_BM >> 4) << 24);
 }
 
-template <int DH> struct AtSmem {
-    static constexpr int SUB = DH / 64;                       // 64-wide sub-tiles along the head
-    __nv_bfloat16 q[SUB][AT_BM * 64];                         // K-major, per sub-tile [128 rows][64]
-    __nv_bfloat16 k[2][SUB][AT_BN * 64];                      // two stages
-    __nv_bfloat16 v[2][SUB][AT_BN * 64];
+template <int DK, int DV> struct AtSmem {
+    static constexpr int SUB_K = DK / 64, SUB_V = DV / 64;    // 64-wide sub-tiles along the head
+    __nv_bfloat16 q[SUB_K][AT_BM * 64];                       // K-major, per sub-tile [128 rows][64]
+    __nv_bfloat16 k[2][SUB_K][AT_BN * 64];                    // two stages
+    __nv_bfloat16 v[2][SUB_V][AT_BN * 64];
     __nv_bfloat16 p[2][AT_BM * 64];                           // [128 rows][128 keys] as two sub-tiles of 64 keys
     unsigned long long q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full, s_free, p_ready, pv_done, met[4];
     unsigned tmem_base;
@@ -230,14 +232,17 @@ template <int DH> struct AtSmem {
 
 // ELEM: the gate, if there is one, has a column per output element (an instance of its own, so that the others carry neither
 // its code nor its registers)
-template <int DH, bool ELEM>
-__global__ void __launch_bounds__(AT_THREADS, DH <= 64 ? 2 : 1)
+// Keys and values may differ in size.  Heads of dk or dv elements that are no multiple of 64 run as ones of DK or DV: TMA fills what
+// lies beyond a cached row with zeros (of a query row it brings the next head's elements, which meet the keys' zeros), and columns
+// of the output beyond dv are not written.
+template <int DK, int DV, bool ELEM>
+__global__ void __launch_bounds__(AT_THREADS, DK <= 64 && DV <= 64 ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, AtArgs a) {
-    constexpr int SUB = DH / 64;
-    constexpr unsigned TMEM_COLS = DH <= 64 ? 256 : 512;      // S: 128 columns; two accumulators of DH columns
+    constexpr int SUB_K = DK / 64, SUB_V = DV / 64;
+    constexpr unsigned TMEM_COLS = DV <= 64 ? 256 : 512;      // S: 128 columns; two accumulators of DV columns
     extern __shared__ __align__(1024) unsigned char at_raw[];      // swizzled tiles need 1024-byte alignment
-    AtSmem<DH> &s = *reinterpret_cast<AtSmem<DH> *>(at_raw);
+    AtSmem<DK, DV> &s = *reinterpret_cast<AtSmem<DK, DV> *>(at_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (smem_u32(at_raw) & 1023u) {                            // never seen; a wrong result is not an option
         if (threadIdx.x == 0) atomicExch(a.status, 14);
@@ -285,19 +290,22 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (warp == 0) {
         // ---- TMA producer: the whole warp; lane = (page of the tile, 64-wide part of the head) ----
         if (lane == 0) {
-            mbar_expect_tx(&s.q_full, AT_BM * DH * 2);
-            for (int u = 0; u < SUB; ++u) tma_load_2d(s.q[u], &map_q, &s.q_full, h * DH + u * 64, row0);
+            mbar_expect_tx(&s.q_full, AT_BM * DK * 2);
+            for (int u = 0; u < SUB_K; ++u) tma_load_2d(s.q[u], &map_q, &s.q_full, h * a.dk + u * 64, row0);
         }
-        const int boxes = pages_per_tile * SUB;                 // at most 16 pages x 2 parts
         for (int i = 0; i < n_kv && !failed; ++i) {
             const int st = i & 1, kv0 = tile_at(i);
-            // this lane's page of the tile, read from the block table once for keys and values;
+            // this lane's page of the tile, read from the block table once for keys and values of one size;
             // a page beyond what the request holds is never looked at: its keys are masked
-            const int pg = lane / SUB, u = lane % SUB;
-            const int blk = kv0 / a.page_size + pg;
-            const int page = (lane < boxes && blk < a.max_blocks) ? bt[blk] : 0;
-            const int grow = (page * a.nkvh + hk) * a.page_size;
+            int pg = lane / SUB_K, u = lane % SUB_K;
+            auto first_row = [&]() {
+                const int blk = kv0 / a.page_size + pg;
+                const int page = (pg < pages_per_tile && blk < a.max_blocks) ? bt[blk] : 0;
+                return (page * a.nkvh + hk) * a.page_size;
+            };
+            int grow = first_row();
             for (int kind = 0; kind < 2; ++kind) {               // 0: keys, 1: values
+                if (SUB_K != SUB_V && kind == 1) { pg = lane / SUB_V; u = lane % SUB_V; grow = first_row(); }
                 unsigned long long *empty = kind ? &s.v_empty[st] : &s.k_empty[st];
                 unsigned long long *full = kind ? &s.v_full[st] : &s.k_full[st];
                 int ok = 1;
@@ -306,9 +314,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     ok = __shfl_sync(0xffffffffu, ok, 0);
                 }
                 if (!ok) { failed = 1; break; }
-                if (lane == 0) mbar_expect_tx(full, AT_BN * DH * 2);
+                if (lane == 0) mbar_expect_tx(full, AT_BN * (kind ? DV : DK) * 2);
                 __syncwarp();
-                if (lane < boxes) {
+                if (pg < pages_per_tile) {                       // at most 16 pages x 2 parts
                     __nv_bfloat16 *dst = (kind ? s.v[st][u] : s.k[st][u]) + pg * a.page_size * 64;
                     tma_load_2d(dst, kind ? &map_v : &map_k, full, u * 64, grow);
                 }
@@ -318,20 +326,20 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     } else if (warp == 1) {
         // ---- product issuer ----
         if (lane == 0) {
-            constexpr unsigned idesc_qk = instr_desc(AT_BN, false), idesc_pv = instr_desc(DH, true);
+            constexpr unsigned idesc_qk = instr_desc(AT_BN, false), idesc_pv = instr_desc(DV, true);
             // descriptor words, built once: low = start address and leading offset, high = stride
             // offset 1024, version 1, 128-byte swizzle
             constexpr unsigned desc_hi = (1024u >> 4) | (1u << 14) | (2u << 29);
             auto lo_k = [](const void *tile) { return ((smem_u32(tile) & 0x3FFFFu) >> 4) | (1u << 16); };
             auto lo_mn = [](const void *tile) { return ((smem_u32(tile) & 0x3FFFFu) >> 4) | ((unsigned)((AT_BN * 64 * 2) >> 4) << 16); };
-            unsigned q_lo[SUB], k_lo[2][SUB], p_lo[2], v_lo[2];
+            unsigned q_lo[SUB_K], k_lo[2][SUB_K], p_lo[2], v_lo[2];
 #pragma unroll
-            for (int u = 0; u < SUB; ++u) { q_lo[u] = lo_k(s.q[u]); k_lo[0][u] = lo_k(s.k[0][u]); k_lo[1][u] = lo_k(s.k[1][u]); }
+            for (int u = 0; u < SUB_K; ++u) { q_lo[u] = lo_k(s.q[u]); k_lo[0][u] = lo_k(s.k[0][u]); k_lo[1][u] = lo_k(s.k[1][u]); }
             p_lo[0] = lo_k(s.p[0]); p_lo[1] = lo_k(s.p[1]);
             v_lo[0] = lo_mn(s.v[0][0]); v_lo[1] = lo_mn(s.v[1][0]);
             auto issue_qk = [&](int st) {
 #pragma unroll
-                for (int u = 0; u < SUB; ++u)
+                for (int u = 0; u < SUB_K; ++u)
 #pragma unroll
                     for (int k = 0; k < 4; ++k)          // 16 of the head's elements per instruction: 32 bytes further
                         umma_bf16_words(tmem_s, q_lo[u] + 2 * k, desc_hi, (st ? k_lo[1][u] : k_lo[0][u]) + 2 * k, desc_hi,
@@ -363,7 +371,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 for (int k = 0; k < AT_BN / 16; ++k) {   // 16 keys per instruction
                     // P: 32 bytes further in the row of sub-tile k / 4; V: 16 rows of 128 bytes further.
                     // Keys 0..63 of the tile add to the first accumulator, keys 64..127 to the second.
-                    umma_bf16_words(tmem_o + (k / 4) * DH, p_lo[k / 4] + 2 * (k % 4), desc_hi,
+                    umma_bf16_words(tmem_o + (k / 4) * DV, p_lo[k / 4] + 2 * (k % 4), desc_hi,
                                     (st ? v_lo[1] : v_lo[0]) + ((k * 16 * 128) >> 4), desc_hi, idesc_pv, (i | (k % 4)) ? 1u : 0u);
                 }
                 umma_commit(&s.pv_done);
@@ -382,7 +390,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         const int lo_row = jk_mask_lo(pos, a.window);
         const unsigned lane_addr = (unsigned)(quarter * 32) << 16;
         const unsigned tmem_sh = tmem_s + lane_addr + half * AT_HALF;     // this thread's scores
-        const unsigned tmem_oh = tmem_o + lane_addr + half * DH;          // this half's accumulator
+        const unsigned tmem_oh = tmem_o + lane_addr + half * DV;          // this half's accumulator
         float m_ref = -INFINITY, l = 0.f;                      // reference maximum (scaled, log2 units) and sum
         bool alive = true;
         for (int i = 0; i < n_kv; ++i) {
@@ -457,7 +465,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             if (__any_sync(0xffffffffu, factor != 1.f) && i > 0) {
                 // rescale this warp's rows of its accumulator (rows that keep their reference multiply by 1)
 #pragma unroll 1
-                for (int c = 0; c < DH / 32; ++c) {
+                for (int c = 0; c < DV / 32; ++c) {
                     unsigned ov[32];
                     tmem_ld32(tmem_oh + c * 32, ov);
 #pragma unroll
@@ -480,7 +488,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 if (!__all_sync(0xffffffffu, mbar_wait(&s.v_full[i & 1], (i >> 1) & 1))) { alive = false; break; }
                 if (tile_at(i) + row > p_last) {
 #pragma unroll
-                    for (int u = 0; u < SUB; ++u) {
+                    for (int u = 0; u < SUB_V; ++u) {
                         uint4 *vrow = reinterpret_cast<uint4 *>(s.v[i & 1][u] + row * 64);      // 128 bytes; the swizzle stays inside
 #pragma unroll
                         for (int c = 0; c < 8; ++c) vrow[c] = make_uint4(0u, 0u, 0u, 0u);
@@ -511,19 +519,21 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             // a sink adds its term 2^(sink - m_all); a gate multiplies the row's output
             float inv = 1.f / (l * w_mine + other.y * w_other + (a.sink ? exp2f(jk_sink_log2(a.sink_w, h) - m_all) : 0.f));
             if (!ELEM && a.gate != nullptr && row < nrows) inv *= jk_sigmoid(a.gate[(size_t)(row0 + row) * a.gate_ld + h]);
-            const float *gate = ELEM && row < nrows ? a.gate + (size_t)(row0 + row) * a.gate_ld + (size_t)h * DH + half * (DH / 2) : nullptr;   // of this thread's columns
+            const float *gate = ELEM && row < nrows ? a.gate + (size_t)(row0 + row) * a.gate_ld + (size_t)h * a.dv + half * (DV / 2) : nullptr;   // of this thread's columns
             const float w0 = (half ? w_other : w_mine) * inv, w1 = (half ? w_mine : w_other) * inv;
-            // this thread writes columns [half * DH / 2, + DH / 2) of its row
-            __nv_bfloat16 *dst = a.out + ((size_t)(row0 + row) * a.nh + h) * DH + half * (DH / 2);
+            // this thread writes columns [half * DV / 2, + DV / 2) of its row, as far as the head has them
+            __nv_bfloat16 *dst = a.out + ((size_t)(row0 + row) * a.nh + h) * a.dv + half * (DV / 2);
+            const int mine = a.dv - half * (DV / 2);
 #pragma unroll 1
-            for (int c = 0; c < DH / 64; ++c) {
+            for (int c = 0; c < DV / 64; ++c) {
                 unsigned o0[32], o1[32];
-                tmem_ld32_issue(tmem_o + lane_addr + half * (DH / 2) + c * 32, o0);
-                tmem_ld32_issue(tmem_o + lane_addr + DH + half * (DH / 2) + c * 32, o1);
+                tmem_ld32_issue(tmem_o + lane_addr + half * (DV / 2) + c * 32, o0);
+                tmem_ld32_issue(tmem_o + lane_addr + DV + half * (DV / 2) + c * 32, o1);
                 tmem_wait_ld();
                 if (row < nrows) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
+                        if (c * 32 + j >= mine) break;
                         unsigned w[4];
                         float z[ELEM ? 8 : 1];
                         if constexpr (ELEM) {
@@ -609,12 +619,12 @@ JK_EXPORT int jk_attention_tcgen05_supports(int dh, int page_size) {
     return (dh == 64 || dh == 128) && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64 || page_size == 128);
 }
 
-template <int DH, bool ELEM>
+template <int DK, int DV, bool ELEM>
 static int launch_at(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const AtArgs &a, cudaStream_t stream) {
-    const size_t smem = sizeof(AtSmem<DH>);
-    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<DH, ELEM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = sizeof(AtSmem<DK, DV>);
+    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<DK, DV, ELEM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) JK_FAIL(JK_CUDA_ERROR, "attention_tcgen05: %s", cudaGetErrorString(e));
-    jk_launch(attention_tcgen05_kernel<DH, ELEM>, dim3(a.nh, a.ntiles), dim3(AT_THREADS), smem, stream, mq, mk, mv, a);
+    jk_launch(attention_tcgen05_kernel<DK, DV, ELEM>, dim3(a.nh, a.ntiles), dim3(AT_THREADS), smem, stream, mq, mk, mv, a);
     JK_CHECK_LAUNCH("attention_tcgen05");
     return JK_OK;
 }
@@ -623,21 +633,28 @@ JK_EXPORT int jk_attention_tcgen05(const void *q, const void *k_pages, const voi
                                    int ntiles, int ntok, const int *req_start, const int *req_pos, const int *block_table,
                                    int max_blocks, int num_pages, int page_size, int nh, int nkvh, int dh, float scale,
                                    int window, int *status, int sink, const float *gate, int gate_ld, float cap, int keep_first,
-                                   const float *sink_w, int gate_elem, cudaStream_t stream) {
+                                   const float *sink_w, int gate_elem, int dv, cudaStream_t stream) {
     if (ntiles == 0) return JK_OK;
-    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dh : 1), "attention_tcgen05: a gate row of %d holds no %d heads", gate_ld, nh);
-    JK_REQUIRE(jk_attention_tcgen05_supports(dh, page_size), "attention_tcgen05: head size %d with pages of %d is not built", dh, page_size);
+    if (dv <= 0) dv = dh;
+    JK_REQUIRE(gate == nullptr || gate_ld >= nh * (gate_elem ? dv : 1), "attention_tcgen05: a gate row of %d holds no %d heads", gate_ld, nh);
+    JK_REQUIRE(jk::attention_tcgen05_takes(dh, page_size, dv), "attention_tcgen05: keys of %d and values of %d with pages of %d are not built", dh, dv, page_size);
     JK_REQUIRE(ntiles > 0 && nh > 0 && nkvh > 0 && nh % nkvh == 0 && ntiles <= 65535, "attention_tcgen05: tiles %d heads %d/%d", ntiles, nh, nkvh);
     JK_REQUIRE(max_blocks > 0 && status != nullptr && num_pages > 0, "attention_tcgen05: bad arguments");
     CUtensorMap mq, mk, mv;
     if (int rc = tensor_map(q, ntok, nh * dh, AT_BM, &mq)) return rc;
     if (int rc = tensor_map(k_pages, (long long)num_pages * nkvh * page_size, dh, page_size, &mk)) return rc;
-    if (int rc = tensor_map(v_pages, (long long)num_pages * nkvh * page_size, dh, page_size, &mv)) return rc;
+    if (int rc = tensor_map(v_pages, (long long)num_pages * nkvh * page_size, dv, page_size, &mv)) return rc;
     AtArgs a{(__nv_bfloat16 *)out, tiles, req_start, req_pos, block_table, status,
              ntiles, nh, nkvh, page_size, max_blocks, window, scale * 1.4426950408889634f, sink, gate, gate_ld,
-             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w};
+             cap > 0.f ? cap / scale : 0.f, window > 0 ? keep_first : 0, sink_w, dh, dv};
     JK_REQUIRE(cap >= 0.f && keep_first >= 0 && scale > 0.f, "attention_tcgen05: cap %g, %d kept keys, scale %g", cap, keep_first, scale);
     const bool elem = gate != nullptr && gate_elem;
-    if (dh == 64) return elem ? launch_at<64, true>(mq, mk, mv, a, stream) : launch_at<64, false>(mq, mk, mv, a, stream);
-    return elem ? launch_at<128, true>(mq, mk, mv, a, stream) : launch_at<128, false>(mq, mk, mv, a, stream);
+#define LAUNCH_AT(DK, DV) return elem ? launch_at<DK, DV, true>(mq, mk, mv, a, stream) : launch_at<DK, DV, false>(mq, mk, mv, a, stream)
+    if (dh <= 64) {
+        if (dv <= 64) LAUNCH_AT(64, 64);
+        LAUNCH_AT(64, 128);
+    }
+    if (dv <= 64) LAUNCH_AT(128, 64);
+    LAUNCH_AT(128, 128);
+#undef LAUNCH_AT
 }

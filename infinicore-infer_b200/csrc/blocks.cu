@@ -151,7 +151,7 @@ JK_EXPORT int jk_norm_add(const float *delta, float *x, const float *w, float ep
     if (rows <= 64 && vec) threads = std::min(1024, std::max(threads, (d / 4 + 31) / 32 * 32));
 #define LAUNCH_V(T, V)                                                                                                              \
     do {                                                                                                                            \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(norm_add_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(norm_add_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         jk_launch(norm_add_kernel<T, V>, dim3(rows), dim3(threads), smem, stream, delta, x, w, eps, w_next, eps2, (T *)out, w_next2, (T *)out2, d);   \
     } while (0)
 #define LAUNCH(T) if (vec) LAUNCH_V(T, true); else LAUNCH_V(T, false)
@@ -1273,7 +1273,7 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
         JK_REQUIRE(grid.y <= 65535, "latent_attention: %d heads", H);
 #define LAUNCH_TC(NT_)                                                                                                                       \
     do {                                                                                                                                    \
-        if (smem_tc > 48 * 1024) cudaFuncSetAttribute(latent_attention_tc_kernel<NT_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_tc); \
+        if (smem_tc > 46 * 1024) cudaFuncSetAttribute(latent_attention_tc_kernel<NT_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_tc); \
         jk_launch(latent_attention_tc_kernel<NT_>, grid, dim3(256), smem_tc, stream, ta);                                                   \
     } while (0)
         if (NT == 2) LAUNCH_TC(2); else if (NT == 4) LAUNCH_TC(4); else if (NT == 8) LAUNCH_TC(8); else LAUNCH_TC(16);
@@ -1292,7 +1292,7 @@ JK_EXPORT int jk_latent_attention(const void *q, const void *pages, void *out, f
     dim3 grid((H + LA_WARPS - 1) / LA_WARPS, T, splits);
 #define LAUNCH_NS(TT, NS)                                                                                                                   \
     do {                                                                                                                                    \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(latent_attention_kernel<TT, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(latent_attention_kernel<TT, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         jk_launch(latent_attention_kernel<TT, NS>, grid, dim3(LA_WARPS * 32), smem, stream, a);                                             \
     } while (0)
 #define LAUNCH(TT)                                  \
@@ -1586,7 +1586,7 @@ JK_EXPORT int jk_selective_scan(const float *x, const float *low, int ld_low, in
     const size_t smem = (size_t)SS_CHUNK * (2 * SS_CHANNELS + SS_THREADS + 2 * N) * sizeof(float);
 #define LAUNCH_N(TT, NPER)                                                                                                                  \
     do {                                                                                                                                    \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(selective_scan_kernel<TT, NPER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(selective_scan_kernel<TT, NPER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         jk_launch(selective_scan_kernel<TT, NPER>, grid, dim3(SS_THREADS), smem, stream, a);                                                \
     } while (0)
 #define LAUNCH(TT)                              \
@@ -2072,8 +2072,8 @@ JK_EXPORT int jk_routed_experts(const void *h, const float *router, const void *
     if (stream_rows) {
         const size_t elem = dtype == JK_F32 ? 4 : 2, smem_up = (size_t)ER_ROWS * D * elem, smem_down = (size_t)ER_ROWS * ff * elem;
 #define LAUNCH(TT)                                                                                                                           \
-    if (smem_up > 48 * 1024) cudaFuncSetAttribute(expert_rows_kernel<TT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_up);  \
-    if (smem_down > 48 * 1024) cudaFuncSetAttribute(expert_rows_kernel<TT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_down); \
+    if (smem_up > 46 * 1024) cudaFuncSetAttribute(expert_rows_kernel<TT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_up);  \
+    if (smem_down > 46 * 1024) cudaFuncSetAttribute(expert_rows_kernel<TT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_down); \
     jk_launch(expert_rows_kernel<TT, true>, dim3(E, (ff + ER_FEATURES - 1) / ER_FEATURES), dim3(256), smem_up, stream, (const TT *)h,        \
               (const TT *)w_gate_up, act, D, ff, E, (const int *)starts, (const int *)entry_row, in_score, actf, limit);          \
     jk_launch(expert_rows_kernel<TT, false>, dim3(E, (D + ER_FEATURES - 1) / ER_FEATURES), dim3(256), smem_down, stream, (const TT *)act,    \
@@ -2234,7 +2234,7 @@ JK_EXPORT int jk_embed_pair(const int *tokens, const int *positions, const int *
     const int threads = T <= 64 ? std::min(1024, std::max(128, (d / 2 + 31) / 32 * 32)) : (d >= 1024 ? 256 : 128);
 #define LAUNCH(TT)                                                                                                                     \
     do {                                                                                                                               \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(embed_pair_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(embed_pair_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
         jk_launch(embed_pair_kernel<TT>, dim3(T), dim3(threads), smem, stream, a);                                                     \
     } while (0)
     BLOCKS_BY_DTYPE(dtype, "embed_pair", LAUNCH);
@@ -2574,7 +2574,7 @@ JK_EXPORT int jk_gated_recurrence(const float *u, const void *w_r, const void *w
         const dim3 grid((g.n + GR_CHANNELS - 1) / GR_CHANNELS, blocks, (T + GR_ROWS - 1) / GR_ROWS);
 #define LAUNCH(TT)                                                                                                                     \
     do {                                                                                                                               \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(gated_rows_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(gated_rows_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
         jk_launch(gated_rows_kernel<TT>, grid, dim3(256), smem, stream, g);                                                            \
     } while (0)
         BLOCKS_BY_DTYPE(dtype, "gated_rows", LAUNCH);

@@ -62,7 +62,7 @@ JK_HOST_EXPORT long long jk_decode_scratch_floats(int nrows, int nh, int dh, int
     return jk::decode_scratch_floats(nrows, nh, dh, splits);
 }
 JK_HOST_EXPORT int jk_decode_keys_hint(int context, int window) { return jk::decode_keys_hint(context, window); }
-JK_HOST_EXPORT int jk_attention_tcgen05_takes(int dh, int page_size) { return jk::attention_tcgen05_takes(dh, page_size) ? 1 : 0; }
+JK_HOST_EXPORT int jk_attention_tcgen05_takes(int dh, int page_size, int dv) { return jk::attention_tcgen05_takes(dh, page_size, dv) ? 1 : 0; }
 JK_HOST_EXPORT int jk_context_bucket(int longest, int max_positions) { return jk::context_bucket(longest, max_positions); }
 // routing[0..5]: sms, tcgen05_min_rows, tcgen05_min_tiles, tcgen05_min_fill_pct, skinny_min_blocks, library_only
 static jk::Routing routing_of(const int *v) {

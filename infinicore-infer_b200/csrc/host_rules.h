@@ -222,9 +222,12 @@ inline int decode_keys_hint(int context, int window) {
     return std::max(1, reach / 2);
 }
 // floats of scratch that `splits` cuts of `nrows` rows need (partial outputs, maxima and sums); none for one cut
-inline long long decode_scratch_floats(int nrows, int nh, int dh, int splits) {
-    return splits <= 1 ? 0 : (long long)nrows * nh * splits * (dh + 2);
+// (`dv`: the size of a value head)
+inline long long decode_scratch_floats(int nrows, int nh, int dv, int splits) {
+    return splits <= 1 ? 0 : (long long)nrows * nh * splits * (dv + 2);
 }
+// the head size by which decode_splits plans a launch: keys and values of unlike sizes run as heads of 64 or 128
+inline int decode_head(int dh, int dv) { return dv > 0 && dv != dh ? ((dh > dv ? dh : dv) <= 64 ? 64 : 128) : dh; }
 // The context length a step is planned for: the longest live request rounded up to a power of two, at least 4,096, at
 // most the model's maximum.  Captured decode steps are kept per (batch bucket, this bucket), so a model with a context of
 // 32k that serves short requests cuts their keys as a model of 4k would.  (Below 4,096 the measured optimum does not move:
@@ -236,9 +239,12 @@ inline int context_bucket(int longest, int max_positions) {
 }
 
 // Head and page sizes for which the tcgen05 prefill attention is built (the page must divide a tile of 128 keys and
-// fill whole groups of 8 swizzled rows).
-inline bool attention_tcgen05_takes(int dh, int page_size) {
-    return (dh == 64 || dh == 128) && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64 || page_size == 128);
+// fill whole groups of 8 swizzled rows): heads of 64 and 128, and keys and values of unlike sizes that are multiples of 8 up to 128
+// (`dv` 0: as dh), which run padded to 64 or 128.
+inline bool attention_unlike_heads(int dh, int dv) { return dv > 0 && dv != dh && dh % 8 == 0 && dv % 8 == 0 && dh <= 128 && dv <= 128; }
+inline bool attention_tcgen05_takes(int dh, int page_size, int dv = 0) {
+    const bool size = dv > 0 && dv != dh ? attention_unlike_heads(dh, dv) : (dh == 64 || dh == 128);
+    return size && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64 || page_size == 128);
 }
 
 // ---- which kernel takes a bfloat16 product ------------------------------------------------------------------------

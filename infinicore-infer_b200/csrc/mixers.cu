@@ -130,7 +130,7 @@ JK_EXPORT int jk_layernorm(const float *src, const int *rows, int nrows, int d, 
     const size_t smem = (size_t)d * sizeof(float);
 #define LN_LAUNCH(T, VEC)                                                                                                   \
     do {                                                                                                                    \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(layernorm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(layernorm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         jk_launch(layernorm_kernel<T, VEC>, dim3(nrows), dim3(threads), smem, stream, src, rows, w, b, eps, x_add, (T *)out, d);   \
     } while (0)
     if (dtype == JK_F32) {
@@ -445,10 +445,10 @@ JK_EXPORT int jk_conv_qkv(const float *u, int ld, int q_off, int k_off, int v_of
     int threads = C >= 2048 ? 512 : (C >= 512 ? 256 : 128);
     if (T <= 64) threads = std::min(1024, std::max(threads, (C / 2 + 31) / 32 * 32));
     if (dtype == JK_F32) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(conv_qkv_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (smem > 46 * 1024) cudaFuncSetAttribute(conv_qkv_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         jk_launch(conv_qkv_kernel<float>, dim3(T), dim3(threads), smem, stream, a);
     } else if (dtype == JK_BF16) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(conv_qkv_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (smem > 46 * 1024) cudaFuncSetAttribute(conv_qkv_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         jk_launch(conv_qkv_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, stream, a);
     } else {
         JK_FAIL(JK_UNSUPPORTED, "conv_qkv: dtype %d", dtype);
@@ -990,15 +990,16 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
         SCAN_LAUNCH_T(float, true);
     JK_CHECK_LAUNCH("linear_scan");
     if (n_pieces > 0) {
+        // (beside its dynamic shared memory the prefix kernel has some of its own: 48 KB of both together need no attribute)
         jk_launch(scan_carry_kernel, dim3((dk * dv + 255) / 256, heads, n_piece_reqs), dim3(256), 0, stream, a);
         JK_CHECK_LAUNCH("scan_carry");
         if (dv <= 64) {
             const size_t pfx = pfx_smem(64, dk);
-            if (pfx > 48 * 1024) cudaFuncSetAttribute(scan_prefix_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pfx);
+            if (pfx > 46 * 1024) cudaFuncSetAttribute(scan_prefix_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pfx);
             jk_launch(scan_prefix_kernel<64>, dim3(n_pieces, heads, 1), dim3(128), pfx, stream, a);
         } else {
             const size_t pfx = pfx_smem(PFX_COLS, dk);
-            if (pfx > 48 * 1024) cudaFuncSetAttribute(scan_prefix_kernel<PFX_COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pfx);
+            if (pfx > 46 * 1024) cudaFuncSetAttribute(scan_prefix_kernel<PFX_COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pfx);
             jk_launch(scan_prefix_kernel<PFX_COLS>, dim3(n_pieces, heads, (dv + PFX_COLS - 1) / PFX_COLS), dim3(128), pfx, stream, a);
         }
         JK_CHECK_LAUNCH("scan_prefix");
@@ -1499,7 +1500,7 @@ JK_EXPORT int jk_delta_rule(const float *c, int ld_c, int q_off, int k_off, int 
 #define LAUNCH(NPER)                                                                                                                         \
     do {                                                                                                                                     \
         const size_t smem = (size_t)2 * DR_ROWS * (2 * DR_LANES * (NPER + 4) + DR_COLS + 8) * sizeof(float);                                 \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<NPER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(delta_scan_kernel<NPER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
         jk_launch(delta_scan_kernel<NPER>, grid, dim3(DR_THREADS), smem, stream, a);                                                         \
     } while (0)
     if (nper == 4) LAUNCH(4); else if (nper == 8) LAUNCH(8); else if (nper == 16) LAUNCH(16); else LAUNCH(32);

@@ -261,12 +261,12 @@ int run_attention(Run &r, const RunnerOp &op) {
     JK_REQUIRE(table != nullptr, "runner: attention reads the cache of group %d, whose block table the step lacks", op.cache_group);
     const int n_short = r.st.list_n[op.list_short], n_tiles = r.st.list_n[op.list_tiles];
     const int *short_rows = r.st.lists[op.list_short], *tiles = r.st.lists[op.list_tiles];
-    const bool tc = !r.env.legacy_tensor_cores && g_fns.attention_tcgen05 != nullptr && jk::attention_tcgen05_takes(dh, page);
+    const bool tc = !r.env.legacy_tensor_cores && g_fns.attention_tcgen05 != nullptr && jk::attention_tcgen05_takes(dh, page, dv);
     bool fast = r.env.dtype == JK_BF16 && !r.env.plain_attention && (n_short > 0 || n_tiles > 0) && dh % 8 == 0 && dh <= 256;
-    // values of another size than the keys: the row kernel's (a sink, a gate, capped scores and kept first keys every
-    // kernel takes)
-    if (dv != dh) fast = false;
-    if (fast && n_tiles > 0 && !(tc || g_fns.attention_prefill_supports(dh))) fast = false;
+    // values of another size than the keys: the tcgen05 tiles and the split decode on tensor cores take them (padded to 64 or
+    // 128), the mma.sync tiles do not; else the row kernel (a sink, a gate, capped scores and kept first keys every kernel takes)
+    if (dv != dh && !jk::attention_unlike_heads(dh, dv)) fast = false;
+    if (fast && n_tiles > 0 && !(tc || (dv == dh && g_fns.attention_prefill_supports(dh)))) fast = false;
     if (!fast) {
         // one warp per (row, head): float32, and every shape the tensor-core kernels are not built for
         RUN(attention, g_fns.attention_rows(q, op.k_pages, op.v_pages, o, r.env.dtype, r.st.positions, r.st.row_req, table,
@@ -279,7 +279,7 @@ int run_attention(Run &r, const RunnerOp &op) {
             RUN(attention_tcgen05, g_fns.attention_tcgen05(q, op.k_pages, op.v_pages, o, tiles, n_tiles, T, r.st.req_start, r.st.req_pos,
                                                            table, r.env.max_blocks, op.num_pages, page, nh, nkvh, dh, op.softmax_scale,
                                                            op.window, r.env.status, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w,
-                                                           op.gated == 2, r.stream));
+                                                           op.gated == 2, dv, r.stream));
         else
             RUN(attention, g_fns.attention_prefill(q, op.k_pages, op.v_pages, o, tiles, n_tiles, jk::TILE_ROWS, r.st.req_start,
                                                    r.st.req_pos, table, r.env.max_blocks, page, nh, nkvh, dh, op.softmax_scale,
@@ -287,14 +287,14 @@ int run_attention(Run &r, const RunnerOp &op) {
     }
     if (n_short > 0) {
         const int context = r.st.context > 0 ? r.st.context : op.max_positions;
-        const int splits = jk::decode_splits(n_short, nkvh, nh / nkvh, jk::decode_keys_hint(context, std::abs(op.window)), r.env.routing.sms, dh);
+        const int splits = jk::decode_splits(n_short, nkvh, nh / nkvh, jk::decode_keys_hint(context, std::abs(op.window)), r.env.routing.sms, jk::decode_head(dh, dv));
         void *scratch = nullptr;
-        const long long need = 4 * jk::decode_scratch_floats(n_short, nh, dh, splits);
+        const long long need = 4 * jk::decode_scratch_floats(n_short, nh, dv, splits);
         if (need > 0)
             if (int rc = r.slot(SLOT_DECODE, need, &scratch, "the split-key attention's partial results")) return rc;
         RUN(attention, g_fns.attention_decode(q, op.k_pages, op.v_pages, o, (float *)scratch, short_rows, n_short, r.st.positions,
                                               r.st.row_req, table, r.env.max_blocks, page, nh, nkvh, dh, op.softmax_scale, op.window,
-                                              splits, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w, op.gated == 2, r.stream));
+                                              splits, op.sink, gate, op.ld, op.cap, op.keep_first, op.sink_w, op.gated == 2, dv, r.stream));
     }
     return JK_OK;
 }
@@ -983,8 +983,8 @@ JK_EXPORT int jk_runner_slot_bytes(const RunnerEnv *env, const RunnerOp *ops, in
                     const int c = context < op.max_positions ? context : op.max_positions;
                     for (int n = 1; n <= max_rows; ++n) {
                         const int s = jk::decode_splits(n, op.kv_heads, op.heads / op.kv_heads, jk::decode_keys_hint(c, std::abs(op.window)),
-                                                        env->routing.sms, op.head_dim);
-                        worst = std::max(worst, jk::decode_scratch_floats(n, op.heads, op.head_dim, s));
+                                                        env->routing.sms, jk::decode_head(op.head_dim, op.v_head_dim));
+                        worst = std::max(worst, jk::decode_scratch_floats(n, op.heads, op.v_head_dim > 0 ? op.v_head_dim : op.head_dim, s));
                         if (s <= 1) break;
                     }
                     if (context >= op.max_positions) break;

@@ -34,13 +34,13 @@ typedef int (*AttentionRowsFn)(const void *, const void *, const void *, void *,
                                cudaStream_t);
 typedef int (*AttentionDecodeFn)(const void *, const void *, const void *, void *, float *, const int *, int, const int *,
                                  const int *, const int *, int, int, int, int, int, float, int, int, int, const float *, int, float, int,
-                                 const float *, int, cudaStream_t);
+                                 const float *, int, int, cudaStream_t);
 typedef int (*AttentionPrefillFn)(const void *, const void *, const void *, void *, const int *, int, int, const int *,
                                   const int *, const int *, int, int, int, int, int, float, int, int, const float *, int, float, int,
                                   const float *, int, cudaStream_t);
 typedef int (*AttentionTcgen05Fn)(const void *, const void *, const void *, void *, const int *, int, int, const int *,
                                   const int *, const int *, int, int, int, int, int, int, float, int, int *, int, const float *, int,
-                                  float, int, const float *, int, cudaStream_t);
+                                  float, int, const float *, int, int, cudaStream_t);
 typedef int (*SupportsFn)(int, int, int);
 typedef int (*LinearSmallPartsFn)(const void *, long long, const int *, int, const void *, void *, int, int, int, int, int, cudaStream_t);
 typedef int (*Supports1Fn)(int);

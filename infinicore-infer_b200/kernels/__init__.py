@@ -503,9 +503,10 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     if rows is not None:
         _need(rows, "rows", torch.int32)
     _, nkvh, page_size, dh = k_pages.shape
+    dv = v_pages.shape[-1]
     lib = _build.load("attention")
     lib.jk_attention_decode_scratch_floats.restype = ctypes.c_longlong
-    need = lib.jk_attention_decode_scratch_floats(_c_int(nrows), _c_int(nh), _c_int(dh), _c_int(splits))
+    need = lib.jk_attention_decode_scratch_floats(_c_int(nrows), _c_int(nh), _c_int(dv), _c_int(splits))
     if need and scratch is None:
         scratch = torch.empty(need, dtype=torch.float32, device=q.device)
     if need:
@@ -516,7 +517,8 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(scratch if need else None), _ptr(rows), _c_int(nrows),
         _ptr(positions), _ptr(row_req), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(page_size),
         _c_int(nh), _c_int(nkvh), _c_int(dh), _c_float(scale), _c_int(window or 0), _c_int(splits), _c_int(1 if sink else 0),
-        *_gate_args(gate, 0, nh * (dh if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
+        *_gate_args(gate, 0, nh * (dv if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _c_int(dv),
+        _stream()))
     if need and splits > 1:
         global launch_count
         launch_count += 1          # the merge kernel
@@ -554,10 +556,10 @@ def attention_prefill(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
     return out
 
 
-def attention_tcgen05_supports(dh: int, page_size: int) -> bool:
-    """Head sizes 64 and 128 with pages that divide a tile of 128 keys and fill whole groups of 8 rows
+def attention_tcgen05_supports(dh: int, page_size: int, dv: int = 0) -> bool:
+    """Head sizes 64 and 128, or keys and values of unlike sizes up to 128, with pages that divide a tile of 128 keys and fill whole groups of 8 rows
     (``jk::attention_tcgen05_takes`` of csrc/host_rules.h; asking does not compile the kernel's module)."""
-    return _host.attention_tcgen05_takes(dh, page_size)
+    return _host.attention_tcgen05_takes(dh, page_size, dv)
 
 
 def attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
@@ -566,12 +568,14 @@ def attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                       gate: Optional[torch.Tensor] = None, cap: float = 0.0, keep_first: int = 0,
                       sink_w: Optional[torch.Tensor] = None, gate_elem: bool = False) -> torch.Tensor:
     """The same attention of TILE_ROWS-row query tiles on the tcgen05 tensor cores (TMA operands, both
-    products with accumulators in tensor memory); head sizes 64 and 128, pages that divide 128."""
+    products with accumulators in tensor memory); head sizes 64 and 128, or keys and values of unlike sizes (multiples of 8 up to
+    128), pages that divide 128."""
     for name, t in (("q", q), ("k_pages", k_pages), ("v_pages", v_pages), ("out", out)):
         _need(t, name, torch.bfloat16)
     for name, t in (("tiles", tiles), ("req_start", req_start), ("req_pos", req_pos), ("block_table", block_table)):
         _need(t, name, torch.int32)
     num_pages, nkvh, page_size, dh = k_pages.shape
+    dv = v_pages.shape[-1]
     if tiles.numel() < 2 * ntiles or q.numel() < ntok * nh * dh:
         raise KernelError("attention_tcgen05: the tile list or q is too short")
     lib = _build.load("attention_tcgen05")
@@ -579,7 +583,8 @@ def attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(tiles), _c_int(ntiles), _c_int(ntok), _ptr(req_start),
         _ptr(req_pos), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(num_pages), _c_int(page_size), _c_int(nh),
         _c_int(nkvh), _c_int(dh), _c_float(scale), _c_int(window or 0), _ptr(gemm_status(q.device)), _c_int(1 if sink else 0),
-        *_gate_args(gate, ntok, nh * (dh if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _stream()))
+        *_gate_args(gate, ntok, nh * (dv if gate_elem else 1)), _c_float(cap), _c_int(keep_first), _ptr(sink_w), _c_int(1 if gate_elem else 0), _c_int(dv),
+        _stream()))
     return out
 
 

@@ -129,8 +129,8 @@ def context_bucket(longest: int, max_positions: int) -> int:
     return lib().jk_context_bucket(longest, max_positions)
 
 
-def attention_tcgen05_takes(dh: int, page_size: int) -> bool:
-    return bool(lib().jk_attention_tcgen05_takes(dh, page_size))
+def attention_tcgen05_takes(dh: int, page_size: int, dv: int = 0) -> bool:
+    return bool(lib().jk_attention_tcgen05_takes(dh, page_size, dv))
 
 
 ROUTE_LIBRARY, ROUTE_SMALL, ROUTE_SKINNY, ROUTE_TCGEN05 = 0, 1, 2, 3

@@ -349,7 +349,7 @@ class ProgramRunner:
         self.env = rt.env(program.page_size, program.max_blocks)
         need_gemm = bool(program.lib.jk_runner_needs_gemm_tcgen05(ctypes.byref(self.env), program.ops, program.count, max_rows))
         need_attn = rt.dtype == torch.bfloat16 and not rt.legacy_tensor_cores and any(
-            program.ops[i].kind == 4 and _host.attention_tcgen05_takes(program.ops[i].head_dim, program.page_size)
+            program.ops[i].kind == 4 and _host.attention_tcgen05_takes(program.ops[i].head_dim, program.page_size, program.ops[i].v_head_dim)
             for i in range(program.count))
         need_mixers = any(program.ops[i].kind in _MIXERS_OPS or (program.ops[i].kind == OP["gate_up"] and program.ops[i].act > ACT["silu"])
                           for i in range(program.count))
