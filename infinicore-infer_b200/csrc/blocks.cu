@@ -2175,7 +2175,13 @@ struct EmbedPairArgs {
     int d;
 };
 
-template <typename TW>
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16 *p) {
+    const uint2 v = *reinterpret_cast<const uint2 *>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+
+template <typename TW, bool VEC>
 __global__ void embed_pair_kernel(EmbedPairArgs a) {
     pdl_trigger();
     pdl_wait();
@@ -2207,17 +2213,34 @@ __global__ void embed_pair_kernel(EmbedPairArgs a) {
     __syncthreads();
     const TW *add = a.pairs != nullptr ? (const TW *)a.pairs + (size_t)pair_row * a.d : nullptr;
     float *dst = a.x + (size_t)t * a.d;
+    float *keep = a.w == nullptr ? dst : row_buf;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
-        float v = a.scale * to_f32(src[c]);
-        if (add != nullptr) v += to_f32(add[c]);
-        if (a.w == nullptr) dst[c] = v;
-        else row_buf[c] = v;
-        ss += v * v;
+    if (VEC) {
+        for (int c = threadIdx.x * 4; c < a.d; c += blockDim.x * 4) {
+            float4 v = load4(src + c);
+            v = make_float4(v.x * a.scale, v.y * a.scale, v.z * a.scale, v.w * a.scale);
+            if (add != nullptr) {
+                const float4 b = load4(add + c);
+                v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+            }
+            *reinterpret_cast<float4 *>(keep + c) = v;
+            ss += sumsq4(v);
+        }
+    } else {
+        for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
+            float v = a.scale * to_f32(src[c]);
+            if (add != nullptr) v += to_f32(add[c]);
+            keep[c] = v;
+            ss += v * v;
+        }
     }
     if (a.w == nullptr) return;
     const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps);
-    for (int c = threadIdx.x; c < a.d; c += blockDim.x) dst[c] = row_buf[c] * inv * a.w[c];
+    if (VEC) {
+        for (int c = threadIdx.x * 4; c < a.d; c += blockDim.x * 4) *reinterpret_cast<float4 *>(dst + c) = scale4(load4(row_buf + c), inv, load4(a.w + c));
+    } else {
+        for (int c = threadIdx.x; c < a.d; c += blockDim.x) dst[c] = row_buf[c] * inv * a.w[c];
+    }
 }
 
 // tables of type `dtype`; pairs [buckets + 1, d]
@@ -2231,11 +2254,13 @@ JK_EXPORT int jk_embed_pair(const int *tokens, const int *positions, const int *
     const size_t smem = w != nullptr ? (size_t)d * sizeof(float) : 0;
     JK_REQUIRE(smem <= 200 * 1024, "embed_pair: width %d does not fit shared memory", d);
     const EmbedPairArgs a{tokens, positions, row_req, req_start, req_pos, slot_ids, table, pairs, buckets, mul_prev, mul_cur, scale, state, w, eps, x, d};
-    const int threads = T <= 64 ? std::min(1024, std::max(128, (d / 2 + 31) / 32 * 32)) : (d >= 1024 ? 256 : 128);
+    const bool vec = d % 4 == 0 && ((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)w | (uintptr_t)x) % 16 == 0;
+    const int threads = T <= 64 ? std::min(1024, std::max(128, (d / 4 + 31) / 32 * 32)) : (d >= 2048 ? 256 : 128);
 #define LAUNCH(TT)                                                                                                                     \
     do {                                                                                                                               \
-        if (smem > 46 * 1024) cudaFuncSetAttribute(embed_pair_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
-        jk_launch(embed_pair_kernel<TT>, dim3(T), dim3(threads), smem, stream, a);                                                     \
+        auto kernel = vec ? embed_pair_kernel<TT, true> : embed_pair_kernel<TT, false>;                                                \
+        if (smem > 46 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
+        jk_launch(kernel, dim3(T), dim3(threads), smem, stream, a);                                                                    \
     } while (0)
     BLOCKS_BY_DTYPE(dtype, "embed_pair", LAUNCH);
 #undef LAUNCH

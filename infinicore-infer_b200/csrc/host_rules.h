@@ -177,6 +177,11 @@ inline AttentionLists attention_work_lists(int B, int pad_B, const int *lens, co
 // `rows` rows has at most scan_max_pieces(rows) pieces.
 constexpr int SCAN_PIECE = 64;
 inline long long scan_max_pieces(long long rows) { return 2 * rows / SCAN_PIECE + 1; }
+// Whether the pieces of a recurrence run as tiled products within the piece (csrc/mixers.cu: piece_state, piece_rows): a constant decay per
+// head, rows that read the state after their own write, and sizes of whole vectors of four floats.
+inline bool scan_runs_tiled(int dk, int dv, int ld, int q_off, int k_off, int v_off, bool projected, bool bonus) {
+    return !projected && !bonus && dk <= 256 && ((dk | dv | ld | q_off | k_off | v_off) & 3) == 0;
+}
 inline long long scan_scratch_floats(long long rows, int heads, int dk, int dv, bool projected) {
     return scan_max_pieces(rows) * heads * dk * dv + (projected ? rows * heads * dk : 0);
 }

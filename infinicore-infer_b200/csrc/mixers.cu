@@ -480,7 +480,9 @@ JK_EXPORT int jk_conv_qkv(const float *u, int ld, int q_off, int k_off, int v_of
 // zeros: a piece leaves its rows' outputs without what came before the piece, its own end state in `piece_state`, and (for
 // a projected decay) the running product of the decays since the piece's start, b_t, in `cum`.  `scan_carry_kernel` then
 // walks each such request's pieces in order, S <- diag(b_end) S + S_piece, leaving in `piece_state` the state at each piece's
-// START and in the slot the state after the last; `scan_prefix_kernel` adds (q_t * b_t)^T S_start to the piece's rows.
+// START and in the slot the state after the last; `scan_prefix_kernel` adds (q_t * b_t)^T S_start to the piece's rows.  Where the decay is
+// a constant, the pieces do not walk their rows at all: their end states and rows are tiled products (`piece_state_kernel` ahead of the
+// carry, `piece_rows_kernel` behind it).
 // Nothing is ever divided by a decay.  The order of the sums of a row depends on where its piece starts (every SCAN_PIECE
 // rows from the start of its portion) and on nothing else of the batch.
 // ---------------------------------------------------------------------------------------------------------------
@@ -890,6 +892,237 @@ scan_prefix_kernel(ScanArgs a) {
     }
 }
 
+// ---- pieces of a recurrence with a constant decay d, as products within the piece ---------------------------------------------------------
+// With t, s the rows of a piece of n rows, the recurrence from zeros written out:
+//     end state   S_piece = sum_s d^(n-1-s) k_s v_s^T                               piece_state_kernel, ahead of the carry
+//     rows        o_t = d^(t+1) S_start^T q_t + sum_(s <= t) d^(t-s) (q_t . k_s) v_s    piece_rows_kernel, behind it
+// Everything is float32 on the CUDA cores, operands through shared memory by asynchronous copies, a register tile a thread; no power of the
+// decay is ever divided by, and those of a piece are made by repeated products.
+// ------------------------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void piece_copy16(float *dst, const float *src, bool valid) {
+    const int bytes = valid ? 16 : 0;           // 0 bytes read: the 16 bytes are filled with zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void piece_copies_done() {
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;\n" ::: "memory");
+}
+// the powers d^0 .. d^SCAN_PIECE (a thread each)
+__device__ __forceinline__ void piece_powers(float d, float *pw) {
+    if (threadIdx.x <= SCAN_PIECE) {
+        float b = 1.f;
+        for (int j = 0; j < threadIdx.x; ++j) b *= d;
+        pw[threadIdx.x] = b;
+    }
+}
+__device__ __forceinline__ float4 piece_act(int act, float4 v, float f) {
+    return make_float4(apply_act(act, v.x) * f, apply_act(act, v.y) * f, apply_act(act, v.z) * f, apply_act(act, v.w) * f);
+}
+
+// A block makes KB x CB of a piece's end state; thread (ty, tx) of 16 x 16 keeps key channels ty * 4 + {0..3} (and 64 on), columns
+// tx * 4 + {0..3} (and 64 on).
+template <int KB, int CB>
+__global__ void __launch_bounds__(256) piece_state_kernel(ScanArgs a) {
+    pdl_trigger();
+    constexpr int KH = KB / 64, CH = CB / 64;
+    extern __shared__ __align__(16) float ps_sm[];      // [64][KB] keys, [64][CB] values
+    __shared__ float pw[SCAN_PIECE + 1];
+    float *Ks = ps_sm, *Vs = ps_sm + SCAN_PIECE * KB;
+    const int p = blockIdx.x, head = blockIdx.y, nkb = (a.dk + KB - 1) / KB;
+    const int k0 = (blockIdx.z % nkb) * KB, c0 = (blockIdx.z / nkb) * CB;
+    const int first = a.pieces[2 * p], n = a.pieces[2 * p + 1];
+    piece_powers(a.decay[head], pw);
+    pdl_wait();
+    const float *u = a.u + (size_t)first * a.ld;
+    for (int i = threadIdx.x; i < SCAN_PIECE * (KB / 4); i += 256) {
+        const int t = i / (KB / 4), kk = k0 + (i % (KB / 4)) * 4;
+        const bool valid = t < n && kk < a.dk;
+        piece_copy16(Ks + 4 * i, valid ? u + (size_t)t * a.ld + a.k_off + head * a.dk + kk : u, valid);
+    }
+    for (int i = threadIdx.x; i < SCAN_PIECE * (CB / 4); i += 256) {
+        const int t = i / (CB / 4), c = c0 + (i % (CB / 4)) * 4;
+        const bool valid = t < n && c < a.dv;
+        piece_copy16(Vs + 4 * i, valid ? u + (size_t)t * a.ld + a.v_off + head * a.dv + c : u, valid);
+    }
+    piece_copies_done();
+    __syncthreads();            // the powers
+    for (int i = threadIdx.x; i < SCAN_PIECE * (KB / 4); i += 256) {        // what this thread brought itself
+        const int t = i / (KB / 4);
+        float4 *v = reinterpret_cast<float4 *>(Ks) + i;
+        *v = piece_act(a.qkv_act, *v, t < n ? pw[n - 1 - t] : 0.f);
+    }
+    if (a.qkv_act != ACT_NONE)
+        for (int i = threadIdx.x; i < SCAN_PIECE * (CB / 4); i += 256) {
+            float4 *v = reinterpret_cast<float4 *>(Vs) + i;
+            *v = piece_act(a.qkv_act, *v, 1.f);
+        }
+    __syncthreads();
+    const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+    float acc[4 * KH][4 * CH];
+#pragma unroll
+    for (int r = 0; r < 4 * KH; ++r)
+#pragma unroll
+        for (int c = 0; c < 4 * CH; ++c) acc[r][c] = 0.f;
+#pragma unroll 2
+    for (int t = 0; t < n; ++t) {
+        float kv[4 * KH], vv[4 * CH];
+#pragma unroll
+        for (int h = 0; h < KH; ++h) *reinterpret_cast<float4 *>(kv + 4 * h) = *reinterpret_cast<const float4 *>(Ks + t * KB + 64 * h + ty * 4);
+#pragma unroll
+        for (int h = 0; h < CH; ++h) *reinterpret_cast<float4 *>(vv + 4 * h) = *reinterpret_cast<const float4 *>(Vs + t * CB + 64 * h + tx * 4);
+#pragma unroll
+        for (int r = 0; r < 4 * KH; ++r)
+#pragma unroll
+            for (int c = 0; c < 4 * CH; ++c) acc[r][c] = fmaf(kv[r], vv[c], acc[r][c]);
+    }
+    float *S = a.piece_state + ((size_t)p * a.heads + head) * a.dk * a.dv;
+#pragma unroll
+    for (int r = 0; r < 4 * KH; ++r) {
+        const int kk = k0 + 64 * (r / 4) + ty * 4 + (r & 3);
+        if (kk >= a.dk) continue;
+#pragma unroll
+        for (int h = 0; h < CH; ++h) {
+            const int c = c0 + 64 * h + tx * 4;
+            if (c < a.dv) *reinterpret_cast<float4 *>(S + (size_t)kk * a.dv + c) = make_float4(acc[r][4 * h], acc[r][4 * h + 1], acc[r][4 * h + 2], acc[r][4 * h + 3]);
+        }
+    }
+}
+
+// A block makes the 64 rows x COLS columns of a piece and head.  First the weights A[t, s] = d^(t-s) (q_t . k_s) for s <= t (thread (ty, tx)
+// of 16 x 16: rows ty * 4 + {0..3}, columns tx + 16 {0..3}); then warp w has rows 8 w .. 8 w + 7, a lane four neighbouring columns.
+template <int COLS>
+__global__ void __launch_bounds__(256, 2) piece_rows_kernel(ScanArgs a) {
+    pdl_trigger();
+    constexpr int L = COLS / 4, GROUPS = 32 / L, ROWS = 8 / GROUPS, AL = SCAN_PIECE + 4;      // lanes a row; rows a thread
+    extern __shared__ __align__(16) float pr_sm[];
+    __shared__ float pw[SCAN_PIECE + 1];
+    const int dkp = a.dk + 4;           // rows of q and k four floats apart in their banks
+    float *Qs = pr_sm, *As = Qs + SCAN_PIECE * dkp, *B = As + SCAN_PIECE * AL;      // B: keys, then pieces of the state, then values
+    const int p = blockIdx.x, head = blockIdx.y, c0 = blockIdx.z * COLS;
+    const int first = a.pieces[2 * p], n = a.pieces[2 * p + 1];
+    piece_powers(a.decay[head], pw);
+    pdl_wait();
+    const float *u = a.u + (size_t)first * a.ld;
+    const int quads = a.dk / 4;
+    for (int i = threadIdx.x; i < SCAN_PIECE * quads; i += 256) {
+        const int t = i / quads, kk = (i - t * quads) * 4;
+        const float *row = t < n ? u + (size_t)t * a.ld + head * a.dk + kk : u;
+        piece_copy16(Qs + t * dkp + kk, t < n ? row + a.q_off : u, t < n);
+        piece_copy16(B + t * dkp + kk, t < n ? row + a.k_off : u, t < n);
+    }
+    piece_copies_done();
+    for (int i = threadIdx.x; i < SCAN_PIECE * quads; i += 256) {
+        const int t = i / quads, kk = (i - t * quads) * 4;
+        float4 *q = reinterpret_cast<float4 *>(Qs + t * dkp + kk), *k = reinterpret_cast<float4 *>(B + t * dkp + kk);
+        *q = piece_act(a.qkv_act, *q, a.q_scale);
+        if (a.qkv_act != ACT_NONE) *k = piece_act(a.qkv_act, *k, 1.f);
+    }
+    __syncthreads();
+    {
+        const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+        float acc[4][4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) acc[r][c] = 0.f;
+        for (int kk = 0; kk < a.dk; kk += 4) {
+            float4 q[4], k[4];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) q[r] = *reinterpret_cast<const float4 *>(Qs + (ty * 4 + r) * dkp + kk);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) k[c] = *reinterpret_cast<const float4 *>(B + (tx + 16 * c) * dkp + kk);
+#pragma unroll
+            for (int r = 0; r < 4; ++r)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    acc[r][c] = fmaf(q[r].x, k[c].x, acc[r][c]); acc[r][c] = fmaf(q[r].y, k[c].y, acc[r][c]);
+                    acc[r][c] = fmaf(q[r].z, k[c].z, acc[r][c]); acc[r][c] = fmaf(q[r].w, k[c].w, acc[r][c]);
+                }
+        }
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int t = ty * 4 + r, s = tx + 16 * c;
+                As[t * AL + s] = s <= t ? acc[r][c] * pw[t - s] : 0.f;
+            }
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = warp * 8 + (lane / L) * ROWS, cl = (lane % L) * 4;
+    float acc[ROWS][4];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) acc[r][c] = 0.f;
+    // acc += X[t0 + r, x0 .. x0 + count) B[.., columns]: X rows of `ldx` floats, count a multiple of four
+    auto rows_product = [&](const float *X, int ldx, int count) {
+        for (int j = 0; j < count; j += 4) {
+            float4 b[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) b[e] = *reinterpret_cast<const float4 *>(B + (j + e) * COLS + cl);
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r) {
+                const float4 x = *reinterpret_cast<const float4 *>(X + (t0 + r) * ldx + j);
+                acc[r][0] = fmaf(x.w, b[3].x, fmaf(x.z, b[2].x, fmaf(x.y, b[1].x, fmaf(x.x, b[0].x, acc[r][0]))));
+                acc[r][1] = fmaf(x.w, b[3].y, fmaf(x.z, b[2].y, fmaf(x.y, b[1].y, fmaf(x.x, b[0].y, acc[r][1]))));
+                acc[r][2] = fmaf(x.w, b[3].z, fmaf(x.z, b[2].z, fmaf(x.y, b[1].z, fmaf(x.x, b[0].z, acc[r][2]))));
+                acc[r][3] = fmaf(x.w, b[3].w, fmaf(x.z, b[2].w, fmaf(x.y, b[1].w, fmaf(x.x, b[0].w, acc[r][3]))));
+            }
+        }
+    };
+    // what came before the piece: the state at its start, 64 key channels at a time
+    const float *S = a.piece_state + ((size_t)p * a.heads + head) * a.dk * a.dv;
+    for (int kb = 0; kb < a.dk; kb += SCAN_PIECE) {
+        const int nk = min(SCAN_PIECE, a.dk - kb);
+        __syncthreads();
+        for (int i = threadIdx.x; i < nk * L; i += 256) {
+            const int kk = i / L, c = c0 + (i % L) * 4;
+            const bool valid = c < a.dv;
+            piece_copy16(B + 4 * i, valid ? S + (size_t)(kb + kk) * a.dv + c : S, valid);
+        }
+        piece_copies_done();
+        __syncthreads();
+        rows_product(Qs + kb, dkp, nk);
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) acc[r][c] *= pw[t0 + r + 1];
+    // the piece's own rows
+    __syncthreads();
+    for (int i = threadIdx.x; i < SCAN_PIECE * L; i += 256) {
+        const int t = i / L, c = c0 + (i % L) * 4;
+        const bool valid = t < n && c < a.dv;
+        piece_copy16(B + 4 * i, valid ? u + (size_t)t * a.ld + a.v_off + head * a.dv + c : u, valid);
+    }
+    piece_copies_done();
+    if (a.qkv_act != ACT_NONE)
+        for (int i = threadIdx.x; i < SCAN_PIECE * L; i += 256) {
+            float4 *v = reinterpret_cast<float4 *>(B) + i;
+            *v = piece_act(a.qkv_act, *v, 1.f);
+        }
+    __syncthreads();
+    rows_product(As, AL, warp * 8 + 8);        // no row of the warp sees a later one
+    if (c0 + cl < a.dv) {
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+            if (t0 + r < n)
+                *reinterpret_cast<float4 *>(a.out + ((size_t)(first + t0 + r) * a.heads + head) * a.dv + c0 + cl) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+    }
+}
+
+template <int KB, int CB>
+static void launch_piece_state(const ScanArgs &a, cudaStream_t stream) {
+    const size_t smem = sizeof(float) * SCAN_PIECE * (KB + CB);
+    cudaFuncSetAttribute(piece_state_kernel<KB, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    jk_launch(piece_state_kernel<KB, CB>, dim3(a.n_pieces, a.heads, ((a.dk + KB - 1) / KB) * ((a.dv + CB - 1) / CB)), dim3(256), smem, stream, a);
+}
+template <int COLS>
+static void launch_piece_rows(const ScanArgs &a, cudaStream_t stream) {
+    const size_t smem = sizeof(float) * SCAN_PIECE * ((a.dk + 4) + (SCAN_PIECE + 4) + std::max(a.dk + 4, COLS));
+    cudaFuncSetAttribute(piece_rows_kernel<COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    jk_launch(piece_rows_kernel<COLS>, dim3(a.n_pieces, a.heads, (a.dv + COLS - 1) / COLS), dim3(256), smem, stream, a);
+}
+
 // Rows of scratch the pieces of a step of `rows` rows need at most: piece_state floats, cum floats.
 JK_EXPORT long long jk_linear_scan_scratch_floats(int rows, int heads, int dk, int dv, int projected) {
     return jk::scan_scratch_floats(rows, heads, dk, dv, projected != 0);
@@ -916,13 +1149,15 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
     // lanes per column: as few as keep a thread's state at 64 values (more beyond 1024 and 512 channels); more of them,
     // and so fewer columns a block and more blocks, while the blocks do not fill the SMs
     const int sm_count = sms > 0 ? sms : 148;
-    const int items = n_direct + n_pieces;
+    const bool tiled = n_pieces > 0 && jk::scan_runs_tiled(dk, dv, ld, q_off, k_off, v_off, w2 != nullptr, bonus != nullptr) &&
+                       ((uintptr_t)u | (uintptr_t)scratch | (uintptr_t)out) % 16 == 0;
+    const int items = n_direct + (tiled ? 0 : n_pieces);        // of the scan kernel
     auto lanes_for = [&](int c) {
         int q = 1;
         while (q < 32 && (dk + q - 1) / q > 64 / c) q *= 2;
         return q;
     };
-    int cpt = n_pieces > 0 ? 4 : 2;
+    int cpt = items > n_direct ? 4 : 2;
     int kq = lanes_for(cpt);
     // a block's columns beyond a head's values are idle threads: fewer columns a thread first, then more lanes a column
     if (cpt == 4 && SCAN_THREADS / kq * cpt > dv) {
@@ -930,7 +1165,7 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
         kq = lanes_for(cpt);
     }
     while (kq < 32 && 2 * kq <= dk && SCAN_THREADS / kq * cpt > dv) kq *= 2;
-    while (kq < 32 && 2 * kq <= dk && (long long)heads * items * ((dv + SCAN_THREADS / kq * cpt - 1) / (SCAN_THREADS / kq * cpt)) < sm_count)
+    while (kq < 32 && 2 * kq <= dk && (long long)heads * std::max(items, 1) * ((dv + SCAN_THREADS / kq * cpt - 1) / (SCAN_THREADS / kq * cpt)) < sm_count)
         kq *= 2;
     const int cols = SCAN_THREADS / kq * cpt;
     const int per_thread = (dk + kq - 1) / kq;
@@ -961,7 +1196,7 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
 #define SCAN_LAUNCH_C(TW, KS, C, P)                                         \
     do {                                                                    \
         if constexpr (KS * C <= 16) {                                       \
-            if (n_pieces > 0) SCAN_LAUNCH_O(TW, KS, C, P, 3);               \
+            if (items > n_direct) SCAN_LAUNCH_O(TW, KS, C, P, 3);               \
             else SCAN_LAUNCH_O(TW, KS, C, P, 2);                            \
         } else {                                                            \
             SCAN_LAUNCH_O(TW, KS, C, P, 2);                                 \
@@ -982,7 +1217,9 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
         else if (per_thread <= 32) SCAN_LAUNCH(TW, 32, P);     \
         else SCAN_LAUNCH(TW, 64, P);                           \
     } while (0)
-    if (w2 == nullptr)
+    if (items == 0)
+        ;
+    else if (w2 == nullptr)
         SCAN_LAUNCH_T(float, false);
     else if (w2_dtype == JK_BF16)
         SCAN_LAUNCH_T(__nv_bfloat16, true);
@@ -990,9 +1227,21 @@ JK_EXPORT int jk_linear_scan(const float *u, int ld, int q_off, int k_off, int v
         SCAN_LAUNCH_T(float, true);
     JK_CHECK_LAUNCH("linear_scan");
     if (n_pieces > 0) {
+        if (tiled) {
+            if (dk <= 64) { if (dv <= 64) launch_piece_state<64, 64>(a, stream); else launch_piece_state<64, 128>(a, stream); }
+            else { if (dv <= 64) launch_piece_state<128, 64>(a, stream); else launch_piece_state<128, 128>(a, stream); }
+            JK_CHECK_LAUNCH("piece_state");
+        }
         // (beside its dynamic shared memory the prefix kernel has some of its own: 48 KB of both together need no attribute)
         jk_launch(scan_carry_kernel, dim3((dk * dv + 255) / 256, heads, n_piece_reqs), dim3(256), 0, stream, a);
         JK_CHECK_LAUNCH("scan_carry");
+        if (tiled) {
+            if (dv <= 32) launch_piece_rows<32>(a, stream);
+            else if (dv <= 64) launch_piece_rows<64>(a, stream);
+            else launch_piece_rows<128>(a, stream);
+            JK_CHECK_LAUNCH("piece_rows");
+            return JK_OK;
+        }
         if (dv <= 64) {
             const size_t pfx = pfx_smem(64, dk);
             if (pfx > 46 * 1024) cudaFuncSetAttribute(scan_prefix_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pfx);

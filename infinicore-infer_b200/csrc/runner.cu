@@ -518,7 +518,9 @@ int run_linear_attention(Run &r, const RunnerOp &op) {
                                   r.st.nreq, T, (float *)mix, r.st.lists[op.list_short], r.st.list_n[op.list_short],
                                   r.st.lists[op.list_tiles], n_pieces, r.st.lists[op.list_aux], r.st.list_n[op.list_aux],
                                   (float *)scratch, scratch_floats, r.env.routing.sms, op.bonus, op.decay_form, op.rank_act, r.stream));
-    if (n_pieces > 0) g_launches += 2;      // the carry and the prefix kernels
+    // the carry and the prefix kernels; pieces that run as tiled products have a kernel beside the one of the requests that run in one go
+    if (n_pieces > 0)
+        g_launches += 2 + (r.st.list_n[op.list_short] > 0 && jk::scan_runs_tiled(op.head_dim, dv, op.ld, op.q_off, op.k_off, op.v_off, op.w2 != nullptr, op.bonus != nullptr) ? 1 : 0);
     RUN(mixers, g_fns.norm_gate((const float *)mix, (const float *)u, op.ld, op.g_off, op.vec, op.eps, op.heads, dv, op.per_head_norm,
                                 op.gate_act, out, r.env.dtype, T, r.stream));
     return JK_OK;
