@@ -121,7 +121,7 @@ PRESETS: Dict[str, Preset] = {
         token_side={"dim": 16}, layers=[
             {"type": "parallel", "mixer": {
                 "left": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.25, "conv": 4, "rot": {"base": 1e4, "dims": 16}},
-                "right": {"heads": 3, "dim": 16, "vdim": 24, "decay": [0.75, 0.96875, 0.998], "rot": {"base": 1e5, "dims": 16}}},
+                "right": {"heads": 3, "dim": 16, "vdim": 24, "decay": [0.75, 0.97, 0.998], "rot": {"base": 1e5, "dims": 16}}},
              "mlp": {"kind": "moe", "router": {"experts": 6, "top": 2, "scale": 1.5}, "expert": {"ff": 48}, "shared": {"ff": 64}}},
             {"type": "rglru", "mixer": {"width": 128, "blocks": 4, "conv": 3}, "mlp": {"kind": "dense", "ff": 160}},
             {"type": "parallel", "mixer": {

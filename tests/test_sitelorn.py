@@ -260,7 +260,7 @@ def scan_inputs(T, H, dk, dv, rank, seed):
     return u, ld
 
 
-@pytest.mark.parametrize("H,dk,dv", [(1, 40, 72), (3, 24, 16), (2, 128, 128), (5, 7, 3)])
+@pytest.mark.parametrize("H,dk,dv", [(1, 40, 72), (3, 24, 16), (2, 128, 128), (5, 7, 3), (2, 64, 128), (1, 96, 64), (1, 200, 36)])
 @pytest.mark.parametrize("projected", [False, True])
 def test_recurrence_carries_its_state_across_cuts_and_slots(H, dk, dv, projected):
     """One sequence run whole, and cut into portions (one of a single row) that go through a state slot; a second
