@@ -2422,22 +2422,31 @@ template <typename T, bool OUT>
 __device__ __forceinline__ float gated_walk(const GatedArgs &g, int c, int first, int last, float s, float *prod) {
     const float yb = OUT && g.y_bias != nullptr ? g.y_bias[c] : 0.f;
     float p = 1.f;
-    for (int t0 = first; t0 < last; t0 += GS_AHEAD) {
-        float a[GS_AHEAD], b[GS_AHEAD], y[GS_AHEAD];
+    float a[2][GS_AHEAD], b[2][GS_AHEAD], y[2][GS_AHEAD];       // two groups of rows that take turns: one on its way, one being walked
+    auto fetch = [&](int t0, float (&fa)[GS_AHEAD], float (&fb)[GS_AHEAD], float (&fy)[GS_AHEAD]) {
 #pragma unroll
         for (int j = 0; j < GS_AHEAD; ++j) {
             const size_t t = min(t0 + j, last - 1);
-            a[j] = g.a[t * g.C + c];
-            b[j] = g.b[t * g.C + c];
-            y[j] = OUT ? g.y[t * g.ld_y + c] : 0.f;
+            fa[j] = g.a[t * g.C + c];
+            fb[j] = g.b[t * g.C + c];
+            fy[j] = OUT ? g.y[t * g.ld_y + c] : 0.f;
         }
+    };
+    auto walk = [&](int t0, const float (&fa)[GS_AHEAD], const float (&fb)[GS_AHEAD], const float (&fy)[GS_AHEAD]) {
 #pragma unroll
         for (int j = 0; j < GS_AHEAD; ++j) {
             if (t0 + j >= last) break;
-            s = fmaf(a[j], s, b[j]);
-            if (OUT) ((T *)g.out)[(size_t)(t0 + j) * g.C + c] = from_f32<T>(s * block_act(g.act, y[j] + yb));
-            else p *= a[j];
+            s = fmaf(fa[j], s, fb[j]);
+            if (OUT) ((T *)g.out)[(size_t)(t0 + j) * g.C + c] = from_f32<T>(s * block_act(g.act, fy[j] + yb));
+            else p *= fa[j];
         }
+    };
+    fetch(first, a[0], b[0], y[0]);
+    for (int t0 = first; t0 < last; t0 += 2 * GS_AHEAD) {
+        if (t0 + GS_AHEAD < last) fetch(t0 + GS_AHEAD, a[1], b[1], y[1]);
+        walk(t0, a[0], b[0], y[0]);
+        if (t0 + 2 * GS_AHEAD < last) fetch(t0 + 2 * GS_AHEAD, a[0], b[0], y[0]);
+        if (t0 + GS_AHEAD < last) walk(t0 + GS_AHEAD, a[1], b[1], y[1]);
     }
     if (!OUT) *prod = p;
     return s;
